@@ -10,7 +10,7 @@ the group, and a (page, kv head) tile of ``page_size x head_dim`` is contiguous.
 """
 from __future__ import annotations
 
-from typing import Dict, Hashable, List, Optional, Tuple
+from typing import Dict, Hashable, List, Optional, Tuple, Union
 
 import torch
 
@@ -18,11 +18,16 @@ from ..parts import LayerCache, ModelPlan, PagedCacheSpec
 from .pages import CacheLayout, GroupLayout
 
 
-def cache_groups_of(plan: ModelPlan) -> Tuple[List[PagedCacheSpec], Dict[int, Tuple[int, int]]]:
+#: a cache id's own rows, or (cache id, "pooled") for the rows of its whole blocks
+CacheKey = Union[int, Tuple[int, str]]
+
+
+def cache_groups_of(plan: ModelPlan) -> Tuple[List[PagedCacheSpec], Dict[CacheKey, Tuple[int, int]]]:
     """Group the plan's cache ids by what they store.  Returns the group specs and
-    cache id -> (group, index inside the group)."""
+    cache id -> (group, index inside the group); a cache id that also keeps a row for every
+    whole block of tokens has those in a group of their own, under (cache id, "pooled")."""
     specs: List[PagedCacheSpec] = []
-    where: Dict[int, Tuple[int, int]] = {}
+    where: Dict[CacheKey, Tuple[int, int]] = {}
     counts: List[int] = []
     for entry, run in enumerate(plan.schedule):
         if plan.cache_id(entry) != entry:
@@ -31,13 +36,23 @@ def cache_groups_of(plan: ModelPlan) -> Tuple[List[PagedCacheSpec], Dict[int, Tu
         spec = mixer.cache_spec() if mixer is not None else None
         if spec is None:
             continue
-        if spec not in specs:
-            specs.append(spec)
-            counts.append(0)
-        g = specs.index(spec)
-        where[entry] = (g, counts[g])
-        counts[g] += 1
+        if spec.pool and (spec.window is None or spec.window < spec.pool):
+            raise ValueError(f"blocks of {spec.pool} tokens need a window that holds one, not {spec.window}")
+        for key, sp in [(entry, spec)] + ([((entry, "pooled"), spec.pooled())] if spec.pool else []):
+            if sp not in specs:
+                specs.append(sp)
+                counts.append(0)
+            g = specs.index(sp)
+            where[key] = (g, counts[g])
+            counts[g] += 1
     return specs, where
+
+
+def pages_for_tokens_each(specs: List[PagedCacheSpec], token_pages: int, max_slots: int) -> List[int]:
+    """Pages of every group for ``token_pages`` pages of tokens: as many, or, where a row stands
+    for a block of tokens, that fraction and a partly filled page for every request slot."""
+    return [token_pages if s.tokens_per_row == 1 else -(-token_pages // s.tokens_per_row) + max_slots
+            for s in specs]
 
 
 def bytes_per_page(plan: ModelPlan, page_size: int, dtype_bytes: int) -> List[int]:
@@ -83,10 +98,12 @@ def pool_sizes_for_bytes(plan: ModelPlan, page_size: int, dtype_bytes: int, kv_c
                     + -(-spec.keep_first // page_size)
                 sizes[g] = max(8, min(share, max_slots * per_request))
             left -= sizes[g] * per_page[g]
-    full_bytes = sum(per_page[g] for g in range(len(specs)) if sizes[g] is None)
+    # pages of tokens the rest pays for; a group whose rows stand for whole blocks takes a
+    # fraction of that many
+    full_bytes = sum(per_page[g] / specs[g].tokens_per_row for g in range(len(specs)) if sizes[g] is None)
     for g in range(len(specs)):
         if sizes[g] is None:
-            sizes[g] = max(8, left // max(1, full_bytes))
+            sizes[g] = max(8, int(left / max(1.0, full_bytes)) // specs[g].tokens_per_row)
     return [int(n) for n in sizes]
 
 
@@ -98,10 +115,10 @@ class KVCacheManager(CacheLayout):
                  poison: Optional[float] = None) -> None:
         specs, where = cache_groups_of(plan)
         if isinstance(num_pages, int):
-            num_pages = [num_pages] * len(specs)
+            num_pages = pages_for_tokens_each(specs, num_pages, max_slots)
         if len(num_pages) != len(specs):
             raise ValueError(f"{len(num_pages)} pool sizes for {len(specs)} cache groups")
-        super().__init__([GroupLayout(s.window, n, s.keep_first if s.window is not None else 0)
+        super().__init__([GroupLayout(s.window, n, s.keep_first if s.window is not None else 0, s.tokens_per_row)
                           for s, n in zip(specs, num_pages)],
                          page_size, max_slots, watermark)
         self.plan = plan
@@ -160,14 +177,19 @@ class KVCacheManager(CacheLayout):
             cid = self.plan.cache_id(entry)
             if cid not in self._where:
                 return None
-            g, idx = self._where[cid]
-            planes = self.storage[g][idx]
-            values = self.value_storage[g][idx] if g in self.value_storage else \
-                (planes[1] if planes.shape[0] > 1 else None)
-            view = LayerCache(planes[0], values, g,
-                              self.page_size, write=self.plan.schedule[entry].writes_cache)
+            write = self.plan.schedule[entry].writes_cache
+            view = self._pages_of(cid, write)
+            if (cid, "pooled") in self._where:
+                view.pooled = self._pages_of((cid, "pooled"), write)
             self._views[entry] = view
         return view
+
+    def _pages_of(self, key: CacheKey, write: bool) -> LayerCache:
+        g, idx = self._where[key]
+        planes = self.storage[g][idx]
+        values = self.value_storage[g][idx] if g in self.value_storage else \
+            (planes[1] if planes.shape[0] > 1 else None)
+        return LayerCache(planes[0], values, g, self.page_size, write=write)
 
     def layer_state(self, entry: int) -> Optional[torch.Tensor]:
         return self.states.get(self.plan.cache_id(entry))

@@ -89,6 +89,7 @@ class GroupLayout:
     window: Optional[int]      # None: all keys; W: the last W keys
     num_pages: int
     keep_first: int = 0        # with a window: the request's first tokens stay as well
+    tokens_per_row: int = 1    # a row stands for a whole block of this many tokens
 
 
 @dataclass
@@ -125,6 +126,11 @@ class CacheLayout:
     def pages_for_tokens(self, n_tokens: int) -> int:
         return -(-n_tokens // self.page_size)
 
+    def pages_in(self, group: int, n_tokens: int) -> int:
+        """Pages of ``group`` that ``n_tokens`` tokens of a request fill: a row a token, or a row
+        for every whole block."""
+        return -(-(n_tokens // self.groups[group].tokens_per_row) // self.page_size)
+
     def kept_pages(self, group: int) -> int:
         """Pages at the start of a request that a window group never gives back."""
         return self.pages_for_tokens(self.groups[group].keep_first)
@@ -134,7 +140,7 @@ class CacheLayout:
         is fed in portions of at most ``largest_portion`` tokens."""
         w = self.groups[group].window
         if w is None:
-            return self.pages_for_tokens(total_tokens)
+            return self.pages_in(group, total_tokens)
         span = min(total_tokens, w + max(1, largest_portion))
         return min(self.pages_for_tokens(total_tokens),
                    self.pages_for_tokens(span) + 1 + self.kept_pages(group))
@@ -182,19 +188,19 @@ class CacheLayout:
     def pages_needed(self, request_id: Hashable, n_new: int) -> List[int]:
         """New pages per group for ``n_new`` more tokens."""
         req = self.requests[request_id]
-        want = self.pages_for_tokens(req.length + n_new)
-        return [max(0, want - len(t)) for t in req.tables]
+        return [max(0, self.pages_in(g, req.length + n_new) - len(t)) for g, t in enumerate(req.tables)]
 
     def pages_needed_each(self, request_ids: Sequence[Hashable], n_new: int = 1) -> List[int]:
         """``pages_needed`` summed over many requests that each get ``n_new`` more tokens (a
         decode step of hundreds of requests asks this every step: one loop, no lists)."""
         need = [0] * len(self.groups)
         requests, page = self.requests, self.page_size
+        rows = [g.tokens_per_row for g in self.groups]
         for rid in request_ids:
             req = requests[rid]
-            want = -(-(req.length + n_new) // page)
+            n = req.length + n_new
             for g, t in enumerate(req.tables):
-                d = want - len(t)
+                d = -(-(n // rows[g]) // page) - len(t)
                 if d > 0:
                     need[g] += d
         return need
@@ -203,12 +209,13 @@ class CacheLayout:
         """``extend`` for every request in turn (the caller has made sure of the pages with
         ``pages_needed_each``; a request that finds none raises as ``extend`` does)."""
         requests, page, pools = self.requests, self.page_size, self.pools
+        rows = [g.tokens_per_row for g in self.groups]
         for rid in request_ids:
             req = requests[rid]
-            want = -(-(req.length + n_new) // page)
+            n = req.length + n_new
             grow = False
             for g, t in enumerate(req.tables):
-                d = want - len(t)
+                d = -(-(n // rows[g]) // page) - len(t)
                 if d > 0:
                     grow = True
                     if d > pools[g].num_free:         # all of a request's groups, or none
@@ -216,7 +223,7 @@ class CacheLayout:
                                          f"{pools[g].num_free} free")
             if grow:
                 for g, t in enumerate(req.tables):
-                    d = want - len(t)
+                    d = -(-(n // rows[g]) // page) - len(t)
                     if d > 0:
                         t.extend(pools[g].take(d, rid))
                         req.version += 1
@@ -238,7 +245,8 @@ class CacheLayout:
         fit = None
         for g, (table, pool) in enumerate(zip(req.tables, self.pools)):
             spare = pool.num_free - (keep_free[g] if keep_free is not None else 0)
-            n = (len(table) + max(0, spare)) * self.page_size - req.length
+            r = self.groups[g].tokens_per_row
+            n = ((len(table) + max(0, spare)) * self.page_size + 1) * r - 1 - req.length
             fit = n if fit is None else min(fit, n)
         return max(0, fit) if fit is not None else 1 << 30
 
@@ -266,9 +274,8 @@ class CacheLayout:
         for rid, n in zip(request_ids, counts):
             req = requests[rid]
             length = req.length + n
-            want = -(-length // page)
-            for t in req.tables:
-                if want > len(t):
+            for g, t in enumerate(req.tables):
+                if -(-(length // self.groups[g].tokens_per_row) // page) > len(t):
                     raise CacheInvariantError(f"request {rid!r} commits tokens it has no pages for")
             req.length = length
 
@@ -277,8 +284,7 @@ class CacheLayout:
         position ``length``, sees keys from ``length - W + 1`` on; pages wholly before
         that are given back now."""
         req = self.requests[request_id]
-        have = min((len(t) for t in req.tables), default=self.pages_for_tokens(req.length + n_new))
-        if self.pages_for_tokens(req.length + n_new) > have:
+        if any(self.pages_needed(request_id, n_new)):
             raise CacheInvariantError(f"request {request_id!r} commits tokens it has no pages for")
         req.length += n_new
         for g, group in enumerate(self.groups):
@@ -319,7 +325,7 @@ class CacheLayout:
             seen: Dict[int, Hashable] = {}
             for rid, req in self.requests.items():
                 table = req.tables[g]
-                if len(table) < self.pages_for_tokens(req.length):
+                if len(table) < self.pages_in(g, req.length):
                     raise CacheInvariantError(f"request {rid!r} has tokens without pages")
                 for j, p in enumerate(table):
                     kept = self.kept_pages(g)

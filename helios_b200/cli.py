@@ -80,11 +80,14 @@ def cmd_info(args: argparse.Namespace) -> int:
     for g, spec in enumerate(specs):
         n_ids = sum(1 for gg, _ in where.values() if gg == g)
         keeps = "every key" if spec.window is None else f"the last {spec.window} keys"
+        if spec.tokens_per_row > 1:
+            keeps = f"a row for every whole block of {spec.tokens_per_row} tokens"
         dims = f"{spec.head_dim}" if spec.value_dim in (None, spec.head_dim) else \
             f"{spec.head_dim} (values {spec.value_dim})"
         print(f"  group {g}: {n_ids} caches of {spec.num_kv_heads} KV heads x {dims}, keeps {keeps}: "
-              f"{per_page[g]:,} bytes a page, {pages[g]:,} pages = {pages[g] * args.block_size:,} tokens")
-    full = [n for n, s in zip(pages, specs) if s.window is None]
+              f"{per_page[g]:,} bytes a page, {pages[g]:,} pages = "
+              f"{pages[g] * args.block_size * spec.tokens_per_row:,} tokens")
+    full = [n * s.tokens_per_row for n, s in zip(pages, specs) if s.window is None]
     if full:
         print(f"  longest context: {min(full) * args.block_size:,} tokens (all requests together)")
     elif specs:

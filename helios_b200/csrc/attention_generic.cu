@@ -11,13 +11,25 @@
 // keeps (`keep_first`: j visible if j <= p and (p - j < window or j < keep_first)); a sink in
 // the softmax, a key without a value whose score is 0 or sink_values[h], so that the weights
 // are exp(s_j) / (exp(sink) + sum exp(s_j)); a gate per (token, head), the head's output times
-// sigmoid(gate[t, h]), or per output value (`gate_wide`: gate[t, h * vd + d]).
+// sigmoid(gate[t, h]), or per output value (`gate_wide`: gate[t, h * vd + d]); means of whole blocks
+// of `pool` tokens behind the window (`pooled`: a key and a value a block in pages of their own,
+// block b seen if (b + 1) * pool <= p - window + 1); a constant `factor` on the output.
 //
 // Scores, softmax and the weighted sum are float32.  The keys are walked in
 // runs of 32 from `lo`, so the order of every sum depends on the token's
 // position alone: not on how the request was cut into steps, nor on the rest of
 // the batch.
 #include "common.cuh"
+
+// Keys and values that stand for whole blocks of tokens; all null / 0: none.
+template <typename T>
+struct PooledPages {
+  const T* k;             // [page, kv head, slot, hd]
+  const T* v;             // [page, kv head, slot, vd]
+  const int* table;       // [requests, table_stride]
+  int table_stride;
+  int pool;
+};
 
 constexpr int ATTN_WARPS = 4;
 constexpr int ATTN_MAX_HD = 256;
@@ -30,7 +42,8 @@ __global__ void attention_generic_kernel(
     const int* __restrict__ positions, int n_rows, int nh, int nkv, int hd, int vd, int page_size,
     int window, float scale, const float* __restrict__ slopes, int sink,
     const T* __restrict__ gate, int gate_stride, const float* __restrict__ bias_table, int bias_rows,
-    const float* __restrict__ sink_values, int keep_first, int gate_wide) {
+    const float* __restrict__ sink_values, int keep_first, int gate_wide, PooledPages<T> pooled,
+    int out_stride, float factor) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float q_smem[ATTN_WARPS][ATTN_MAX_HD];
@@ -40,7 +53,7 @@ __global__ void attention_generic_kernel(
   const int t = row / nh, h = row - t * nh;
   const int kvh = h / (nh / nkv);
   const int pos = positions[t];
-  const int* table = block_table + (size_t)seq_of_token[t] * bt_stride;
+  const int* token_table = block_table + (size_t)seq_of_token[t] * bt_stride;
   const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
 
   float* qs = q_smem[warp];
@@ -55,11 +68,15 @@ __global__ void attention_generic_kernel(
   float m = -INFINITY, l = 0.f;
   const float slope = slopes ? slopes[h] : 0.f;
 
-  // two stretches of keys: the first tokens a window keeps (those it has passed), then the
-  // window itself; each in runs of 32 from its own first key
-  for (int stretch = 0; stretch < 2; ++stretch) {
-    const int first = stretch == 0 ? 0 : lo;
-    const int last = stretch == 0 ? min(keep_first, lo) - 1 : pos;
+  // three stretches of keys: the means of the blocks behind the window, the first tokens a
+  // window keeps (those it has passed), then the window itself; each in runs of 32 from its own
+  // first key
+  for (int stretch = pooled.pool > 0 ? -1 : 0; stretch < 2; ++stretch) {
+    const int first = stretch <= 0 ? 0 : lo;
+    const int last = stretch < 0 ? lo / pooled.pool - 1 : stretch == 0 ? min(keep_first, lo) - 1 : pos;
+    const int* table = stretch < 0 ? pooled.table + (size_t)seq_of_token[t] * pooled.table_stride : token_table;
+    const T* kp = stretch < 0 ? pooled.k : k_pages;
+    const T* vp = stretch < 0 ? pooled.v : v_pages;
     for (int base = first; base <= last; base += 32) {
       const int key = base + lane;
       const bool valid = key <= last;
@@ -67,7 +84,7 @@ __global__ void attention_generic_kernel(
       float score = -INFINITY;
       if (valid) {
         page = table[key / page_size];
-        const T* kr = k_pages + (((size_t)page * nkv + kvh) * page_size + key % page_size) * hd;
+        const T* kr = kp + (((size_t)page * nkv + kvh) * page_size + key % page_size) * hd;
         float dot = 0.f;
         for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], to_float(kr[d]), dot);
         score = dot * scale - slope * (float)(pos - key);
@@ -84,7 +101,7 @@ __global__ void attention_generic_kernel(
       for (int j = 0; j < n_valid; ++j) {
         const float pj = __shfl_sync(0xffffffffu, p, j);
         const int pagej = __shfl_sync(0xffffffffu, page, j);
-        const T* vr = v_pages + (((size_t)pagej * nkv + kvh) * page_size + (base + j) % page_size) * vd;
+        const T* vr = vp + (((size_t)pagej * nkv + kvh) * page_size + (base + j) % page_size) * vd;
 #pragma unroll
         for (int i = 0; i < ND; ++i) {
           const int d = lane + 32 * i;
@@ -101,9 +118,9 @@ __global__ void attention_generic_kernel(
 #pragma unroll
     for (int i = 0; i < ND; ++i) acc[i] *= corr;
   }
-  float inv = 1.f / l;
+  float inv = factor / l;
   if (gate && !gate_wide) inv /= 1.f + expf(-to_float(gate[(size_t)t * gate_stride + h]));
-  T* orow = out + (size_t)t * nh * vd + (size_t)h * vd;
+  T* orow = out + (size_t)t * out_stride + (size_t)h * vd;
 #pragma unroll
   for (int i = 0; i < ND; ++i) {
     const int d = lane + 32 * i;
@@ -121,11 +138,14 @@ HB_EXPORT int hb_attention_generic(void* out, const void* q, int q_stride, const
                                    int nkv, int hd, int vd, int page_size, int window, float scale,
                                    const float* slopes, int sink, const void* gate,
                                    int gate_stride, const float* bias_table, int bias_rows,
-                                   const float* sink_values, int keep_first, int gate_wide, int act_dt,
+                                   const float* sink_values, int keep_first, int gate_wide,
+                                   const void* pooled_k, const void* pooled_v, const int* pooled_table,
+                                   int pooled_table_stride, int pool, int out_stride, float factor, int act_dt,
                                    cudaStream_t stream) {
   if (T <= 0) return HB_OK;
   if (hd <= 0 || hd > ATTN_MAX_HD || vd <= 0 || vd > ATTN_MAX_HD || nkv <= 0 || nh % nkv != 0 ||
-      page_size <= 0 || keep_first < 0 || (bias_table != nullptr && bias_rows <= 0))
+      page_size <= 0 || keep_first < 0 || pool < 0 || out_stride < nh * vd ||
+      (pool > 0 && (window <= 0 || !pooled_k || !pooled_v || !pooled_table)) || (bias_table != nullptr && bias_rows <= 0))
     return HB_BAD_ARGUMENT;
   const int n_rows = T * nh;
   const int blocks = (n_rows + ATTN_WARPS - 1) / ATTN_WARPS;
@@ -134,6 +154,8 @@ HB_EXPORT int hb_attention_generic(void* out, const void* q, int q_stride, const
         (TA*)out, (const TA*)q, q_stride, (const TA*)k_pages, (const TA*)v_pages, block_table,
         bt_stride, seq_of_token, positions, n_rows, nh, nkv, hd, vd, page_size, window, scale,
         slopes, sink, (const TA*)gate, gate_stride, bias_table, bias_rows, sink_values, keep_first,
-        gate_wide));
+        gate_wide,
+        PooledPages<TA>{(const TA*)pooled_k, (const TA*)pooled_v, pooled_table, pooled_table_stride, pool},
+        out_stride, factor));
   return hb_check_launch();
 }

@@ -43,6 +43,8 @@ LIBRARIES: Dict[str, str] = {
     "delta_rule": "delta_rule.cu",
     "moe": "moe.cu",
     "ssm": "ssm.cu",
+    "linear_attention": "linear_attention.cu",
+    "pooled_window": "pooled_window.cu",
 }
 _HEADERS = ["common.cuh", "tcgen05.cuh"]
 # further files a library's source includes
@@ -50,7 +52,9 @@ _INCLUDES: Dict[str, List[str]] = {"gemm_bf16_noalloc": ["gemm_bf16.cu", "gemm_b
                                    "attention_bf16": ["attention_mma.cuh", "attention_options.cuh"],
                                    "attention_generic": ["attention_options.cuh"],
                                    "attention_tc": ["attention_options.cuh"],
-                                   "latent_attention": ["attention_mma.cuh"]}
+                                   "latent_attention": ["attention_mma.cuh"],
+                                   "delta_rule": ["causal_conv.cuh"],
+                                   "pooled_window": ["causal_conv.cuh"]}
 
 NVCC_FLAGS = [
     "-O3", "-std=c++17",

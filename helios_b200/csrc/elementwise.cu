@@ -610,6 +610,86 @@ HB_EXPORT int hb_rmsnorm_add(float* residual, const void* y, const float* weight
   return hb_check_launch();
 }
 
+// ---------------------------------------------------------------- norm of a weighted sum
+// residual[r, :] = norm(factor * residual[r, :] + y[r, :]) * weight (float32, RMS norm with eps
+// inside the root), for a block whose norm takes the SUM and gives the new stream; `copy` (may be
+// null) receives the new row in the activation dtype, which is what the next sublayer reads.
+// A row is held in registers between the two passes.
+template <typename TY, typename TC, bool VEC>
+__global__ void __launch_bounds__(NORM_THREADS)
+scaled_sum_rmsnorm_kernel(float* __restrict__ residual, const TY* __restrict__ y,
+                          const float* __restrict__ weight, TC* __restrict__ copy, int H, float eps,
+                          float factor) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  float* res = residual + (size_t)blockIdx.x * H;
+  const TY* yr = y + (size_t)blockIdx.x * H;
+  TC* cp = copy ? copy + (size_t)blockIdx.x * H : nullptr;
+  float ss = 0.f;
+  if constexpr (VEC) {
+    float v[NORM_GROUPS][4], d[NORM_GROUPS][4];
+#pragma unroll
+    for (int g = 0; g < NORM_GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) { load4(res + c, v[g]); load4(yr + c, d[g]); }
+    }
+#pragma unroll
+    for (int g = 0; g < NORM_GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[g][e] = fmaf(factor, v[g][e], d[g][e]);
+          ss = fmaf(v[g][e], v[g][e], ss);
+        }
+      }
+    }
+    const float rstd = rsqrtf(block_sum(ss, scratch) / (float)H + eps);
+#pragma unroll
+    for (int g = 0; g < NORM_GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) {
+        float w[4];
+        load4(weight + c, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[g][e] *= rstd * w[e];
+        store4(res + c, v[g]);
+        if (cp) store4(cp + c, v[g]);
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+      const float v = fmaf(factor, res[c], to_float(yr[c]));
+      res[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+    const float rstd = rsqrtf(block_sum(ss, scratch) / (float)H + eps);
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+      const float v = res[c] * rstd * weight[c];
+      res[c] = v;
+      if (cp) cp[c] = from_float<TC>(v);
+    }
+  }
+}
+
+HB_EXPORT int hb_scaled_sum_rmsnorm(float* residual, const void* y, const float* weight, void* copy, int n, int H,
+                                    float eps, float factor, int y_dt, int copy_dt, cudaStream_t stream) {
+  if (n <= 0) return HB_OK;
+  if (H <= 0) return HB_BAD_ARGUMENT;
+  const bool vec = H % 4 == 0 && H <= NORM_THREADS * NORM_GROUPS * 4 &&
+                   (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)weight | (uintptr_t)copy) & 15) == 0;
+  HB_DISPATCH_DTYPE(y_dt, TY,
+    HB_DISPATCH_DTYPE(copy_dt, TC,
+      if (vec)
+        hb_launch(scaled_sum_rmsnorm_kernel<TY, TC, true>, dim3(n), dim3(NORM_THREADS), 0, stream, residual,
+                  (const TY*)y, weight, (TC*)copy, H, eps, factor);
+      else
+        hb_launch(scaled_sum_rmsnorm_kernel<TY, TC, false>, dim3(n), dim3(NORM_THREADS), 0, stream, residual,
+                  (const TY*)y, weight, (TC*)copy, H, eps, factor)));
+  return hb_check_launch();
+}
+
 // ---------------------------------------------------------------- layer norm with a pending sum
 // A block whose sublayers all read ONE norm of the stream leaves its outputs to be added:
 //   residual[r, c] += mult * (sa[c] * a[r, c] + sb[c] * b[r, c])      (float32; a, b, sa, sb optional)

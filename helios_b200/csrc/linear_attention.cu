@@ -1,0 +1,560 @@
+// Linear attention with ONE fixed decay per head: per head, with q, k [N] and v [M] of a token
+// and the head's constant a,
+//
+//   S <- a S + k v^T        (S is [N, M], float32, carried from token to token in the request's slot)
+//   o  = S^T q
+//
+// q, k and v are columns of a fused projection's rows; on the way in they may pass silu, or q
+// and k a rotation of their first `rot` values (value i paired with value i + rot / 2, cos/sin
+// tables [T, rot / 2]); k is multiplied by key_scale.  All of that, the recurrence and the
+// norms and gates after it are float32.
+//
+// The decay is a constant, so a stretch of C tokens can be taken at once: with the state S0
+// before it,
+//   o_i = a^(i+1) S0^T q_i + sum_(j <= i) a^(i-j) (q_i . k_j) v_j
+//   S   = a^C S0 + sum_j a^(C-1-j) k_j v_j^T
+// Kernels:
+//   la_scan       token by token, a block per (request, head, 32 columns of S): steps of few
+//                 tokens a request
+//   la_chunk_kv   (portions) the sums k_j v_j^T of every chunk of 64 tokens, all chunks in parallel
+//   la_states     one pass over a request's chunks: the state before every chunk, and the slot's
+//   la_chunk_out  o of every chunk from the state before it and the chunk's own tokens, all
+//                 chunks in parallel; with a norm per head also norm and gate
+//   la_gate_norm  norm (per head or over the row) times the gate, for what the others leave as
+//                 plain float32 o
+// The products of the chunked form run on the float32 FMA pipes: the operands are float32 (a
+// rotated key, a decayed state), and nothing of the recurrence is rounded to 16 bits.
+#include "common.cuh"
+
+namespace {
+
+constexpr int LA_C = 64;             // tokens a chunk
+constexpr int LA_BLK = 64;           // rows / columns of S a tile
+constexpr int LA_LD = LA_BLK + 4;    // row stride of a tile in shared memory (16-byte rows)
+
+enum { LA_NONE = 0, LA_SILU = 1 };
+
+template <typename T>
+struct LaIn {
+  const T* rows;        // [tokens, ld]
+  int ld;
+  int q_off, k_off, v_off, g_off;
+  const float* cos;     // [tokens, half] or null
+  const float* sin;
+  int half;
+  int act;
+  float key_scale;
+  int vec;              // four neighbouring columns may be read at once
+};
+
+__device__ __forceinline__ float la_silu(float x) { return x / (1.f + expf(-x)); }
+
+// Column d of a q or k head (x: the head's first column of the token's row).
+template <typename T>
+__device__ __forceinline__ float la_qk(const LaIn<T>& in, const T* x, int t, int d) {
+  float v = to_float(x[d]);
+  if (in.act == LA_SILU) v = la_silu(v);
+  if (in.half > 0 && d < 2 * in.half) {
+    const int p = d < in.half ? d : d - in.half;
+    const float c = in.cos[(size_t)t * in.half + p], s = in.sin[(size_t)t * in.half + p];
+    const float o = to_float(x[d < in.half ? d + in.half : d - in.half]);
+    v = d < in.half ? v * c - o * s : v * c + o * s;
+  }
+  return v;
+}
+
+template <typename T>
+__device__ __forceinline__ void la_load4(const T* p, float (&f)[4]) {
+  if constexpr (sizeof(T) == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
+  } else {
+    const uint2 x = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+}
+
+// Columns d .. d + 3 of a q or k head (zeros from column N on).
+template <typename T>
+__device__ __forceinline__ void la_qk4(const LaIn<T>& in, const T* x, int t, int d, int N, float (&f)[4]) {
+  if (in.vec && d < N) {          // N, half and all offsets are multiples of 4
+    la_load4(x + d, f);
+    if (in.act == LA_SILU) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) f[e] = la_silu(f[e]);
+    }
+    if (d < 2 * in.half) {
+      const bool lower = d < in.half;
+      const int p = lower ? d : d - in.half;
+      const float4 c = *reinterpret_cast<const float4*>(in.cos + (size_t)t * in.half + p);
+      const float4 s = *reinterpret_cast<const float4*>(in.sin + (size_t)t * in.half + p);
+      float o[4];
+      la_load4(x + (lower ? d + in.half : d - in.half), o);
+      const float sg = lower ? -1.f : 1.f;
+      f[0] = f[0] * c.x + sg * o[0] * s.x;
+      f[1] = f[1] * c.y + sg * o[1] * s.y;
+      f[2] = f[2] * c.z + sg * o[2] * s.z;
+      f[3] = f[3] * c.w + sg * o[3] * s.w;
+    }
+    return;
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) f[e] = d + e < N ? la_qk(in, x, t, d + e) : 0.f;
+}
+
+template <typename T>
+__device__ __forceinline__ void la_v4(const LaIn<T>& in, const T* x, int d, int M, float (&f)[4]) {
+  if (in.vec && d < M) {
+    la_load4(x + d, f);
+  } else {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) f[e] = d + e < M ? to_float(x[d + e]) : 0.f;
+  }
+  if (in.act == LA_SILU) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) f[e] = la_silu(f[e]);
+  }
+}
+
+__device__ __forceinline__ float la_gate(float g, int kind) {
+  const float s = 1.f / (1.f + expf(-g));
+  return kind == 0 ? g * s : s;              // silu | sigmoid
+}
+
+// ---------------------------------------------------------------- token by token
+constexpr int LA_COLS = 32;          // columns of S a block owns, a lane each
+constexpr int LA_PARTS = 8;          // warps that share a column's rows
+constexpr int LA_STAGE = 8;          // tokens staged in shared memory at a time
+
+template <typename T, int ROWS>
+__global__ void __launch_bounds__(LA_COLS * LA_PARTS)
+la_scan_kernel(float* __restrict__ o, LaIn<T> in, float* __restrict__ state, long state_stride,
+               const float* __restrict__ powers, const int* __restrict__ cu_tokens,
+               const int* __restrict__ slots, int heads, int N, int M) {
+  pdl_launch_dependents();
+  constexpr int NP = ROWS * LA_PARTS;
+  __shared__ float qs[LA_STAGE][NP], ks[LA_STAGE][NP], vs[LA_STAGE][LA_COLS];
+  __shared__ float shares[2][LA_PARTS][LA_COLS];
+  const int h = blockIdx.y, seq = blockIdx.z;
+  const int lane = threadIdx.x & 31, part = threadIdx.x >> 5;
+  const int col0 = blockIdx.x * LA_COLS, col = col0 + lane;
+  const bool live = col < M;
+  const float a = powers[(size_t)h * (LA_C + 1) + 1];
+  const int t0 = cu_tokens[seq], t1 = cu_tokens[seq + 1];
+  float* S = state + (size_t)slots[seq] * state_stride + (size_t)h * N * M;
+  pdl_wait();
+  float s[ROWS];
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const int n = part + LA_PARTS * i;
+    s[i] = (live && n < N) ? S[(size_t)n * M + col] : 0.f;
+  }
+  int turn = 0;
+  for (int c0 = t0; c0 < t1; c0 += LA_STAGE) {
+    const int n_tok = min(LA_STAGE, t1 - c0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < n_tok * NP; i += blockDim.x) {
+      const int j = i / NP, n = i - j * NP;
+      const T* r = in.rows + (size_t)(c0 + j) * in.ld + h * N;
+      qs[j][n] = n < N ? la_qk(in, r + in.q_off, c0 + j, n) : 0.f;
+      ks[j][n] = n < N ? la_qk(in, r + in.k_off, c0 + j, n) * in.key_scale : 0.f;
+    }
+    for (int i = threadIdx.x; i < n_tok * LA_COLS; i += blockDim.x) {
+      const int j = i / LA_COLS, c = i - j * LA_COLS;
+      float v = col0 + c < M ? to_float(in.rows[(size_t)(c0 + j) * in.ld + in.v_off + (size_t)h * M + col0 + c]) : 0.f;
+      if (in.act == LA_SILU) v = la_silu(v);
+      vs[j][c] = v;
+    }
+    __syncthreads();
+    for (int j = 0; j < n_tok; ++j) {
+      const float v = vs[j][lane];
+      float acc = 0.f;
+#pragma unroll
+      for (int i = 0; i < ROWS; ++i) {
+        const int n = part + LA_PARTS * i;
+        s[i] = fmaf(a, s[i], ks[j][n] * v);
+        acc = fmaf(s[i], qs[j][n], acc);
+      }
+      shares[turn][part][lane] = acc;
+      __syncthreads();
+      if (part == 0 && live) {
+        float r = 0.f;
+#pragma unroll
+        for (int p = 0; p < LA_PARTS; ++p) r += shares[turn][p][lane];
+        o[((size_t)(c0 + j) * heads + h) * M + col] = r;
+      }
+      turn ^= 1;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const int n = part + LA_PARTS * i;
+    if (live && n < N) S[(size_t)n * M + col] = s[i];
+  }
+}
+
+// ---------------------------------------------------------------- chunks
+// q_tiles: (request, first token of the chunk inside the request's step) per chunk of LA_C tokens,
+// in the requests' order; a tile at or beyond the request's tokens holds no work.
+__device__ __forceinline__ int la_tile_tokens(const int* q_tiles, const int* cu_tokens, int tile, int& tok0) {
+  const int seq = q_tiles[2 * tile], l0 = q_tiles[2 * tile + 1];
+  const int begin = cu_tokens[seq], n = cu_tokens[seq + 1] - begin;
+  if (l0 >= n) return 0;
+  tok0 = begin + l0;
+  return min(LA_C, n - l0);
+}
+
+// acc[4][4] += A^T B over a shared-memory tile: A [64][LA_LD] and B [64][LA_LD] by the inner index.
+__device__ __forceinline__ void la_mma(float (&acc)[4][4], const float* A, const float* B, int ty, int tx, int inner) {
+#pragma unroll 8
+  for (int d = 0; d < inner; ++d) {
+    const float4 x = *reinterpret_cast<const float4*>(A + d * LA_LD + 4 * ty);
+    const float4 y = *reinterpret_cast<const float4*>(B + d * LA_LD + 4 * tx);
+    const float xa[4] = {x.x, x.y, x.z, x.w}, ya[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xa[i], ya[j], acc[i][j]);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+la_chunk_kv_kernel(float* __restrict__ sums, LaIn<T> in, const float* __restrict__ powers,
+                   const int* __restrict__ q_tiles, const int* __restrict__ cu_tokens, int heads, int N, int M) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float sm[];
+  float* Ks = sm;                              // [token][LA_LD]
+  float* Vs = sm + LA_C * LA_LD;               // [token][LA_LD]
+  const int tile = blockIdx.x, h = blockIdx.y;
+  const int vblocks = (M + LA_BLK - 1) / LA_BLK;
+  const int n0 = (blockIdx.z / vblocks) * LA_BLK, m0 = (blockIdx.z % vblocks) * LA_BLK;
+  int tok0 = 0;
+  const int n_tok = la_tile_tokens(q_tiles, cu_tokens, tile, tok0);
+  pdl_wait();
+  if (n_tok == 0) return;
+  const float* pw = powers + (size_t)h * (LA_C + 1);
+  for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
+    const int j = i / (LA_BLK / 4), d = (i - j * (LA_BLK / 4)) * 4;
+    float k4[4] = {0.f, 0.f, 0.f, 0.f}, v4[4] = {0.f, 0.f, 0.f, 0.f};
+    if (j < n_tok) {
+      const T* r = in.rows + (size_t)(tok0 + j) * in.ld;
+      la_qk4(in, r + in.k_off + (size_t)h * N, tok0 + j, n0 + d, N, k4);
+      la_v4(in, r + in.v_off + (size_t)h * M, m0 + d, M, v4);
+      const float f = in.key_scale * pw[n_tok - 1 - j];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) k4[e] *= f;
+    }
+    *reinterpret_cast<float4*>(Ks + j * LA_LD + d) = make_float4(k4[0], k4[1], k4[2], k4[3]);
+    *reinterpret_cast<float4*>(Vs + j * LA_LD + d) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+  }
+  __syncthreads();
+  const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+  float acc[4][4] = {};
+  la_mma(acc, Ks, Vs, ty, tx, n_tok);
+  float* dst = sums + ((size_t)tile * heads + h) * N * M;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int n = n0 + 4 * ty + i, m = m0 + 4 * tx;
+    if (n >= N) continue;
+    if ((M & 3) == 0) {
+      if (m < M) *reinterpret_cast<float4*>(dst + (size_t)n * M + m) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) if (m + e < M) dst[(size_t)n * M + m + e] = acc[i][e];
+    }
+  }
+}
+
+// sums[tile] (a chunk's own sum) becomes the state BEFORE the chunk; the slot's state moves on
+// to the end of the request's tokens.  A thread an entry of S; a request's chunks in order.
+__global__ void __launch_bounds__(256)
+la_states_kernel(float* __restrict__ sums, float* __restrict__ state, long state_stride,
+                 const float* __restrict__ powers, const int* __restrict__ cu_tokens,
+                 const int* __restrict__ slots, int heads, int NM) {
+  pdl_launch_dependents();
+  __shared__ int before[8];
+  const int h = blockIdx.y, seq = blockIdx.z;
+  // chunks of the requests before this one
+  int c = 0;
+  for (int s = threadIdx.x; s < seq; s += 256) c += (cu_tokens[s + 1] - cu_tokens[s] + LA_C - 1) / LA_C;
+  for (int w = 16; w > 0; w >>= 1) c += __shfl_xor_sync(0xffffffffu, c, w);
+  if ((threadIdx.x & 31) == 0) before[threadIdx.x >> 5] = c;
+  __syncthreads();
+  int tile = 0;
+  for (int w = 0; w < 8; ++w) tile += before[w];
+  const int n = cu_tokens[seq + 1] - cu_tokens[seq];
+  const int chunks = (n + LA_C - 1) / LA_C;
+  pdl_wait();
+  const int e = blockIdx.x * 256 + threadIdx.x;
+  if (e >= NM || chunks == 0) return;
+  const float* pw = powers + (size_t)h * (LA_C + 1);
+  const float whole = pw[LA_C], rest = pw[n - (chunks - 1) * LA_C];
+  float* mine = state + (size_t)slots[seq] * state_stride + (size_t)h * NM + e;
+  float s = *mine;
+  const size_t step = (size_t)heads * NM;
+  float* u = sums + ((size_t)tile * heads + h) * NM + e;
+  constexpr int AHEAD = 8;
+  for (int k0 = 0; k0 < chunks; k0 += AHEAD) {
+    float v[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) v[k] = k0 + k < chunks ? u[(size_t)(k0 + k) * step] : 0.f;
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+      if (k0 + k < chunks) {
+        u[(size_t)(k0 + k) * step] = s;
+        s = fmaf(k0 + k == chunks - 1 ? rest : whole, s, v[k]);
+      }
+    }
+  }
+  *mine = s;
+}
+
+// VB: blocks of 64 columns of v a head has.  `o` (float32 [T, heads, M]) is written when it is
+// given; else the row's norm per head and the gate are applied and `out` is written.
+template <typename T, int VB>
+__global__ void __launch_bounds__(256)
+la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn<T> in,
+                    const float* __restrict__ states, const float* __restrict__ powers,
+                    const int* __restrict__ q_tiles, const int* __restrict__ cu_tokens, int heads, int N, int M,
+                    int gate_kind, float eps, float factor) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float sm[];
+  float* Qt = sm;                              // [d][token]
+  float* Kt = Qt + LA_BLK * LA_LD;             // [d][token], later P^T [key token][query token]
+  float* Bs = Kt + LA_BLK * LA_LD;             // a block of S [d][column], later of V [token][column]
+  float* pw = Bs + LA_BLK * LA_LD;             // [LA_C + 1]
+  const int tile = blockIdx.x, h = blockIdx.y;
+  int tok0 = 0;
+  const int n_tok = la_tile_tokens(q_tiles, cu_tokens, tile, tok0);
+  for (int i = threadIdx.x; i <= LA_C; i += 256) pw[i] = powers[(size_t)h * (LA_C + 1) + i];
+  pdl_wait();
+  if (n_tok == 0) return;
+  const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+  float p[4][4] = {};
+  float acc[VB][4][4] = {};
+  const float* S = states + ((size_t)tile * heads + h) * N * M;
+  for (int n0 = 0; n0 < N; n0 += LA_BLK) {
+    __syncthreads();
+    for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
+      // neighbouring threads take neighbouring tokens of one piece of d: the transposed stores
+      // fall into different banks
+      const int j = i & (LA_C - 1), d = (i / LA_C) * 4;
+      float q4[4] = {0.f, 0.f, 0.f, 0.f}, k4[4] = {0.f, 0.f, 0.f, 0.f};
+      if (j < n_tok) {
+        const T* r = in.rows + (size_t)(tok0 + j) * in.ld + (size_t)h * N;
+        la_qk4(in, r + in.q_off, tok0 + j, n0 + d, N, q4);
+        la_qk4(in, r + in.k_off, tok0 + j, n0 + d, N, k4);
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        Qt[(d + e) * LA_LD + j] = q4[e];
+        Kt[(d + e) * LA_LD + j] = k4[e] * in.key_scale;
+      }
+    }
+    const int inner = min(LA_BLK, N - n0);
+#pragma unroll
+    for (int vb = 0; vb < VB; ++vb) {
+      if (vb > 0) __syncthreads();
+      for (int i = threadIdx.x; i < LA_BLK * (LA_BLK / 4); i += 256) {
+        const int d = i / (LA_BLK / 4), m = (i - d * (LA_BLK / 4)) * 4;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        const int mm = vb * LA_BLK + m;
+        if (d < inner && mm < M) {
+          const float* src = S + (size_t)(n0 + d) * M + mm;
+          if ((M & 3) == 0) x = *reinterpret_cast<const float4*>(src);
+          else {
+            x.x = src[0];
+            if (mm + 1 < M) x.y = src[1];
+            if (mm + 2 < M) x.z = src[2];
+            if (mm + 3 < M) x.w = src[3];
+          }
+        }
+        *reinterpret_cast<float4*>(Bs + d * LA_LD + m) = x;
+      }
+      __syncthreads();
+      if (vb == 0) la_mma(p, Qt, Kt, ty, tx, inner);
+      la_mma(acc[vb], Qt, Bs, ty, tx, inner);
+    }
+  }
+  // the state's share decays by the tokens since; the chunk's own tokens by their distance
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float f = pw[min(4 * ty + i + 1, LA_C)];
+#pragma unroll
+    for (int vb = 0; vb < VB; ++vb)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[vb][i][j] *= f;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    float w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int dist = 4 * ty + i - (4 * tx + j);
+      w[i] = dist >= 0 ? p[i][j] * pw[dist] : 0.f;
+    }
+    *reinterpret_cast<float4*>(Kt + (4 * tx + j) * LA_LD + 4 * ty) = make_float4(w[0], w[1], w[2], w[3]);
+  }
+#pragma unroll
+  for (int vb = 0; vb < VB; ++vb) {
+    if (vb > 0) __syncthreads();
+    for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
+      const int j = i / (LA_BLK / 4), m = (i - j * (LA_BLK / 4)) * 4;
+      float v4[4] = {0.f, 0.f, 0.f, 0.f};
+      if (j < n_tok) la_v4(in, in.rows + (size_t)(tok0 + j) * in.ld + in.v_off + (size_t)h * M, vb * LA_BLK + m, M, v4);
+      *reinterpret_cast<float4*>(Bs + j * LA_LD + m) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+    }
+    __syncthreads();
+    la_mma(acc[vb], Kt, Bs, ty, tx, n_tok);
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int j = 4 * ty + i;
+    float ss = 0.f;
+    if (o == nullptr) {           // the sixteen threads of a row are neighbouring lanes
+#pragma unroll
+      for (int vb = 0; vb < VB; ++vb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss = fmaf(acc[vb][i][e], acc[vb][i][e], ss);
+#pragma unroll
+      for (int w = 8; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+    }
+    if (j >= n_tok) continue;
+    const int t = tok0 + j;
+    const float rstd = factor * rsqrtf(ss / (float)M + eps);
+#pragma unroll
+    for (int vb = 0; vb < VB; ++vb) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int m = vb * LA_BLK + 4 * tx + e;
+        if (m >= M) continue;
+        if (o != nullptr) o[((size_t)t * heads + h) * M + m] = acc[vb][i][e];
+        else
+          out[(size_t)t * out_ld + (size_t)h * M + m] = from_float<T>(
+              acc[vb][i][e] * rstd * la_gate(to_float(in.rows[(size_t)t * in.ld + in.g_off + (size_t)h * M + m]), gate_kind));
+      }
+    }
+  }
+}
+
+// ---------------------------------------------------------------- norm and gate
+// out = factor * o / rms(o) (* weight) * gate(g): per head (a block a (token, head), weight null)
+// or over the row (a block a token).
+template <typename T>
+__global__ void la_gate_norm_kernel(T* __restrict__ out, int out_ld, const float* __restrict__ o,
+                                    const T* __restrict__ gate, int gate_ld, const float* __restrict__ weight,
+                                    int parts, int width, int gate_kind, float eps, float factor) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const int t = blockIdx.x / parts, part = blockIdx.x - t * parts;
+  const float* x = o + (size_t)blockIdx.x * width;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) ss = fmaf(x[c], x[c], ss);
+  const float rstd = factor * rsqrtf(block_sum(ss, scratch) / (float)width + eps);
+  const T* g = gate + (size_t)t * gate_ld + (size_t)part * width;
+  T* y = out + (size_t)t * out_ld + (size_t)part * width;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float v = x[c] * rstd * la_gate(to_float(g[c]), gate_kind);
+    if (weight) v *= weight[c];
+    y[c] = from_float<T>(v);
+  }
+}
+
+template <typename T>
+LaIn<T> la_in(const void* rows, int ld, int q_off, int k_off, int v_off, int g_off, const float* cos,
+              const float* sin, int rot, int act, float key_scale, int N, int M) {
+  LaIn<T> in;
+  in.rows = (const T*)rows; in.ld = ld;
+  in.q_off = q_off; in.k_off = k_off; in.v_off = v_off; in.g_off = g_off;
+  in.cos = cos; in.sin = sin; in.half = cos ? rot / 2 : 0;
+  in.act = act; in.key_scale = key_scale;
+  in.vec = ((ld | q_off | k_off | v_off | N | M | in.half) & 3) == 0 && ((uintptr_t)rows & 15) == 0 &&
+           ((uintptr_t)cos & 15) == 0 && ((uintptr_t)sin & 15) == 0;
+  return in;
+}
+
+template <typename T, int VB>
+int la_launch_out(float* o, T* out, int out_ld, const LaIn<T>& in, const float* states, const float* powers,
+                  const int* q_tiles, int n_tiles, const int* cu_tokens, int heads, int N, int M, int gate_kind,
+                  float eps, float factor, cudaStream_t stream) {
+  constexpr size_t SMEM = (3 * LA_BLK * LA_LD + LA_C + 1) * sizeof(float);
+  auto kernel = la_chunk_out_kernel<T, VB>;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess)
+      return HB_LAUNCH_FAILED;
+    configured = true;
+  }
+  hb_launch(kernel, dim3(n_tiles, heads), dim3(256), SMEM, stream, o, out, out_ld, in, states, powers, q_tiles,
+            cu_tokens, heads, N, M, gate_kind, eps, factor);
+  return hb_check_launch();
+}
+
+}  // namespace
+
+// rows [T, ld]: q, k (heads x N), v and the gate (heads x M) at the given columns.  powers
+// [heads, 65]: the decay to the power 0..64.  o [T, heads, M] float32.
+HB_EXPORT int hb_la_scan(float* o, const void* rows, int ld, int q_off, int k_off, int v_off, const float* cos,
+                         const float* sin, int rot, int act, float key_scale, float* state, long state_stride,
+                         const float* powers, const int* cu_tokens, const int* slots, int T, int S, int heads, int N,
+                         int M, int act_dt, cudaStream_t stream) {
+  if (T <= 0 || S <= 0) return HB_OK;
+  if (N <= 0 || N > 256 || M <= 0 || heads <= 0) return HB_BAD_ARGUMENT;
+  const dim3 grid((M + LA_COLS - 1) / LA_COLS, heads, S);
+#define HB_LA_SCAN(TA, R)                                                                                   \
+  hb_launch(la_scan_kernel<TA, R>, grid, dim3(LA_COLS * LA_PARTS), 0, stream, o,                              \
+            la_in<TA>(rows, ld, q_off, k_off, v_off, 0, cos, sin, rot, act, key_scale, N, M), state,          \
+            state_stride, powers, cu_tokens, slots, heads, N, M)
+  HB_DISPATCH_DTYPE(act_dt, TA,
+    if (N <= 32) HB_LA_SCAN(TA, 4);
+    else if (N <= 64) HB_LA_SCAN(TA, 8);
+    else if (N <= 128) HB_LA_SCAN(TA, 16);
+    else HB_LA_SCAN(TA, 32));
+#undef HB_LA_SCAN
+  return hb_check_launch();
+}
+
+// Chunked: sums [tiles, heads, N, M] float32 is scratch.  `o` null: norm per head and gate are
+// applied and `out` (rows out_ld apart) is written; else o [T, heads, M] float32.
+HB_EXPORT int hb_la_chunked(float* o, void* out, int out_ld, float* sums, const void* rows, int ld, int q_off,
+                            int k_off, int v_off, int g_off, const float* cos, const float* sin, int rot, int act,
+                            float key_scale, float* state, long state_stride, const float* powers,
+                            const int* q_tiles, int n_tiles, const int* cu_tokens, const int* slots, int S, int heads,
+                            int N, int M, int gate_kind, float eps, float factor, int act_dt, cudaStream_t stream) {
+  if (n_tiles <= 0 || S <= 0) return HB_OK;
+  if (N <= 0 || N > 256 || M <= 0 || M > 256 || heads <= 0) return HB_BAD_ARGUMENT;
+  const int nb = (N + LA_BLK - 1) / LA_BLK, vb = (M + LA_BLK - 1) / LA_BLK;
+  constexpr size_t SMEM_KV = 2 * LA_C * LA_LD * sizeof(float);
+  HB_DISPATCH_DTYPE(act_dt, TA, {
+    const LaIn<TA> in = la_in<TA>(rows, ld, q_off, k_off, v_off, g_off, cos, sin, rot, act, key_scale, N, M);
+    hb_launch(la_chunk_kv_kernel<TA>, dim3(n_tiles, heads, nb * vb), dim3(256), SMEM_KV, stream, sums, in, powers,
+              q_tiles, cu_tokens, heads, N, M);
+    hb_launch(la_states_kernel, dim3((N * M + 255) / 256, heads, S), dim3(256), 0, stream, sums, state, state_stride,
+              powers, cu_tokens, slots, heads, N * M);
+    int st;
+    if (vb == 1) st = la_launch_out<TA, 1>(o, (TA*)out, out_ld, in, sums, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, gate_kind, eps, factor, stream);
+    else if (vb == 2) st = la_launch_out<TA, 2>(o, (TA*)out, out_ld, in, sums, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, gate_kind, eps, factor, stream);
+    else st = la_launch_out<TA, 4>(o, (TA*)out, out_ld, in, sums, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, gate_kind, eps, factor, stream);
+    return st;
+  });
+  return HB_OK;
+}
+
+// parts: norms a row has (heads: per head, 1: over the row), each `width` values wide.
+HB_EXPORT int hb_la_gate_norm(void* out, int out_ld, const float* o, const void* gate, int gate_ld,
+                              const float* weight, int T, int parts, int width, int gate_kind, float eps,
+                              float factor, int act_dt, cudaStream_t stream) {
+  if (T <= 0) return HB_OK;
+  if (parts <= 0 || width <= 0 || (weight != nullptr && parts != 1)) return HB_BAD_ARGUMENT;
+  int threads = 32;
+  while (threads < 256 && threads * 2 < width) threads *= 2;
+  HB_DISPATCH_DTYPE(act_dt, TA,
+    hb_launch(la_gate_norm_kernel<TA>, dim3((unsigned)(T * parts)), dim3(threads), 0, stream, (TA*)out, out_ld, o,
+              (const TA*)gate, gate_ld, weight, parts, width, gate_kind, eps, factor));
+  return hb_check_launch();
+}

@@ -432,10 +432,13 @@ def attention_generic(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
                       block_table: torch.Tensor, seq_of_token: torch.Tensor,
                       positions: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
                       page_size: int, window: Optional[int], scale: float,
-                      options: Optional["AttentionOptions"] = None) -> torch.Tensor:
+                      options: Optional["AttentionOptions"] = None, pooled=None,
+                      out: Optional[torch.Tensor] = None, factor: float = 1.0) -> torch.Tensor:
     """Attention of every token of the batch over its request's pages; q is read from the
     first ``nh * hd`` columns of ``qkv``.  Returns [T, nh * vd] in qkv's dtype (vd = hd
-    unless ``options`` says otherwise)."""
+    unless ``options`` says otherwise).  ``pooled`` = (key pages, value pages, block table, tokens
+    a block): means of whole blocks behind the window.  ``out``: rows to write to (they may be
+    strided); ``factor``: a constant on the output."""
     _check(qkv, "qkv", None, 2)
     _check(k_pages, "k_pages", qkv.dtype, 4)
     _check(v_pages, "v_pages", qkv.dtype, 4)
@@ -456,19 +459,47 @@ def attention_generic(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.T
     if not 0 < vd <= 256 or tuple(v_pages.shape[1:]) != (num_kv_heads, page_size, vd):
         raise KernelError(f"v_pages has shape {tuple(v_pages.shape)}, expected "
                           f"[pages, {num_kv_heads}, {page_size}, {vd}] with at most 256 values a head")
-    out = torch.empty((T, num_heads * vd), dtype=qkv.dtype, device=qkv.device)
+    if out is None:
+        out = torch.empty((T, num_heads * vd), dtype=qkv.dtype, device=qkv.device)
+    else:
+        _check_out_rows(out, T, num_heads * vd, qkv)
+    pk = pv = pt = None
+    pool = 0
+    if pooled is not None:
+        pk, pv, pt, pool = _check_pooled(pooled, qkv, num_kv_heads, page_size, head_dim, vd, window)
     f = _fn("attention_generic", "hb_attention_generic",
             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
-             c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
+             c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+             c_float, c_int, c_void_p])
     _run(f(_p(out), _p(qkv), qkv.shape[1], _p(k_pages), _p(v_pages), _p(block_table),
            block_table.shape[1], _p(seq_of_token), _p(positions), T, num_heads, num_kv_heads,
            head_dim, vd, page_size, int(window or 0), float(scale), _p(opt.slopes), int(opt.sink),
            _p(opt.gate), opt.gate_stride, _p(opt.bias_table),
            0 if opt.bias_table is None else opt.bias_table.shape[0], _p(opt.sink_values),
-           opt.keep_first if window else 0, 1 if opt.gate_wide else 0, _dt(qkv.dtype), _stream()),
+           opt.keep_first if window else 0, 1 if opt.gate_wide else 0, _p(pk), _p(pv), _p(pt),
+           0 if pt is None else pt.shape[1], pool, out.stride(0), float(factor), _dt(qkv.dtype), _stream()),
          "attention_generic")
     return out
+
+
+def _check_out_rows(out: torch.Tensor, tokens: int, columns: int, like: torch.Tensor) -> None:
+    if not out.is_cuda or out.dtype != like.dtype or out.dim() != 2 or out.shape[0] != tokens \
+            or out.shape[1] < columns or out.stride(1) != 1:
+        raise KernelError(f"out must be [{tokens}, >= {columns}] {like.dtype} with unit column stride")
+
+
+def _check_pooled(pooled, like, num_kv_heads, page_size, head_dim, value_dim, window):
+    pk, pv, pt, pool = pooled
+    for name, pages, d in (("pooled keys", pk, head_dim), ("pooled values", pv, value_dim)):
+        _check(pages, name, like.dtype, 4)
+        if tuple(pages.shape[1:]) != (num_kv_heads, page_size, d):
+            raise KernelError(f"{name} have shape {tuple(pages.shape)}, expected "
+                              f"[pages, {num_kv_heads}, {page_size}, {d}]")
+    _check(pt, "pooled block table", torch.int32, 2)
+    if not window or pool < 1:
+        raise KernelError("pooled blocks lie behind a window and hold at least one token")
+    return pk, pv, pt, int(pool)
 
 
 # ------------------------------------------------------------------ feed-forward gate
@@ -1628,6 +1659,29 @@ def rmsnorm_add(residual: torch.Tensor, y: Optional[torch.Tensor], weight: Optio
     return residual if copy is None else copy
 
 
+def scaled_sum_rmsnorm(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
+                       factor: float, copy_dtype: Optional[torch.dtype]) -> Optional[torch.Tensor]:
+    """``residual <- v / sqrt(mean(v^2) + eps) * weight`` with ``v = factor * residual + y`` row by
+    row, in float32 and in place (a block that norms the SUM).  With ``copy_dtype`` other than
+    float32 the new stream is also returned in that dtype; for float32 the stream itself is."""
+    _check(residual, "residual", torch.float32, 2)
+    _check(y, "y", None, 2)
+    _check(weight, "weight", torch.float32, 1)
+    n, H = residual.shape
+    if tuple(y.shape) != (n, H) or weight.numel() != H:
+        raise KernelError(f"y {tuple(y.shape)} / weight {weight.numel()} do not match residual {(n, H)}")
+    copy = None
+    if copy_dtype is not None and copy_dtype != torch.float32:
+        copy = torch.empty((n, H), dtype=copy_dtype, device=residual.device)
+    f = _fn("elementwise", "hb_scaled_sum_rmsnorm",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p])
+    _run(f(_p(residual), _p(y), _p(weight), _p(copy), n, H, float(eps), float(factor), _dt(y.dtype),
+           _dt(copy.dtype) if copy is not None else _F32, _stream()), "scaled_sum_rmsnorm")
+    if copy_dtype is None:
+        return None
+    return residual if copy is None else copy
+
+
 # ------------------------------------------------------------------ attention over a latent cache
 _LONG = ctypes.c_long
 
@@ -1987,6 +2041,202 @@ def gated_group_rmsnorm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, 
     _run(f(_p(out), _p(y), _p(z), z.stride(0), _p(weight), T, inner, parts, float(eps), _dt(z.dtype),
            _stream()), "gated_group_rmsnorm")
     return out
+
+
+# ------------------------------------------------------------------ linear attention, fixed decay
+LINEAR_ATTENTION_ACTIVATIONS = {"none": 0, "silu": 1}
+LINEAR_ATTENTION_NORMS = ("head", "row")
+LINEAR_ATTENTION_GATES = {"silu": 0, "sigmoid": 1}
+#: tokens a chunk of the chunked form
+LINEAR_ATTENTION_CHUNK = 64
+#: steps whose requests bring at most this many tokens each run token by token
+LINEAR_ATTENTION_SCAN_TOKENS = 8
+
+
+def decay_power_table(decay, device) -> torch.Tensor:
+    """float32 [heads, chunk + 1]: every head's decay to the power 0 .. chunk, from float64."""
+    d = torch.tensor([float(x) for x in decay], dtype=torch.float64)
+    n = torch.arange(LINEAR_ATTENTION_CHUNK + 1, dtype=torch.float64)
+    return (d[:, None] ** n[None, :]).float().to(device).contiguous()
+
+
+def linear_attention(ctx, rows: torch.Tensor, offsets, state: torch.Tensor, decay_powers: torch.Tensor,
+                     heads: int, dk: int, dv: int, out: torch.Tensor, *, cos=None, sin=None,
+                     key_scale: float = 1.0, activation: str = "none", norm: str = "head",
+                     norm_weight: Optional[torch.Tensor] = None, gate: str = "silu", eps: float = 1e-6,
+                     factor: float = 1.0) -> None:
+    """S <- a S + k v^T, o = S^T q per head over the step's tokens, request by request, from the
+    state each request's slot holds (``state`` [slots, heads * dk * dv] float32, rows may be
+    strided; left updated), then o / rms(o) (``norm`` "head": per head; "row": over all heads,
+    times ``norm_weight``) times the gate times ``factor`` into ``out`` [T, heads * dv] (rows may
+    be strided).  ``rows`` [T, .] holds q, k (heads x dk), v and the gate (heads x dv) at the
+    column ``offsets``; q, k and v may pass silu (``activation``), q and k a rotation by
+    ``cos`` / ``sin`` [T, rot / 2] of their first ``rot`` values in halves; k is multiplied by
+    ``key_scale``.  ``decay_powers``: ``decay_power_table``.  All of it float32.
+
+    Steps of few tokens a request run token by token, others in chunks of 64 tokens that are
+    taken in parallel."""
+    _check(rows, "rows", None, 2)
+    T = rows.shape[0]
+    _check(decay_powers, "decay_powers", torch.float32, 2)
+    if tuple(decay_powers.shape) != (heads, LINEAR_ATTENTION_CHUNK + 1):
+        raise KernelError(f"decay_powers {tuple(decay_powers.shape)} for {heads} heads")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 \
+            or state.shape[1] != heads * dk * dv or not state.is_cuda:
+        raise KernelError(f"state {tuple(state.shape)} does not fit {heads} heads of {dk} x {dv}")
+    if dk > 256 or dv > 256:
+        raise KernelError(f"heads of {dk} x {dv} are not supported (at most 256)")
+    q_off, k_off, v_off, g_off = (int(o) for o in offsets)
+    if min(q_off, k_off, v_off, g_off) < 0 or max(q_off + heads * dk, k_off + heads * dk, v_off + heads * dv,
+                                                   g_off + heads * dv) > rows.shape[1]:
+        raise KernelError(f"rows of {rows.shape[1]} columns do not hold the columns {tuple(offsets)}")
+    rot = 0
+    if cos is not None:
+        _check(cos, "cos", torch.float32, 2)
+        _check(sin, "sin", torch.float32, 2)
+        rot = 2 * cos.shape[1]
+        if cos.shape != sin.shape or cos.shape[0] != T or rot > dk:
+            raise KernelError(f"cos/sin tables {tuple(cos.shape)} do not fit {T} tokens of heads of {dk}")
+    if (norm == "row") != (norm_weight is not None) or norm not in LINEAR_ATTENTION_NORMS:
+        raise KernelError(f"norm {norm!r} and its weight do not go together")
+    if norm_weight is not None:
+        _check(norm_weight, "norm_weight", torch.float32, 1)
+        if norm_weight.numel() != heads * dv:
+            raise KernelError(f"norm weight has {norm_weight.numel()} entries for {heads * dv} columns")
+    _check_out_rows(out, T, heads * dv, rows)
+    act, gk = LINEAR_ATTENTION_ACTIVATIONS[activation], LINEAR_ATTENTION_GATES[gate]
+    most = getattr(ctx, "max_tokens_per_seq", T)
+    o = None
+    if most > LINEAR_ATTENTION_SCAN_TOKENS:
+        tiles = _step_tiles(ctx, LINEAR_ATTENTION_CHUNK, False, rows.device)
+        n_tiles = tiles.shape[0]
+        sums = torch.empty((n_tiles * heads * dk * dv,), dtype=torch.float32, device=rows.device)
+        if norm == "row":
+            o = torch.empty((T, heads * dv), dtype=torch.float32, device=rows.device)
+        f = _fn("linear_attention", "hb_la_chunked",
+                [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                 c_int, c_int, c_float, c_void_p, _LONG, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                 c_int, c_int, c_int, c_float, c_float, c_int, c_void_p])
+        _run(f(_p(o), _p(out), out.stride(0), _p(sums), _p(rows), rows.shape[1], q_off, k_off, v_off, g_off,
+               _p(cos), _p(sin), rot, act, float(key_scale), _p(state), state.stride(0), _p(decay_powers), _p(tiles),
+               n_tiles, _p(ctx.cu_tokens), _p(ctx.slots), ctx.num_seqs, heads, dk, dv, gk, float(eps), float(factor),
+               _dt(rows.dtype), _stream()), "linear_attention_chunked")
+        if o is None:
+            return
+    else:
+        o = torch.empty((T, heads * dv), dtype=torch.float32, device=rows.device)
+        f = _fn("linear_attention", "hb_la_scan",
+                [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p,
+                 _LONG, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+        _run(f(_p(o), _p(rows), rows.shape[1], q_off, k_off, v_off, _p(cos), _p(sin), rot, act, float(key_scale),
+               _p(state), state.stride(0), _p(decay_powers), _p(ctx.cu_tokens), _p(ctx.slots), T, ctx.num_seqs,
+               heads, dk, dv, _dt(rows.dtype), _stream()), "linear_attention_scan")
+    f = _fn("linear_attention", "hb_la_gate_norm",
+            [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+             c_int, c_void_p])
+    parts = heads if norm == "head" else 1
+    _run(f(_p(out), out.stride(0), _p(o), _p(rows) + g_off * rows.element_size(), rows.shape[1], _p(norm_weight), T,
+           parts, heads * dv // parts, gk, float(eps), float(factor), _dt(rows.dtype), _stream()),
+         "linear_attention_gate_norm")
+
+
+# ------------------------------------------------------------------ window attention with pooled blocks
+def pooled_attention_libraries(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int,
+                               value_dim: int):
+    """Libraries window attention with pooled blocks runs on at these sizes."""
+    return ("pooled_window", "attention_generic")
+
+
+def _check_pages(cache, like: torch.Tensor, num_kv_heads: int, head_dim: int, value_dim: int) -> None:
+    for name, pages, d in (("k_pages", cache.k_pages, head_dim), ("v_pages", cache.v_pages, value_dim)):
+        _check(pages, name, like.dtype, 4)
+        if tuple(pages.shape[1:]) != (num_kv_heads, cache.page_size, d):
+            raise KernelError(f"{name} has shape {tuple(pages.shape)}, expected "
+                              f"[pages, {num_kv_heads}, {cache.page_size}, {d}]")
+
+
+def conv_norm_rotate_write(ctx, rows: torch.Tensor, col0: int, conv: Optional[torch.Tensor],
+                           state: Optional[torch.Tensor], q_weight: torch.Tensor, k_weight: torch.Tensor,
+                           eps: float, cos: torch.Tensor, sin: torch.Tensor, cache, num_heads: int,
+                           num_kv_heads: int, head_dim: int, value_dim: int) -> torch.Tensor:
+    """From the columns q | k | v of ``rows`` [T, .] at ``col0``: a short causal convolution per
+    channel (``conv`` float32 [channels, taps], last column the current token's; None: none; the
+    inputs before the step's first token come from ``state`` [slots, channels * (taps - 1)]
+    float32, which is left holding the last ones), an RMS norm per q and k head with a weight,
+    the rotation of q's and k's first values by ``cos`` / ``sin`` [T, rot / 2] in halves.  k and v
+    go to the cache's pages, q is returned [T, heads * head_dim].  Float32 in between."""
+    _check(rows, "rows", None, 2)
+    T = rows.shape[0]
+    channels = num_heads * head_dim + num_kv_heads * (head_dim + value_dim)
+    if col0 < 0 or rows.shape[1] < col0 + channels:
+        raise KernelError(f"rows of {rows.shape[1]} columns do not hold {channels} from column {col0}")
+    taps = 1
+    if conv is not None:
+        _check(conv, "conv", torch.float32, 2)
+        taps = conv.shape[1]
+        if conv.shape[0] != channels or taps < 1:
+            raise KernelError(f"conv weight {tuple(conv.shape)} does not fit {channels} channels")
+        if taps > 1 and (state is None or state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1
+                         or state.shape[1] != channels * (taps - 1)):
+            raise KernelError(f"the convolution's state does not fit {channels} channels x {taps - 1}")
+    for name, w in (("q_weight", q_weight), ("k_weight", k_weight)):
+        _check(w, name, torch.float32, 1)
+        if w.numel() != head_dim:
+            raise KernelError(f"{name} has {w.numel()} entries for heads of {head_dim}")
+    _check(cos, "cos", torch.float32, 2)
+    _check(sin, "sin", torch.float32, 2)
+    rot = 2 * cos.shape[1]
+    if cos.shape != sin.shape or cos.shape[0] != T or rot > head_dim:
+        raise KernelError(f"cos/sin tables {tuple(cos.shape)} do not fit {T} tokens of heads of {head_dim}")
+    _check_pages(cache, rows, num_kv_heads, head_dim, value_dim)
+    table = ctx.block_tables[cache.group]
+    _check(table, "block_table", torch.int32, 2)
+    q = torch.empty((T, num_heads * head_dim), dtype=rows.dtype, device=rows.device)
+    moves = taps > 1
+    f = _fn("pooled_window", "hb_conv_norm_rotate_write",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, _LONG, c_int, c_void_p, c_void_p,
+             c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _run(f(_p(q), _p(cache.k_pages) if cache.write else 0, _p(cache.v_pages) if cache.write else 0,
+           _p(rows) + col0 * rows.element_size(), rows.shape[1], _p(conv), _p(state) if moves else 0,
+           state.stride(0) if moves else 0, taps, _p(q_weight), _p(k_weight), float(eps), _p(cos), _p(sin), rot,
+           _p(ctx.positions), _p(ctx.seq_of_token), _p(ctx.cu_tokens), _p(ctx.slots), _p(table), table.shape[1], T,
+           ctx.num_seqs, num_heads, num_kv_heads, head_dim, value_dim, cache.page_size,
+           1 if ctx.decode_only else 0, _dt(rows.dtype), _stream()), "conv_norm_rotate_write")
+    return q
+
+
+def pool_blocks(ctx, cache, pool: int) -> None:
+    """For every token of the step that ends a whole block of ``pool`` tokens of its request: the
+    means of the block's keys and values, as the pages hold them, into the pooled pages."""
+    pooled = cache.pooled
+    G, hd = cache.k_pages.shape[1], cache.k_pages.shape[3]
+    vd = cache.v_pages.shape[3]
+    _check_pages(cache, cache.k_pages, G, hd, vd)
+    _check_pages(pooled, cache.k_pages, G, hd, vd)
+    table, ptable = ctx.block_tables[cache.group], ctx.block_tables[pooled.group]
+    f = _fn("pooled_window", "hb_pool_blocks",
+            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _run(f(_p(pooled.k_pages), _p(pooled.v_pages), _p(ptable), ptable.shape[1], _p(cache.k_pages), _p(cache.v_pages),
+           _p(table), table.shape[1], _p(ctx.positions), _p(ctx.seq_of_token), ctx.num_tokens, G, hd, vd,
+           cache.page_size, int(pool), _dt(cache.k_pages.dtype), _stream()), "pool_blocks")
+
+
+def pooled_attention(ctx, q: torch.Tensor, cache, num_heads: int, num_kv_heads: int, head_dim: int,
+                     value_dim: int, window: int, pool: int, scale: float, out: torch.Tensor,
+                     factor: float = 1.0) -> None:
+    """Attention of the step's tokens over the last ``window`` tokens of their requests and, with
+    ``pool``, one key and value for every whole block of ``pool`` tokens that lies before the
+    window, under one softmax; ``factor`` times the result into ``out`` [T, heads * value_dim]
+    (rows may be strided)."""
+    pooled = None
+    if pool:
+        pooled = (cache.pooled.k_pages, cache.pooled.v_pages, ctx.block_tables[cache.pooled.group], pool)
+    options = None if value_dim == head_dim else AttentionOptions(value_dim=value_dim)
+    attention_generic(q, cache.k_pages, cache.v_pages, ctx.block_tables[cache.group], ctx.seq_of_token,
+                      ctx.positions, num_heads, num_kv_heads, head_dim, cache.page_size, window, scale, options,
+                      pooled=pooled, out=out, factor=factor)
 
 
 # ------------------------------------------------------------------ routed experts

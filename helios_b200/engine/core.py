@@ -147,6 +147,10 @@ class EngineCore:
     #: take these token counts too.
     SMALL_MODEL_PARAMETERS = 2_000_000_000
     SMALL_MODEL_TOKEN_BUCKETS = (640, 768, 896, 1024, 1280, 1536, 1792, 2048)
+    #: captured steps hold block tables for contexts of at most this many tokens; where neither
+    #: a pool nor the model bounds a request's length (windows, states), a step with a longer
+    #: context runs kernel by kernel
+    GRAPH_MOST_CONTEXT = 1 << 18
     MAX_FULL_GRAPHS = 8
     FULL_GRAPH_EAGER_RUNS = 6
 
@@ -179,8 +183,9 @@ class EngineCore:
         if pool_tokens is None:
             pool_tokens = max_model_len or \
                 (max(p.num_pages for p in self.cache.pools) * page_size if self.cache.pools else 0)
-        self.graph_max_context = min(max_model_len or pool_tokens, pool_tokens) or 1
-        self.graph_table_widths = [-(-self.graph_max_context // page_size)] * len(self.cache.groups)
+        self.graph_max_context = min(max_model_len or pool_tokens, pool_tokens, self.GRAPH_MOST_CONTEXT) or 1
+        self.graph_table_widths = [max(1, self.cache.pages_in(g, self.graph_max_context))
+                                   for g in range(len(self.cache.groups))]
         self._graphs = {}
         self._bucket_seen = {}
         parameters = sum(_numel(spec.shape) for _prefix, part in model.plan.named_parts()
@@ -207,7 +212,7 @@ class EngineCore:
     def context_limit(groups, page_size: int) -> Optional[int]:
         """Tokens the smallest pool among the groups that keep every key holds; None when
         every group has a window (then the pools bound no request's length)."""
-        full = [g.num_pages for g in groups if g.window is None]
+        full = [g.num_pages * g.tokens_per_row for g in groups if g.window is None]
         return min(full) * page_size if full else None
 
     @staticmethod

@@ -116,10 +116,10 @@ class LLMEngine:
         self.model = model or DecoderModel.from_folder(config.model_dir, dtype=config.dtype,
                                                        device=config.device)
         mcfg = self.model.config
-        from ..cache.manager import cache_groups_of
+        from ..cache.manager import cache_groups_of, pages_for_tokens_each
         specs, _ = cache_groups_of(self.model.plan)
         if config.num_blocks:
-            num_pages = [config.num_blocks] * len(specs)
+            num_pages = pages_for_tokens_each(specs, config.num_blocks, config.max_num_seqs)
         else:
             num_pages = EngineCore.pages_for_bytes(
                 self.model, config.block_size, config.kv_cache_bytes, config.max_num_seqs,
@@ -127,7 +127,7 @@ class LLMEngine:
         # a context longer than the pool is a promise that cannot be kept
         # (python/helios/engine.py:157-160); only the groups that keep every key bound it:
         # where every layer has a window, the window buys any length
-        keeps_all = [n for n, s in zip(num_pages, specs) if s.window is None]
+        keeps_all = [n * s.tokens_per_row for n, s in zip(num_pages, specs) if s.window is None]
         pool_tokens = min(keeps_all) * config.block_size if keeps_all else None
         max_len = config.max_model_len or getattr(mcfg, "max_position_embeddings", None) \
             or pool_tokens or max(num_pages, default=8) * config.block_size

@@ -9,8 +9,11 @@ from .moe import RoutedExperts
 from .latent_attention import LatentAttention
 from .delta_rule import GatedDeltaMixer
 from .ssm import SelectiveStateMixer
+from .side_by_side import BranchMixer, SideBySideMixer
+from .linear_attention import FixedDecayMixer
+from .pooled_window import PooledWindowAttention
 from .embedding import LearnedPositions, NormedHead, OutputHead, TokenEmbedding
-from .block import ParallelBlock, PostNormBlock, PreNormBlock
+from .block import NormedSumBlock, ParallelBlock, PostNormBlock, PreNormBlock
 from .stream import StreamInputMix
 from .plan import ModelPlan, Run
 
@@ -21,4 +24,5 @@ __all__ = ["Block", "DeferredNorm", "FeedForward", "InputStage", "OutputStage", 
            "GatedMLP", "RoutedExperts", "LatentAttention", "GatedDeltaMixer", "PostNormBlock",
            "yarn_frequencies", "yarn_attention_factor", "PendingSum", "StreamStage", "settle", "LayerNorm",
            "SinkGQAAttention", "distance_slopes", "LearnedPositions", "ParallelBlock", "StreamInputMix",
-           "SelectiveStateMixer"]
+           "SelectiveStateMixer", "BranchMixer", "SideBySideMixer", "FixedDecayMixer",
+           "PooledWindowAttention", "NormedSumBlock"]

@@ -46,6 +46,16 @@ class PagedCacheSpec:
     planes: int = 2                   # 2: keys and values; 1: one row a token (a latent cache)
     value_dim: Optional[int] = None   # values per head where they differ from head_dim (planes 2)
     keep_first: int = 0               # with a window: the request's first tokens stay as well
+    # beside the tokens, a key and a value for every whole block of ``pool`` tokens (the mixer
+    # writes them), kept for good in pages of their own; needs a window of at least a block,
+    # so that a block's tokens stay until it is whole
+    pool: int = 0
+    tokens_per_row: int = 1           # tokens a stored row stands for
+
+    def pooled(self) -> "PagedCacheSpec":
+        """The pages that hold the blocks' keys and values."""
+        return PagedCacheSpec(self.num_kv_heads, self.head_dim, planes=self.planes, value_dim=self.value_dim,
+                              tokens_per_row=self.pool)
 
 
 @dataclass(frozen=True)
@@ -63,6 +73,7 @@ class LayerCache:
     group: int                    # index into StepContext.block_tables
     page_size: int
     write: bool = True            # False: this run reads what another run wrote
+    pooled: Optional["LayerCache"] = None   # the blocks' keys and values (``PagedCacheSpec.pool``)
 
 
 class Part:
@@ -110,6 +121,15 @@ class Norm(Part):
         float32).  ``y`` None: nothing is added.  The default does it in two steps."""
         if y is not None:
             residual.add_(self.forward(y).float())
+        return residual if out_dtype == torch.float32 else residual.to(out_dtype)
+
+    def normed_sum(self, residual: torch.Tensor, y: torch.Tensor, factor: float,
+                   out_dtype: torch.dtype) -> torch.Tensor:
+        """``residual <- norm(factor * residual + y)`` in float32 and in place, for a block that
+        norms the SUM; returns the new residual in ``out_dtype`` (the residual itself for
+        float32).  The default does it in two steps."""
+        residual.mul_(factor).add_(y.float())
+        residual.copy_(self.forward(residual))
         return residual if out_dtype == torch.float32 else residual.to(out_dtype)
 
 

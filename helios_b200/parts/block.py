@@ -103,6 +103,10 @@ class PostNormBlock(Block):
     def graph_safe(self) -> bool:
         return all(p.graph_safe for _, p in self.named_parts())
 
+    def _join(self, norm: Norm, residual: torch.Tensor, y: torch.Tensor, dtype) -> torch.Tensor:
+        """A sublayer's output joins the stream in place; returns the stream in ``dtype``."""
+        return norm.add_normed(residual, y, dtype)
+
     def forward(self, ctx, residual: torch.Tensor, delta, cache: Optional[LayerCache],
                 state: Optional[torch.Tensor]):
         if isinstance(delta, DeferredNorm):
@@ -116,14 +120,34 @@ class PostNormBlock(Block):
         else:
             h = self.mixer_norm.add_normed(residual, None, ctx.act_dtype) \
                 if ctx.act_dtype != torch.float32 else residual
-        h = self.mixer_norm.add_normed(residual, self._mixer.forward(ctx, h, cache, state), ctx.act_dtype)
+        h = self._join(self.mixer_norm, residual, self._mixer.forward(ctx, h, cache, state), ctx.act_dtype)
         if self.ffn is not None:
-            h = self.ffn_norm.add_normed(residual, self.ffn.forward(ctx, h), ctx.act_dtype)
+            h = self._join(self.ffn_norm, residual, self.ffn.forward(ctx, h), ctx.act_dtype)
         ctx.step_tables[self._COPY] = (ctx.run_index, h)
         return residual, None
 
 
 register_part("block", "post_norm", PostNormBlock)
+
+
+class NormedSumBlock(PostNormBlock):
+    """norm(factor * x + mixer(x)), then norm(factor * x + feed_forward(x)): the norm takes the SUM
+    of the weighted stream and the sublayer's output, and its result IS the new stream.  The
+    sublayers read the stream itself (in the activation dtype).  The feed-forward, with its
+    norm, may be absent.  Sum and norm are float32 and one kernel, which also leaves the new
+    stream in the activation dtype."""
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm, ffn: Optional[FeedForward] = None,
+                 ffn_norm: Optional[Norm] = None, factor: float = 1.0,
+                 names: Tuple[str, str, str, str] = ("mix.", "norm1", "mlp.", "norm2")) -> None:
+        super().__init__(mixer, mixer_norm, ffn, ffn_norm, names)
+        self.factor = float(factor)
+
+    def _join(self, norm: Norm, residual: torch.Tensor, y: torch.Tensor, dtype) -> torch.Tensor:
+        return norm.normed_sum(residual, y, self.factor, dtype)
+
+
+register_part("block", "normed_sum", NormedSumBlock)
 
 
 class ChannelScale(Part):

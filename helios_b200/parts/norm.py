@@ -61,6 +61,9 @@ class RMSNorm(Norm):
         """``y`` None: only the residual in ``out_dtype``."""
         return ops.rmsnorm_add(residual, y, self.weight, self.eps, out_dtype)
 
+    def normed_sum(self, residual, y, factor, out_dtype):
+        return ops.scaled_sum_rmsnorm(residual, y, self.weight, self.eps, factor, out_dtype)
+
 
 register_part("norm", "rmsnorm", RMSNorm)
 
