@@ -133,7 +133,7 @@ def window_mixer(h, t, p, mx, eps):
     q = rotate_half(rms_norm(project("q", H, d), t[p + "q.norm"], eps), pos, mx["rot"])
     k = rotate_half(rms_norm(project("k", G, d), t[p + "k.norm"], eps), pos, mx["rot"])
     v = project("v", G, dv)
-    P = mx["mask"]["pool"]
+    P = mx["mask"].get("pool") or T + 1          # without blocks: one that is never whole
     nb = T // P
     kp = k[:nb * P].view(nb, P, G, d).mean(1)
     vp = v[:nb * P].view(nb, P, G, dv).mean(1)

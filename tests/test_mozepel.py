@@ -1,0 +1,760 @@
+"""The Mozepel design against a plain float64 implementation (``plain_mozepel``): every
+mechanism alone on made inputs, then whole models of several shapes through the step function
+(whole prompts, decoding, portions, mixed batches, replay, generation)."""
+from __future__ import annotations
+
+import json
+import math
+from types import SimpleNamespace
+
+import pytest
+import torch
+
+import plain_mozepel as pm
+import trace_util as tu
+from conftest import random_tokens, read_folder
+
+DTYPES = ["float32", "bfloat16"]
+
+
+# ---------------------------------------------------------------------- configurations
+def _ret(heads, dim, vdim, decay, rot, base, scaling=None):
+    r = {"dims": rot, "base": base}
+    if scaling:
+        r["scaling"] = scaling
+    return {"type": "retention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay, "rot": r}}
+
+
+def _par(heads, kv, dim, vdim, scale, size, pool, rot, base, taps, ls, rs, rheads, rdim, rvdim, decay, scaling=None):
+    r = {"dims": rot, "base": base}
+    if scaling:
+        r["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    mask = {"size": size}
+    if pool:
+        mask["pool"] = pool
+    left = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": scale, "mask": mask, "rot": r}
+    if taps:
+        left["conv"] = taps
+    return {"type": "parallel", "mixer": {"left": left, "left_scale": ls, "right_scale": rs,
+                                          "right": {"heads": rheads, "dim": rdim, "vdim": rvdim, "decay": decay}}}
+
+
+def _model(vocab, width, eps, alpha, layers):
+    out = []
+    for layer in layers:
+        if isinstance(layer, int):
+            out.append({**out[layer], "weights_of": layer})
+        else:
+            out.append({**layer[0], "mlp": {"kind": "dense", "ff": layer[1]} if layer[1] else None})
+    return {"architecture": "Mozepel", "vocab": vocab, "width": width, "norm": {"eps": eps}, "postln_alpha": alpha,
+            "layers": out}
+
+
+# heads of 32, a window that is no multiple of a page or a block, layers run twice
+MZ_A = _model(211, 96, 1e-5, 1.7, [
+    (_ret(3, 32, 48, [0.9, 0.995, 1.0], 16, 10000.0), 56),
+    (_par(4, 2, 32, 32, 0.3, 27, 6, 16, 5000.0, 4, 0.8, 0.7, 2, 24, 20, [0.5, 0.99], (3.0, 1.0, 4.0, 64)), 56),
+    0, 1,
+])
+# values larger than keys, one head a group, blocks longer than the window, blocks that begin
+# anywhere in a page, no feed-forward here and there, one tap, odd sizes
+MZ_B = _model(150, 72, 3e-6, 1.0, [
+    (_par(3, 3, 20, 36, 0.4, 9, 14, 20, 700.0, 1, 1.3, 0.4, 5, 6, 10, [0.7, 0.8, 0.9, 0.95, 0.999]), None),
+    (_ret(5, 14, 22, [0.99, 0.5, 0.97, 0.999, 0.0], 14, 300.0), 40),
+    1,
+    (_ret(2, 40, 12, [0.8, 0.998], 8, 1e6), None),
+])
+# heads of 64 and 128 (the tensor-core kernels' sizes), blocks of a page, a rotation of part
+# of a head with stretched waves
+MZ_C = _model(180, 128, 1e-5, 2.2, [
+    (_par(8, 2, 64, 128, 0.2, 48, 16, 32, 200000.0, 3, 0.6, 0.9, 4, 64, 32, [0.6, 0.9, 0.97, 0.999],
+          (8.0, 1.0, 2.0, 32)), 96),
+    (_ret(2, 128, 64, [0.97, 0.999], 128, 50000.0), 64),
+    (_par(4, 1, 128, 128, 0.1, 33, 8, 128, 10000.0, 2, 0.9, 0.5, 2, 130, 70, [0.95, 0.99]), None),
+    2, 0,
+])
+# values smaller than keys, a window of one token, blocks of one token, no convolution; and a
+# window that sees nothing behind itself
+MZ_D = _model(131, 50, 2e-6, 3.0, [
+    (_par(5, 1, 30, 10, 0.5, 1, 1, 30, 77.0, 0, 0.5, 1.5, 1, 7, 9, [0.9]), 12),
+    (_par(2, 2, 16, 16, 0.3, 17, 0, 4, 77.0, 5, 1.0, 1.0, 3, 8, 8, [0.9, 0.99, 0.3]), 30),
+    (_ret(1, 10, 6, [0.96], 2, 5.0), 18),
+])
+MZ_CONFIGS = {"mz_a": MZ_A, "mz_b": MZ_B, "mz_c": MZ_C, "mz_d": MZ_D}
+MZ_SEEDS = {"mz_a": 3, "mz_b": 4, "mz_c": 5, "mz_d": 6}
+MZ_ALONE = {
+    "retention_only": _model(97, 64, 1e-5, 1.2, [(_ret(4, 16, 24, [0.9, 0.97, 0.99, 0.5], 8, 1000.0), None)]),
+    "side_by_side_only": _model(97, 64, 1e-5, 1.2, [
+        (_par(4, 2, 16, 24, 0.3, 21, 5, 8, 1000.0, 3, 0.7, 0.6, 2, 12, 16, [0.9, 0.98]), None)]),
+    "dense_ff": _model(97, 64, 1e-5, 1.2, [(_ret(2, 8, 8, [0.9, 0.8], 8, 100.0), 48)]),
+}
+
+
+def _lively(weights):
+    """Matrices of a size at which every sublayer moves the stream (with a few hundredths a
+    factor on the stream would drown it), rounded to what bfloat16 holds.  The key projection of
+    the layers with a norm per head leans on the query projection: at a request's first tokens o
+    is (q . k) v and little else, the norm keeps of q . k the sign only, and where that number
+    is near 0 by chance rounding decides it."""
+    out = {}
+    for k, v in weights.items():
+        if v.dim() >= 2 and not k.endswith(".conv"):
+            if k.endswith(".mix.k"):
+                v = 0.9 * weights[k[:-1] + "q"] + 0.43 * v
+            f = {"embed": 50.0, "head": 1.0}.get(k, 0.9 / math.sqrt(v.shape[1]) / 0.02)
+            out[k] = (v * f).to(torch.bfloat16).float()
+        else:
+            out[k] = v
+    return out
+
+
+@pytest.fixture(scope="module")
+def mz_folders(tmp_path_factory):
+    from safetensors.torch import save_file
+    from helios_b200.weights import write_model_folder
+
+    out = {}
+    base = tmp_path_factory.mktemp("mozepel")
+    for name, cfg in {**MZ_CONFIGS, **MZ_ALONE}.items():
+        folder = write_model_folder(base / name, cfg, MZ_SEEDS.get(name, 9))
+        _cfg, weights = read_folder(folder)
+        save_file(_lively(weights), str(folder / "model.safetensors"))
+        out[name] = folder
+    return out
+
+
+def _f64(weights):
+    return {k: v.double() for k, v in weights.items()}
+
+
+def _plain(cfg, weights, requests):
+    w = _f64(weights)
+    return {rid: pm.model(cfg, w, toks)[0] for rid, toks in requests.items()}
+
+
+def _core(folder, dtype, max_tokens, page_size=16, max_slots=4, graphs=True):
+    from helios_b200.engine.core import EngineCore
+    from helios_b200.engine.model import DecoderModel
+
+    model = DecoderModel.from_folder(folder, dtype=dtype)
+    return EngineCore(model, page_size=page_size, num_pages=-(-max_tokens // page_size),
+                      max_slots=max_slots, poison_cache=float("nan"), use_cuda_graphs=graphs)
+
+
+def _requests(cfg, lengths, seed):
+    return {f"q{i}": random_tokens(cfg["vocab"], n, seed + i) for i, n in enumerate(lengths)}
+
+
+def _dt(dtype):
+    return torch.float32 if dtype == "float32" else torch.bfloat16
+
+
+# ====================================================================== without a GPU
+def test_configuration_is_read_layer_by_layer_and_faults_name_the_key():
+    from helios_b200.config import ConfigError
+    from helios_b200.config.mozepel_config import MozepelConfig, RetentionConfig, SideBySideConfig
+
+    cfg = MozepelConfig.from_json(MZ_A)
+    assert [type(l.mixer) for l in cfg.layers] == [RetentionConfig, SideBySideConfig] * 2
+    assert [l.weights_of for l in cfg.layers] == [0, 1, 0, 1] and cfg.residual_factor == 1.7
+    left = cfg.layers[3].mixer.left
+    assert (left.conv, left.window, left.pool, left.rot.scaling.high_freq_factor) == (4, 27, 6, 4.0)
+    assert cfg.layers[1].mixer.right.decay == (0.5, 0.99)
+    d = MozepelConfig.from_json(MZ_D)
+    assert d.layers[0].mixer.left.conv == 0 and d.layers[1].mixer.left.pool == 0
+    assert MozepelConfig.from_json(MZ_B).layers[0].mlp is None
+    chain = json.loads(json.dumps(MZ_A))
+    chain["layers"][3] = {"weights_of": 2}               # an entry that points on to one that points on
+    assert [l.weights_of for l in MozepelConfig.from_json(chain).layers] == [0, 1, 0, 0]
+    for path, value, word in [(("layers", 0, "mixer", "decay"), [0.5], "decay"),
+                              (("layers", 0, "mixer", "decay"), [0.5, 1.5, 0.9], "decay"),
+                              (("layers", 1, "mixer", "left", "rot", "dims"), 7, "dims"),
+                              (("layers", 1, "mixer", "left", "kv_heads"), 3, "kv_heads"),
+                              (("layers", 1, "mixer", "left", "mask"), {}, "size"),
+                              (("layers", 1, "mixer", "right_scale"), None, "right_scale"),
+                              (("layers", 1, "mixer", "left", "rot", "scaling", "high"), 0.5, "high"),
+                              (("layers", 0, "mlp", "kind"), "moe", "kind"),
+                              (("layers", 0, "type"), "conv", "type"),
+                              (("layers", 2, "weights_of"), 9, "weights_of"),
+                              (("layers", 2, "weights_of"), 2, "weights_of"),
+                              (("layers", 2, "mlp"), None, "mlp"),
+                              (("postln_alpha",), None, "postln_alpha"),
+                              (("norm",), {}, "eps")]:
+        bad = json.loads(json.dumps(MZ_A))
+        at = bad
+        for key in path[:-1]:
+            at = at[key]
+        if value is None and path[-1] != "mlp":
+            del at[path[-1]]
+        else:
+            at[path[-1]] = value
+        with pytest.raises(ConfigError, match=word):
+            MozepelConfig.from_json(bad)
+
+
+def test_plan_names_every_tensor_once_and_sizes_caches_and_state():
+    from helios_b200.cache.manager import cache_groups_of, pages_for_tokens_each, pool_sizes_for_bytes
+    from helios_b200.config.mozepel_config import MozepelConfig
+    from helios_b200.models import build_mozepel_plan
+    from helios_b200.weights.loader import expected_tensors
+
+    plan = build_mozepel_plan(MozepelConfig.from_json(MZ_A))
+    names = expected_tensors(plan)
+    left = {f"l1.mix.left.{n}" for n in ("q", "k", "v", "o", "q.norm", "k.norm", "q.conv", "k.conv", "v.conv")}
+    right = {f"l1.mix.right.{n}" for n in ("q", "k", "v", "g", "o", "norm")}
+    mlps = {f"l{i}.{n}" for i in (0, 1) for n in ("norm1", "norm2", "mlp.gate", "mlp.up", "mlp.down")}
+    assert set(names) == {"embed", "head", "final.norm"} | left | right | mlps | {
+        f"l0.mix.{n}" for n in "qkvgo"}
+    assert names["l0.mix.g"][2].shape == (3 * 48, 96) and names["l1.mix.left.v.conv"][2].shape == (2 * 32, 4)
+    assert len(plan.layers) == 2 and [r.layer for r in plan.schedule] == [0, 1, 0, 1]
+    assert plan.layers[0].mixer.position is not plan.layers[1].mixer.branches[0].position
+    specs, where = cache_groups_of(plan)
+    assert set(where) == {1, (1, "pooled"), 3, (3, "pooled")}       # two runs of one layer: two caches
+    assert {s.tokens_per_row for s in specs} == {1, 6} and specs[0].window == 27 and specs[1].window is None
+    assert pages_for_tokens_each(specs, 24, 4) == [24, 4 + 4]
+    sizes = pool_sizes_for_bytes(plan, 16, 2, 1 << 22, 4, 64)
+    assert sizes[0] == 4 * (-(-(27 + 64) // 16) + 2) and sizes[1] > 8
+    pair = plan.layers[1].mixer
+    assert pair.state_spec().shape == ((4 * 32 + 2 * 64) * 3 + 2 * 24 * 20,)
+    # blocks longer than the window: their tokens stay until they are whole
+    wide = cache_groups_of(build_mozepel_plan(MozepelConfig.from_json(MZ_B)))[0]
+    assert [s.window for s in wide] == [14, None] and wide[0].value_dim == 36
+    plain = cache_groups_of(build_mozepel_plan(MozepelConfig.from_json(MZ_D)))[0]
+    assert sum(s.tokens_per_row > 1 for s in plain) == 0 and [s.window for s in plain] == [1, None, 17]
+
+
+def test_toy_model_of_the_design_from_the_command_line(tmp_path, capsys):
+    from helios_b200 import cli
+
+    assert cli.main(["make-toy-model", "--arch", "mozepel", "--out", str(tmp_path / "toy"), "--layers", "5",
+                     "--hidden", "64", "--heads", "4", "--kv-heads", "2"]) == 0
+    assert cli.main(["info", "--model", str(tmp_path / "toy")]) == 0
+    text = capsys.readouterr().out
+    assert "Mozepel" in text and "SideBySideMixer" in text and "FixedDecayMixer" in text
+    assert "4 layers, 5 runs a step" in text and "whole block of 8 tokens" in text
+
+
+def test_rows_for_whole_blocks_take_pages_as_blocks_fill():
+    from helios_b200.cache.pages import CacheLayout, GroupLayout, OutOfPages
+
+    lay = CacheLayout([GroupLayout(9, 20), GroupLayout(None, 3, tokens_per_row=5)], 4, 2)
+    lay.admit("a")
+    for n in [3, 1, 1, 14, 1, 2, 30]:
+        lay.extend("a", n)
+        lay.commit("a", n)
+        lay.check_invariants()
+        assert len(lay.table("a", 1)) == -(-(lay.length("a") // 5) // 4)
+    assert lay.length("a") == 52 and all(p >= 0 for p in lay.table("a", 1))
+    assert all(p < 0 for p in lay.table("a", 0)[:(52 - 9 + 1) // 4])
+    assert lay.peak_pages(1, 59, 8) == 3 and lay.tokens_that_fit("a") == (12 + 1) * 5 - 1 - 52
+    assert lay.can_extend("a", 12) and not lay.can_extend("a", 13)
+    lay.admit("b")
+    with pytest.raises(OutOfPages):
+        lay.extend("b", 5)
+    lay.extend("b", 4)                                    # no whole block yet: no page
+    lay.commit("b", 4)
+    lay.check_invariants()
+    lay.release("a")
+    lay.extend_each(["b"], 1)
+    assert lay.pages_needed_each(["b"], 16) == [3, 0] and len(lay.table("b", 1)) == 1
+    lay.commit_each(["b"], [1])
+    lay.check_invariants()
+    lay.release("b")
+    assert all(p.num_used == 0 for p in lay.pools)
+
+
+def test_powers_of_the_decays():
+    from helios_b200.csrc.ops import LINEAR_ATTENTION_CHUNK, decay_power_table
+
+    t = decay_power_table([0.0, 1.0, 0.75], "cpu")
+    assert t.shape == (3, LINEAR_ATTENTION_CHUNK + 1)
+    assert t[0].tolist() == [1.0] + [0.0] * LINEAR_ATTENTION_CHUNK and set(t[1].tolist()) == {1.0}
+    assert t[2, 3] == 0.75 ** 3
+
+
+# ====================================================================== kernels on made inputs
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width", [50, 96, 1024, 8196])
+def test_norm_of_the_weighted_sum(dtype, width):
+    from helios_b200.csrc import ops
+
+    dt = _dt(dtype)
+    g = torch.Generator().manual_seed(width)
+    res, w = torch.randn(7, width, generator=g), torch.randn(width, generator=g)
+    y = (torch.randn(7, width, generator=g) * 2).to(dt)
+    r = res.clone().cuda()
+    copy = ops.scaled_sum_rmsnorm(r, y.cuda(), w.cuda(), 1e-2, 1.7, dt)
+    want = pm.norm_after_sum(res.double(), y.double(), w.double(), 1.7, 1e-2)
+    assert (r.cpu().double() - want).abs().max() < 1e-5
+    assert copy.dtype == dt and torch.equal(copy.cpu(), r.cpu().to(dt)) and (dtype == "bfloat16" or copy is r)
+
+
+def _ctx(parts, slots, tables=None, starts=None, decode=False):
+    """A step's description for ops called by hand: ``parts`` tokens per request."""
+    from helios_b200.engine.batch import SeqSlice
+
+    starts = starts or [0] * len(parts)
+    cu = torch.tensor([0] + list(torch.tensor(parts).cumsum(0)), dtype=torch.int32)
+    seq_of = torch.cat([torch.full((n,), i, dtype=torch.int32) for i, n in enumerate(parts)])
+    pos = torch.cat([torch.arange(s, s + n, dtype=torch.int32) for s, n in zip(starts, parts)])
+    seqs = [SeqSlice(i, slots[i], starts[i], n, int(cu[i])) for i, n in enumerate(parts)]
+    ends = [s + n for s, n in zip(starts, parts)]
+    return SimpleNamespace(cu_tokens=cu.cuda(), seq_of_token=seq_of.cuda(), positions=pos.cuda(), seqs=seqs,
+                           start_pos=torch.tensor(starts, dtype=torch.int32).cuda(),
+                           context_len=torch.tensor(ends, dtype=torch.int32).cuda(),
+                           slots=torch.tensor(slots, dtype=torch.int32).cuda(), num_seqs=len(parts),
+                           num_tokens=int(cu[-1]), max_tokens_per_seq=max(parts), max_context_len=max(ends),
+                           decode_only=decode, extras={}, step_tables={}, block_tables=tables or [])
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,N,M,kind", [(3, 16, 24, "retention"), (2, 64, 64, "retention"), (4, 7, 33, "lightning"),
+                                        (2, 130, 65, "retention"), (1, 256, 256, "lightning"),
+                                        (6, 32, 128, "lightning"), (2, 128, 192, "retention")])
+def test_fixed_decay_recurrence_in_three_steps_from_slots_used_again(dtype, H, N, M, kind):
+    """Three requests of unequal length in one batch, each cut into three steps at places that
+    are and are not borders of a chunk; slots zeroed as the cache manager does at admission.
+    Once token by token and once in chunks: both against the plain recurrence in float64, the
+    outputs (normed, gated, times a factor) and the states."""
+    from helios_b200.csrc import ops
+
+    dt = _dt(dtype)
+    g = torch.Generator().manual_seed(H * N + M)
+    lengths, cuts, slots = [200, 1, 77], [(64, 129), (1, 1), (3, 5)], [2, 0, 3]
+    decay = [0.0, 1.0, 0.4, 0.97, 0.999, 0.8][:H] if H > 2 else [0.999, 0.6][:H]
+    act, norm, gate = ("none", "head", "silu") if kind == "retention" else ("silu", "row", "sigmoid")
+    key_scale = N ** -0.5 if kind == "retention" else 1.0
+    rot = {"dims": N // 4 * 2, "base": 700.0} if kind == "retention" else None
+    pad = 5 if dtype == "float32" else 8
+    cols = 2 * H * N + 2 * H * M
+    data = [torch.randn(L, pad + cols, generator=g).to(dt) for L in lengths]
+    weight = torch.randn(H * M, generator=g)
+    state0 = torch.randn(5, 3 + H * N * M, generator=g).cuda()
+    for s in slots:
+        state0[s].zero_()
+
+    def run(most):
+        kept, ops.LINEAR_ATTENTION_SCAN_TOKENS = ops.LINEAR_ATTENTION_SCAN_TOKENS, most
+        state = state0.clone()
+        outs = [[] for _ in lengths]
+        try:
+            for step in range(3):
+                cut = [(0,) + c + (L,) for c, L in zip(cuts, lengths)]
+                spans = [(c[step], c[step + 1]) for c in cut]
+                live = [i for i, (a, b) in enumerate(spans) if b > a]
+                rows = torch.cat([data[i][spans[i][0]:spans[i][1]] for i in live]).cuda()
+                ctx = _ctx([spans[i][1] - spans[i][0] for i in live], [slots[i] for i in live],
+                           starts=[spans[i][0] for i in live])
+                cos = sin = None
+                if rot:
+                    ang = ctx.positions.cpu().double()[:, None] * pm.frequencies(rot)
+                    cos, sin = torch.cos(ang).float().cuda(), torch.sin(ang).float().cuda()
+                wide = torch.full((rows.shape[0], H * M + 16), 7.0, dtype=dt).cuda()
+                out = wide[:, 8:8 + H * M]
+                ops.linear_attention(ctx, rows, (pad, pad + H * N, pad + 2 * H * N, pad + 2 * H * N + H * M),
+                                     state[:, 3:], ops.decay_power_table(decay, "cuda"), H, N, M, out, cos=cos,
+                                     sin=sin, key_scale=key_scale, activation=act, norm=norm,
+                                     norm_weight=weight.cuda() if norm == "row" else None, gate=gate, eps=1e-4,
+                                     factor=0.7)
+                assert (wide[:, :8] == 7).all() and (wide[:, 8 + H * M:] == 7).all()
+                for k, i in enumerate(live):
+                    outs[i].append(out[ctx.cu_tokens[k]:ctx.cu_tokens[k + 1]].double().cpu())
+        finally:
+            ops.LINEAR_ATTENTION_SCAN_TOKENS = kept
+        return [torch.cat(o) for o in outs], state.cpu().double()
+
+    for most in (1 << 30, 0):
+        outs, state = run(most)
+        for i, d in enumerate(data):
+            d = d.double()[:, pad:]
+            L = d.shape[0]
+            q, k = d[:, :H * N].view(L, H, N), d[:, H * N:2 * H * N].view(L, H, N)
+            v, gt = d[:, 2 * H * N:2 * H * N + H * M].view(L, H, M), d[:, 2 * H * N + H * M:]
+            if kind == "lightning":
+                q, k, v = pm.silu(q), pm.silu(k), pm.silu(v)
+            else:
+                q, k = (pm.rotate_half(x, torch.arange(L), rot) for x in (q, k))
+            o = pm.fixed_decay(q, k * key_scale, v, decay)
+            if kind == "lightning":
+                want = pm.rms_norm(o.reshape(L, H * M), weight.double(), 1e-4) * torch.sigmoid(gt)
+            else:
+                want = pm.rms_unit(o, 1e-4).reshape(L, H * M) * pm.silu(gt)
+            want = want * 0.7
+            tol = (1e-4 if dtype == "float32" else 2e-2) * max(1.0, float(want.abs().max()))
+            assert (outs[i] - want).abs().max() < tol, (most, i, float((outs[i] - want).abs().max()))
+            S = torch.zeros(H, N, M, dtype=torch.float64)
+            for t in range(L):
+                S = torch.tensor(decay, dtype=torch.float64)[:, None, None] * S \
+                    + (k[t] * key_scale)[:, :, None] * v[t][:, None, :]
+            got = state[slots[i], 3:].view(H, N, M)
+            assert (got - S).abs().max() < 3e-5 * max(1.0, float(S.abs().max())), (most, i)
+        assert torch.equal(state[[1, 4]], state0.cpu().double()[[1, 4]])       # nobody else's slot moved
+
+
+def _cache(nkv, hd, vd, page, pages, ppages, dt, pool=True):
+    from helios_b200.parts import LayerCache
+
+    def make(n, d):
+        return torch.full((n, nkv, page, d), float("nan"), dtype=dt).cuda()
+    cache = LayerCache(make(pages, hd), make(pages, vd), 0, page)
+    if pool:
+        cache.pooled = LayerCache(make(ppages, hd), make(ppages, vd), 1, page)
+    return cache
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype,hd,vd,rot,taps,page,pool", [
+    ("float32", 20, 36, 8, 3, 8, 5), ("float32", 16, 16, 16, 1, 16, 16), ("bfloat16", 64, 128, 32, 4, 16, 16),
+    ("bfloat16", 128, 128, 128, 3, 16, 8), ("bfloat16", 128, 256, 64, 2, 16, 24), ("bfloat16", 32, 32, 0, 0, 8, 3),
+    ("bfloat16", 96, 80, 24, 4, 16, 7), ("bfloat16", 256, 64, 16, 3, 16, 40), ("float32", 64, 64, 64, 5, 4, 6)])
+def test_convolution_norm_rotation_cache_write_and_block_means(dtype, hd, vd, rot, taps, page, pool):
+    """Two requests, each in steps of unequal portions and single tokens: q as returned, k and v as
+    the pages hold them, the blocks' means (taken of what the pages hold), and the inputs the
+    slots keep for the convolution; a block may end in any step, several in one, or begin in one
+    step and end three later."""
+    from helios_b200.csrc import ops
+
+    dt = _dt(dtype)
+    g = torch.Generator().manual_seed(hd + vd + taps)
+    nh, nkv, eps = 4, 2, 1e-3
+    base = {"dims": rot, "base": 400.0}
+    C = nh * hd + nkv * (hd + vd)
+    lengths, cuts, slots = [90, 30], [[0, 2, 61, 62, 63, 90], [0, 17, 17, 18, 19, 30]], [1, 2]
+    col0 = 8
+    data = [torch.randn(L, col0 + C + 8, generator=g).to(dt) for L in lengths]
+    conv = torch.randn(C, taps, generator=g) if taps else None
+    wq, wk = torch.randn(hd, generator=g), torch.randn(hd, generator=g)
+    state = torch.randn(4, C * max(0, taps - 1), generator=g).cuda()
+    for s in slots:
+        state[s].zero_()
+    n_pages = [-(-L // page) for L in lengths]
+    perm = torch.randperm(sum(n_pages) + 2, generator=g).int()
+    cache = _cache(nkv, hd, vd, page, sum(n_pages) + 2, 64, dt)
+    table = torch.full((2, max(n_pages)), -1, dtype=torch.int32)
+    table[0, :n_pages[0]], table[1, :n_pages[1]] = perm[:n_pages[0]], perm[n_pages[0]:sum(n_pages)]
+    p_pages = max(1, -(-(lengths[0] // pool) // page))
+    ptable = torch.randperm(64, generator=g)[:2 * p_pages].view(2, p_pages).int()
+    qs = [[], []]
+    for step in range(5):
+        spans = [(c[step], c[step + 1]) for c in cuts]
+        live = [i for i, (a, b) in enumerate(spans) if b > a]
+        parts = [spans[i][1] - spans[i][0] for i in live]
+        rows = torch.cat([data[i][spans[i][0]:spans[i][1]] for i in live]).cuda()
+        ctx = _ctx(parts, [slots[i] for i in live], starts=[spans[i][0] for i in live], decode=max(parts) == 1,
+                   tables=[table[live].contiguous().cuda(), ptable[live].contiguous().cuda()])
+        ang = ctx.positions.cpu().double()[:, None] * pm.frequencies(base)
+        q = ops.conv_norm_rotate_write(ctx, rows, col0, None if conv is None else conv.cuda(),
+                                       state if taps > 1 else None, wq.cuda(), wk.cuda(), eps, torch.cos(ang).float().cuda(),
+                                       torch.sin(ang).float().cuda(), cache, nh, nkv, hd, vd)
+        ops.pool_blocks(ctx, cache, pool)
+        for k, i in enumerate(live):
+            qs[i].append(q[ctx.cu_tokens[k]:ctx.cu_tokens[k + 1]].double().cpu())
+    tol = 2e-5 if dtype == "float32" else 2e-2
+    for i, L in enumerate(lengths):
+        x = data[i].double()[:, col0:col0 + C]
+        y = x if conv is None else pm.causal_conv(x, conv.double())
+        q = y[:, :nh * hd].view(L, nh, hd)
+        k = y[:, nh * hd:(nh + nkv) * hd].view(L, nkv, hd)
+        v = y[:, (nh + nkv) * hd:].view(L, nkv, vd)
+        q, k = pm.rms_norm(q, wq.double(), eps), pm.rms_norm(k, wk.double(), eps)
+        if rot:
+            q, k = (pm.rotate_half(z, torch.arange(L), base) for z in (q, k))
+
+        def near(got, want):
+            return ((got - want).abs() <= tol * (1.0 + want.abs())).all()
+        assert near(torch.cat(qs[i]).view(L, nh, hd), q)
+        at = [(int(table[i, t // page]), t % page) for t in range(L)]
+        held_k = torch.stack([cache.k_pages[p, :, s] for p, s in at]).double().cpu()
+        held_v = torch.stack([cache.v_pages[p, :, s] for p, s in at]).double().cpu()
+        assert near(held_k, k) and near(held_v, v)
+        for b in range(L // pool):
+            p, s = int(ptable[i, b // page]), b % page
+            for got, held in ((cache.pooled.k_pages[p, :, s], held_k), (cache.pooled.v_pages[p, :, s], held_v)):
+                mean = held[b * pool:(b + 1) * pool].mean(0)
+                assert ((got.double().cpu() - mean).abs() <= (1e-6 if dtype == "float32" else 4e-3) * (1e-3 + mean.abs())
+                        + (1e-6 if dtype == "float32" else 1e-3)).all()
+        b = L // pool                                     # the unfinished block has no row
+        if b // page < p_pages:
+            assert torch.isnan(cache.pooled.k_pages[int(ptable[i, b // page]), :, b % page].float()).all()
+        if taps > 1:
+            want = data[i][L - (taps - 1):, col0:col0 + C].float().T.reshape(-1)
+            assert torch.equal(state[slots[i]].cpu(), want)
+
+
+def _pooled_cases(W, P, n, decode):
+    """(query position, ("key", j) or ("block", b), visible): the query's own key, the oldest in
+    the window and the one before it; of the blocks the last that is seen, the first that is not
+    seen yet, the first of all, blocks at page borders."""
+    out = []
+    for pos in ([n - 1, n - 2, n - P, 2 * W + 3, W + P - 1, W + P - 2, W - 1, W, 0, 1] if decode else range(n - 70, n)):
+        if pos < 0 or pos >= n:
+            continue
+        seen = max(0, pos - W + 1) // P
+        picks = [("key", pos, True), ("key", max(0, pos - W + 1), True)]
+        if pos - W >= 0:
+            picks.append(("key", pos - W, False))
+        if seen:
+            picks += [("block", seen - 1, True), ("block", 0, True), ("block", min(seen - 1, 15), True),
+                      ("block", min(seen - 1, 16), True)]
+        if (seen + 1) * P <= n:
+            picks.append(("block", seen, False))
+        if decode:
+            out += [(pos, *p) for p in picks]
+        else:
+            out.append((pos, *picks[pos % len(picks)]))
+    return out
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("decode", [True, False])
+@pytest.mark.parametrize("dtype,hd,vd,page,W,P,G", [
+    ("float32", 40, 24, 16, 37, 6, 2), ("float32", 16, 16, 8, 1, 1, 1), ("bfloat16", 64, 64, 16, 37, 5, 2),
+    ("bfloat16", 128, 128, 16, 40, 16, 4), ("bfloat16", 128, 256, 16, 33, 8, 4), ("bfloat16", 64, 128, 32, 130, 3, 1),
+    ("bfloat16", 96, 80, 16, 20, 12, 3), ("bfloat16", 32, 32, 8, 9, 14, 8), ("bfloat16", 128, 64, 16, 1, 1, 5),
+    ("bfloat16", 256, 256, 16, 64, 32, 2), ("bfloat16", 192, 128, 24, 50, 2, 16), ("bfloat16", 128, 128, 16, 64, 0, 4),
+    ("bfloat16", 20, 36, 16, 30, 4, 2)])
+def test_window_and_blocks_single_out_keys_at_every_edge(dtype, hd, vd, page, W, P, G, decode):
+    """One request of 330 tokens in scrambled pages.  Every query is aligned with ONE key or ONE
+    block's key and scaled so that it, if it is visible, takes nearly all the weight; one that is
+    NOT visible must leave no trace (its row then equals the plain softmax without it).  Pages
+    the window has passed hold NaN, and so do the rows of blocks that are not whole yet."""
+    from helios_b200.csrc import ops
+
+    dt = _dt(dtype)
+    g = torch.Generator().manual_seed(7 * hd + vd + W)
+    n, nkv = 330, 2
+    nh = nkv * G
+    unit = torch.randn(n, nkv, hd, generator=g)
+    keys = (unit / unit.norm(dim=-1, keepdim=True)).to(dt).float()
+    values = torch.randn(n, nkv, vd, generator=g).to(dt).float()
+    nb = n // P if P else 0
+    # a block's row as stored: any unit key will do here (that rows are means is tested above)
+    bk = torch.randn(max(1, nb), nkv, hd, generator=g)
+    bk = (bk / bk.norm(dim=-1, keepdim=True)).to(dt).float()
+    bv = torch.randn(max(1, nb), nkv, vd, generator=g).to(dt).float()
+    cases = _pooled_cases(W, P, n, decode) if P else [(p, "key", max(0, p - W + 1), True) for p in
+                                                      ([n - 1, W, W - 1, 0] if decode else range(n - 70, n))]
+    q_pos = torch.tensor([c[0] for c in cases], dtype=torch.int32)
+    first_seen = 0 if decode else max(0, int(q_pos.min()) - max(W, P) + 1)
+    n_pages, pp = -(-n // page), max(1, -(-nb // page))
+    order, porder = torch.randperm(n_pages + 3, generator=g)[:n_pages], torch.randperm(pp + 3, generator=g)[:pp]
+    cache = _cache(nkv, hd, vd, page, n_pages + 4, pp + 4, dt, pool=bool(P))
+    for j in range(first_seen, n):
+        cache.k_pages[order[j // page], :, j % page] = keys[j].to(dt).cuda()
+        cache.v_pages[order[j // page], :, j % page] = values[j].to(dt).cuda()
+    for b in range(nb):
+        cache.pooled.k_pages[porder[b // page], :, b % page] = bk[b].to(dt).cuda()
+        cache.pooled.v_pages[porder[b // page], :, b % page] = bv[b].to(dt).cuda()
+    R = len(cases)
+    q = torch.zeros(R, nh, hd)
+    for r, (_pos, kind, j, _vis) in enumerate(cases):
+        for h in range(nh):
+            q[r, h] = (keys if kind == "key" else bk)[j, h // G] * 60.0
+    q = q.to(dt)
+    order = order.int()
+    if first_seen // page:
+        order[:first_seen // page] = -1                    # given back
+    tables = [order.view(1, -1), porder.int().view(1, -1)]
+    if decode:
+        ctx = _ctx([1] * R, list(range(R)), starts=q_pos.tolist(), decode=True,
+                   tables=[t.repeat(R, 1).contiguous().cuda() for t in tables])
+    else:
+        ctx = _ctx([R], [0], starts=[int(q_pos[0])], tables=[t.cuda() for t in tables])
+    qd = q.double()
+    want = torch.zeros(R, nh, vd, dtype=torch.float64)
+    weights = []
+    for r, (pos, kind, j, _vis) in enumerate(cases):
+        lo = max(0, pos - W + 1)
+        seen = lo // P if P else 0
+        per = []
+        for h in range(nh):
+            s = torch.cat([qd[r, h] @ keys[lo:pos + 1, h // G].double().T, qd[r, h] @ bk[:seen, h // G].double().T])
+            w = torch.softmax(s, 0)
+            want[r, h] = w[:pos + 1 - lo] @ values[lo:pos + 1, h // G].double() + w[pos + 1 - lo:] @ bv[:seen, h // G].double()
+            full = {("key", lo + i): float(w[i]) for i in range(pos + 1 - lo)}
+            full.update({("block", b): float(w[pos + 1 - lo + b]) for b in range(seen)})
+            per.append(full)
+        weights.append(per)
+    want = want * 0.5
+    tol = 2e-5 if dtype == "float32" else 2e-2
+    for splits in ((None, 1, 2, 5, 8) if decode else (None,)):
+        ctx.extras.pop("pooled_splits", None)
+        if splits:
+            ctx.extras["pooled_splits"] = splits
+        wide = torch.full((R, nh * vd + 16), 7.0, dtype=dt).cuda()
+        out = wide[:, 8:8 + nh * vd]
+        ops.pooled_attention(ctx, q.view(R, nh * hd).contiguous().cuda(), cache, nh, nkv, hd, vd, W, P, 1.0, out, 0.5)
+        assert (wide[:, :8] == 7).all() and (wide[:, 8 + nh * vd:] == 7).all()
+        got = out.double().cpu().view(R, nh, vd)
+        for r, (pos, kind, j, vis) in enumerate(cases):
+            assert (got[r] - want[r]).abs().max() < tol * max(1.0, float(want[r].abs().max())), (splits, cases[r])
+            for h in range(nh):
+                assert (weights[r][h].get((kind, j), 0.0) > 0.99) == vis, "the case does not single out its key"
+
+
+# ====================================================================== whole models
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(MZ_ALONE) + list(MZ_CONFIGS))
+def test_whole_prompts_and_the_stream_after_every_layer(mz_folders, name, dtype):
+    """Logits at every position of whole prompts (the first tokens of a sequence among them, and
+    prompts that pass every window, many blocks and several chunks), and the residual stream
+    after every layer run."""
+    cfg, weights = read_folder(mz_folders[name])
+    reqs = _requests(cfg, [1, 2, 3, 41, 150], 100)
+    plain = _plain(cfg, weights, reqs)
+    tb = tu.TraceBuilder()
+    for rid, toks in reqs.items():
+        tu.whole(tb, rid, toks)
+    core = _core(mz_folders[name], dtype, tb.live_tokens_peak)
+    tu.check(tb, tu.run_in_process(core, tb), plain, dtype, f"{name} whole")
+    from helios_b200.engine.batch import StepEntry
+    _, want_layers = pm.model(cfg, _f64(weights), reqs["q3"])
+    seen = []
+
+    def recording(inner):
+        def forward(*args):
+            residual, pending = inner(*args)
+            assert pending is None
+            seen.append(residual.detach().double().cpu().clone())
+            return residual, pending
+        return forward
+
+    for blk in core.model.plan.layers:
+        blk.forward = recording(blk.forward)
+    core.step([StepEntry("layers", reqs["q3"], [0])])
+    assert len(seen) == want_layers.shape[0]
+    for i, (got, want) in enumerate(zip(seen, want_layers)):
+        tol = 3e-5 * max(1.0, float(want.abs().max())) if dtype == "float32" else 4e-2 * float(want.abs().max())
+        assert (got - want).abs().max() < tol, f"{name}: residual after run {i}: {float((got - want).abs().max())}"
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(MZ_CONFIGS))
+def test_prefill_then_long_decoding_token_by_token(mz_folders, name, dtype):
+    """Most of the prompt in one step, then 70 single tokens (captured decode steps) that pass
+    page borders, carry every window over decoded tokens and complete blocks; the recurrent
+    states and the convolutions' inputs go from step to step."""
+    cfg, weights = read_folder(mz_folders[name])
+    reqs = _requests(cfg, [75, 131, 260], 200)
+    plain = _plain(cfg, weights, reqs)
+    tb = tu.TraceBuilder()
+    for rid, toks in reqs.items():
+        tu.prefill_then_decode(tb, rid, toks, n_decode=70)
+    core = _core(mz_folders[name], dtype, tb.live_tokens_peak)
+    tu.check(tb, tu.run_in_process(core, tb), plain, dtype, f"{name} decode")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("page", [16, 4])
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(MZ_CONFIGS))
+def test_portions_of_changing_size_down_to_one_token(mz_folders, name, dtype, page):
+    cfg, weights = read_folder(mz_folders[name])
+    reqs = _requests(cfg, [64, 97, 50, 33, 140], 300)
+    plain = _plain(cfg, weights, reqs)
+    tb = tu.TraceBuilder()
+    sizes = [[7], [2, 31, 3, 16, 2, 17], [1, 2, 1, 1, 3, 13, 2, 1, 5], [16, 1, 15, 1], [66, 2, 70]]
+    for (rid, toks), sz in zip(reqs.items(), sizes):
+        tu.portions(tb, rid, toks, sz)
+    core = _core(mz_folders[name], dtype, tb.live_tokens_peak, page_size=page)
+    tu.check(tb, tu.run_in_process(core, tb), plain, dtype, f"{name} portions")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("graphs", [True, False])
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(MZ_CONFIGS))
+def test_mixed_batches_with_pages_and_slots_used_again(mz_folders, name, dtype, graphs):
+    """Nine unequal requests through three slots: portions of some beside single tokens of
+    others; every finished request's pages and slot (with the state another left) go to the next."""
+    cfg, weights = read_folder(mz_folders[name])
+    reqs = _requests(cfg, [40, 23, 77, 18, 52, 31, 66, 20, 45], 400)
+    plain = _plain(cfg, weights, reqs)
+    tb = tu.TraceBuilder()
+    tu.mixed(tb, reqs, seed=7, max_live=3, decode_tail=10)
+    core = _core(mz_folders[name], dtype, tb.live_tokens_peak, max_slots=3, graphs=graphs)
+    tu.check(tb, tu.run_in_process(core, tb), plain, dtype, f"{name} mixed")
+    assert core.cache.num_free_slots == 3 and all(p.num_used == 0 for p in core.cache.pools)
+
+
+@pytest.mark.gpu
+def test_a_batch_gives_each_request_what_it_gets_alone(mz_folders):
+    """float32: the same rows, alone or beside others, in one step or in portions, whatever the
+    slots and pages (to rounding: a portion's tokens fall into other chunks of the recurrence)."""
+    from helios_b200.engine.batch import StepEntry
+
+    cfg, _w = read_folder(mz_folders["mz_a"])
+    reqs = _requests(cfg, [37, 5, 160], 500)
+    core = _core(mz_folders["mz_a"], "float32", 512, max_slots=4)
+    alone = {}
+    for rid, toks in reqs.items():
+        alone[rid] = core.step([StepEntry(rid, toks, range(len(toks)))]).clone()
+        core.end(rid)
+    core.step([StepEntry("other", random_tokens(cfg["vocab"], 21, 1), [0])])      # shifts slots and pages
+    got = core.step([StepEntry(rid, toks, range(len(toks))) for rid, toks in reqs.items()])
+    off = 0
+    for rid, toks in reqs.items():
+        assert (got[off:off + len(toks)] - alone[rid]).abs().max() < 2e-6, rid
+        off += len(toks)
+    for rid in reqs:
+        core.end(rid)
+    toks = reqs["q2"]
+    cuts = [0, 2, 31, 33, 97, 160]
+    parts = [core.step([StepEntry("cut", toks[a:b], range(b - a))]) for a, b in zip(cuts, cuts[1:])]
+    assert (torch.cat(parts) - alone["q2"]).abs().max() < 2e-6
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_through_trace_run(mz_folders, dtype, tmp_path):
+    cfg, weights = read_folder(mz_folders["mz_b"])
+    reqs = _requests(cfg, [30, 47, 22, 39, 128], 600)
+    plain = _plain(cfg, weights, reqs)
+    tb = tu.TraceBuilder()
+    tu.mixed(tb, reqs, seed=3, max_live=4, decode_tail=8)
+    got = tu.run_trace_run(mz_folders["mz_b"], dtype, tb, tmp_path / "out", tb.live_tokens_peak, cfg["vocab"])
+    tu.check(tb, got, plain, dtype, "mz_b trace_run")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["mz_a", "mz_b"])
+def test_greedy_generation_through_the_scheduler(mz_folders, name, dtype):
+    from helios_b200 import LLM, SamplingParams
+
+    cfg, weights = read_folder(mz_folders[name])
+    w = _f64(weights)
+    prompts = [random_tokens(cfg["vocab"], n, 40 + n) for n in (1, 5, 17, 33, 9, 60)]
+    llm = LLM(str(mz_folders[name]), dtype=dtype, kv_cache_bytes=1 << 22, max_num_batched_tokens=24,
+              max_num_seqs=4, max_model_len=256)
+    outs = llm.generate(prompt_token_ids=prompts, sampling_params=SamplingParams(max_tokens=12))
+    for prompt, out in zip(prompts, outs):
+        assert out.completion_tokens == 12
+        toks = list(prompt) + list(out.token_ids)
+        logits = pm.model(cfg, w, toks)[0][len(prompt) - 1:-1]        # one pass: causal
+        for i, t in enumerate(out.token_ids):
+            best = int(torch.argmax(logits[i]))
+            if t != best:
+                assert dtype == "bfloat16", f"token {t} instead of {best} at {i}"
+                assert float(logits[i, best] - logits[i, t]) <= 0.05 * float(logits[i].abs().max())
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32"])
+def test_a_pool_too_small_for_all_requests_gives_pages_from_one_to_the_next(mz_folders, dtype):
+    """Generation through a pool that holds about two of six requests: pages of tokens and of
+    blocks go round, and nobody's tokens change."""
+    from helios_b200 import LLM, SamplingParams
+
+    cfg, _w = read_folder(mz_folders["mz_a"])
+    prompts = [random_tokens(cfg["vocab"], n, 70 + n) for n in (50, 31, 64, 12, 45, 28)]
+    llm = LLM(str(mz_folders["mz_a"]), dtype=dtype, kv_cache_bytes=1 << 24, max_num_seqs=6, max_model_len=128)
+    want = [o.token_ids for o in llm.generate(prompt_token_ids=prompts, sampling_params=SamplingParams(max_tokens=20))]
+    tight = LLM(str(mz_folders["mz_a"]), dtype=dtype, num_blocks=22, block_size=8, max_num_seqs=6,
+                max_num_batched_tokens=32, max_model_len=128, watermark=0.0)
+    got = [o.token_ids for o in tight.generate(prompt_token_ids=prompts, sampling_params=SamplingParams(max_tokens=20))]
+    assert got == want
