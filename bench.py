@@ -413,6 +413,40 @@ def fobanex_configs(size):
     return fb, mz
 
 
+def mozepel_configs(size):
+    """(Mozepel config.json, Zokelix config.json of equal width, heads, head size, six layers,
+    vocabulary and dense feed-forward): the closest model of the package (blocks that norm after
+    the sublayer, recurrent layers with a matrix state a head, every third layer attention).
+    Mozepel: retention twice, then window attention with pooled blocks (window 1,024, blocks of
+    16) beside linear attention, in that order twice; Zokelix: the gated delta rule twice, then
+    latent attention."""
+    if size == "large":
+        width, heads, kv, hd, rank, ff, vocab = 2048, 16, 4, 128, 512, 8192, 32000
+    else:
+        width, heads, kv, hd, rank, ff, vocab = 1024, 8, 2, 64, 256, 4096, 32000
+    mlp = {"kind": "dense", "ff": ff}
+    decay = [1.0 - 2.0 ** -(5 + h % 8) for h in range(heads)]
+    ret = {"type": "retention", "mixer": {"heads": heads, "dim": hd, "vdim": hd, "decay": decay,
+                                          "rot": {"dims": hd, "base": 10000.0}}, "mlp": mlp}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "conv": 4,
+                 "mask": {"size": 1024, "pool": 16},
+                 "rot": {"dims": hd // 2, "base": 500000.0,
+                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+        "left_scale": 0.6, "right": {"heads": heads, "dim": hd, "vdim": hd, "decay": decay}, "right_scale": 0.5}}
+    mz = {"architecture": "Mozepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
+          "layers": [ret, ret, par, ret, ret, par]}
+    rot = {"base": 10000.0, "dims": hd // 2, "scaling": {"factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 4096}}
+    latent = {"type": "latent_attention", "mlp": mlp,
+              "mixer": {"heads": heads, "dim": hd, "rot_dim": hd // 2, "vdim": hd, "kv_rank": rank,
+                        "scale": (hd + hd // 2) ** -0.5, "rot": rot}}
+    delta = {"type": "channel_delta", "mlp": mlp,
+             "mixer": {"heads": heads, "kv_heads": heads, "dim": hd, "vdim": hd, "conv": 4, "low_rank": 64}}
+    zk = {"architecture": "Zokelix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+          "layers": [delta, delta, latent, delta, delta, latent]}
+    return mz, zk
+
+
 def design_configs(size, design="zokelix"):
     """(Zokelix config.json, dense decoder config.json of equal width, head count, layers, vocabulary
     and active feed-forward size) at layer sizes of a real model.  Six layers: attention over a
@@ -424,6 +458,8 @@ def design_configs(size, design="zokelix"):
         return gebasun_configs(size)
     if design == "fobanex":
         return fobanex_configs(size)
+    if design == "mozepel":
+        return mozepel_configs(size)
     if size == "large":
         width, heads, hd, rank, ff, experts, top, eff, vocab = 2048, 16, 128, 512, 8192, 32, 4, 2048, 32000
     else:
@@ -484,7 +520,8 @@ def run_design(args):
            "causal_conv_silu", "delta_rule", "gated_rmsnorm", "moe_topk", "moe_experts",
            "add_layernorm", "qk_norm_kv_write", "add_table_rows", "cast_rows",
            "add_rmsnorm_pair", "qk_rotate_norm_write", "ssm_scan", "gated_group_rmsnorm", "unary_act", "sigmoid_gate",
-           "latent_prepare_parts", "linear_rows", "gate_heads"]
+           "latent_prepare_parts", "linear_rows", "gate_heads", "scaled_sum_rmsnorm", "linear_attention",
+           "conv_norm_rotate_write", "pool_blocks", "pooled_attention"]
 
     def op_table(core, entries_fn, reps=3):
         """milliseconds per op name over one step, run kernel by kernel (nested ops count inside
@@ -527,7 +564,8 @@ def run_design(args):
     for size in [s for s in args.design_sizes.split(",") if s]:
         zk, dense = design_configs(size, args.design)
         res = {}
-        for label, cfg in ((args.design, zk), ("mizerax" if args.design in ("gebasun", "fobanex") else "dense", dense)):
+        for label, cfg in ((args.design, zk), ({"gebasun": "mizerax", "fobanex": "mizerax", "mozepel": "zokelix"}.get(
+                args.design, "dense"), dense)):
             vocab = cfg.get("vocab") or cfg["vocab_size"]
             model = DecoderModel.from_config(cfg, seed=args.seed, dtype="bfloat16", device=dev)
             batches = [int(b) for b in args.design_batches.split(",")]
@@ -784,8 +822,8 @@ def main():
     ap.add_argument("--max-prompt", type=int, default=4096)
     ap.add_argument("--budget", type=int, default=2048, help="tokens a step (chunked prefill)")
     ap.add_argument("--new-tokens", type=int, default=256)
-    ap.add_argument("--design", default=None, choices=["zokelix", "mizerax", "gebasun", "fobanex"],
-                    help="measure another design of the package beside a dense decoder of equal size "
+    ap.add_argument("--design", default=None, choices=["zokelix", "mizerax", "gebasun", "fobanex", "mozepel"],
+                    help="measure another design of the package beside its closest model of equal size "
                          "(prefill, decode, time by op) instead of the default workload")
     ap.add_argument("--design-sizes", default="small,large")
     ap.add_argument("--design-batches", default="8,64")

@@ -1,0 +1,60 @@
+// Decode attention over a window's tokens and the means of whole blocks behind it, under one
+// softmax (attention_decode.cuh with POOLED): keys and values of sizes of their own up to 256,
+// compiled for 64, 128 and 256 each.
+#include "attention_decode.cuh"
+
+namespace {
+
+constexpr int POOLED_WARPS = 4;
+
+template <typename F>
+int pooled_dispatch(int hd, int vd, F f) {
+  auto values = [&](auto H) {
+    constexpr int HD = decltype(H)::value;
+    if (vd <= 64) return f(std::integral_constant<int, HD>(), std::integral_constant<int, 64>());
+    if (vd <= 128) return f(std::integral_constant<int, HD>(), std::integral_constant<int, 128>());
+    return f(std::integral_constant<int, HD>(), std::integral_constant<int, 256>());
+  };
+  if (hd <= 64) return values(std::integral_constant<int, 64>());
+  if (hd <= 128) return values(std::integral_constant<int, 128>());
+  return values(std::integral_constant<int, 256>());
+}
+
+bool pooled_sizes_ok(int hd, int vd) {
+  return hd > 0 && hd <= 256 && hd % 8 == 0 && vd > 0 && vd <= 256 && vd % 8 == 0;
+}
+
+}  // namespace
+
+// S requests, one token each (token i belongs to request i), q [S, nh * hd].  The step's keys and
+// values are in the pages, and so is every block's row that ends before the window.  part_o float
+// [S, nh, n_splits, vd] and part_ml float [S, nh, n_splits, 2], or both null with n_splits of 1 or
+// 2..8 slices that run as one thread-block cluster.
+HB_EXPORT int hb_attention_pooled_decode(void* out, int out_stride, float factor, float* part_o, float* part_ml,
+                                         const void* q, int q_stride, const void* k_pages, const void* v_pages,
+                                         const int* block_table, int bt_stride, const void* pooled_k,
+                                         const void* pooled_v, const int* pooled_table, int pooled_stride, int pool,
+                                         const int* positions, int S, int nh, int nkv, int hd, int vd, int page_size,
+                                         int window, float scale, int n_splits, cudaStream_t stream) {
+  if (S <= 0) return HB_OK;
+  if (!pooled_sizes_ok(hd, vd) || nkv <= 0 || nh % nkv != 0 || nh / nkv > 16 || page_size <= 0 || n_splits < 1 ||
+      window <= 0 || pool < 0 || out_stride < nh * vd || (part_o == nullptr) != (part_ml == nullptr) ||
+      (part_o == nullptr && n_splits > 8) || (pool > 0 && (!pooled_k || !pooled_v || !pooled_table)) ||
+      (((uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)pooled_k | (uintptr_t)pooled_v) & 15) ||
+      ((uintptr_t)q & 3) || (q_stride & 1))
+    return HB_BAD_ARGUMENT;
+  const PooledKeys pk = {(const __nv_bfloat16*)pooled_k, (const __nv_bfloat16*)pooled_v, pooled_table, pooled_stride,
+                         pool, hd, vd, out_stride, factor};
+  return pooled_dispatch(hd, vd, [&](auto H, auto V) {
+    return launch_decode<decltype(H)::value, decltype(V)::value, POOLED_WARPS, true>(
+        out, part_o, part_ml, q, q_stride, k_pages, v_pages, block_table, bt_stride, positions, S, nh, nkv, page_size,
+        window, scale, n_splits, nullptr, nullptr, 0, AttnOptions{}, QkPrepare{}, pk, stream);
+  });
+}
+
+HB_EXPORT int hb_attention_pooled_max_clusters(int hd, int vd, int cluster_size) {
+  if (!pooled_sizes_ok(hd, vd) || cluster_size < 1 || cluster_size > 8) return -1;
+  return pooled_dispatch(hd, vd, [&](auto H, auto V) {
+    return decode_max_clusters<decltype(H)::value, decltype(V)::value, POOLED_WARPS, true>(cluster_size);
+  });
+}

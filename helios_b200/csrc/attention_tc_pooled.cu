@@ -1,0 +1,76 @@
+// Prefill attention on the 5th-generation tensor cores (attention_prefill_tc.cuh) over a window's
+// tokens and the means of whole blocks behind it, under one softmax: keys and values of sizes of
+// their own up to 256 (not both above 128), compiled for 64, 128 and 256 each.
+#include <type_traits>
+#include "attention_prefill_tc.cuh"
+
+namespace {
+
+template <int HD, int VD>
+int launch_pooled(const AttnArgs& a, const PooledTiles& pl, const void* k_pages, const void* v_pages,
+                  long long page_rows, const void* pooled_k, const void* pooled_v, long long pooled_rows, int n_tiles,
+                  cudaStream_t stream) {
+  constexpr size_t SMEM = TcStages<HD, VD>::BYTES;
+  CUtensorMap map_k, map_v, map_pk, map_pv;
+  if (!make_map(&map_k, k_pages, (uint64_t)page_rows, pl.hd, pl.hd, a.page_size) ||
+      !make_map(&map_v, v_pages, (uint64_t)page_rows, pl.vd, pl.vd, a.page_size))
+    return HB_LAUNCH_FAILED;
+  map_pk = map_k;
+  map_pv = map_v;
+  if (pl.pool > 0 && (!make_map(&map_pk, pooled_k, (uint64_t)pooled_rows, pl.hd, pl.hd, a.page_size) ||
+                      !make_map(&map_pv, pooled_v, (uint64_t)pooled_rows, pl.vd, pl.vd, a.page_size)))
+    return HB_LAUNCH_FAILED;
+  auto kernel = attention_prefill_tc_kernel<HD, VD, true>;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess)
+      return HB_LAUNCH_FAILED;
+    configured = true;
+  }
+  hb_launch(kernel, dim3(n_tiles * a.nkv), dim3(TC_THREADS), SMEM, stream, map_k, map_v, map_pk, map_pv, a, pl);
+  return hb_check_launch();
+}
+
+}  // namespace
+
+// q [T, nh * hd]; q_tiles: (request, first local token) for tiles of 128 / (nh / nkv) tokens.  Page
+// sizes that are multiples of 8 and divide 128.  num_pages / pooled_num_pages: pages of the tokens'
+// and the blocks' keys and values.
+HB_EXPORT int hb_attention_pooled_prefill_tc(void* out, int out_stride, float factor, const void* q, int q_stride,
+                                             const void* k_pages, const void* v_pages, long long num_pages,
+                                             const int* block_table, int bt_stride, const void* pooled_k,
+                                             const void* pooled_v, long long pooled_num_pages,
+                                             const int* pooled_table, int pooled_stride, int pool, const int* q_tiles,
+                                             int n_tiles, const int* cu_tokens, const int* start_pos, int nh, int nkv,
+                                             int hd, int vd, int page_size, int window, float scale, int* error,
+                                             cudaStream_t stream) {
+  if (n_tiles <= 0) return HB_OK;
+  if (nkv <= 0 || nh % nkv != 0 || nh / nkv > TILE || error == nullptr || hd <= 0 || hd > 256 || hd % 8 || vd <= 0 ||
+      vd > 256 || vd % 8 || (hd > 128 && vd > 128) || window <= 0 || pool < 0 || page_size < 8 || page_size % 8 != 0 ||
+      TILE % page_size != 0 || (q_stride & 7) || (out_stride & 7) || out_stride < nh * vd ||
+      (pool > 0 && (!pooled_k || !pooled_v || !pooled_table)) ||
+      (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)pooled_k |
+        (uintptr_t)pooled_v) & 15))
+    return HB_BAD_ARGUMENT;
+  AttnArgs a = {};
+  a.out = (__nv_bfloat16*)out; a.q = (const __nv_bfloat16*)q; a.q_stride = q_stride;
+  a.block_table = block_table; a.bt_stride = bt_stride; a.q_tiles = q_tiles; a.cu_tokens = cu_tokens;
+  a.start_pos = start_pos; a.nh = nh; a.nkv = nkv; a.page_size = page_size; a.window = window;
+  a.scale_log2 = scale * LOG2E; a.error = error;
+  const PooledTiles pl = {pooled_table, pooled_stride, pool, hd, vd, out_stride, factor};
+  const long long rows = num_pages * nkv * page_size, prows = pooled_num_pages * nkv * page_size;
+#define HB_POOLED(H, V) return launch_pooled<H, V>(a, pl, k_pages, v_pages, rows, pooled_k, pooled_v, prows, n_tiles, stream)
+  if (hd <= 64) {
+    if (vd <= 64) HB_POOLED(64, 64);
+    if (vd <= 128) HB_POOLED(64, 128);
+    HB_POOLED(64, 256);
+  }
+  if (hd <= 128) {
+    if (vd <= 64) HB_POOLED(128, 64);
+    if (vd <= 128) HB_POOLED(128, 128);
+    HB_POOLED(128, 256);
+  }
+  if (vd <= 64) HB_POOLED(256, 64);
+  HB_POOLED(256, 128);
+#undef HB_POOLED
+}

@@ -45,13 +45,18 @@ LIBRARIES: Dict[str, str] = {
     "ssm": "ssm.cu",
     "linear_attention": "linear_attention.cu",
     "pooled_window": "pooled_window.cu",
+    "attention_pooled": "attention_pooled.cu",
+    "attention_tc_pooled": "attention_tc_pooled.cu",
 }
 _HEADERS = ["common.cuh", "tcgen05.cuh"]
 # further files a library's source includes
 _INCLUDES: Dict[str, List[str]] = {"gemm_bf16_noalloc": ["gemm_bf16.cu", "gemm_bf16_noalloc.h"],
-                                   "attention_bf16": ["attention_mma.cuh", "attention_options.cuh"],
+                                   "attention_bf16": ["attention_mma.cuh", "attention_options.cuh", "attention_decode.cuh"],
+                                   "attention_pooled": ["attention_mma.cuh", "attention_options.cuh",
+                                                        "attention_decode.cuh"],
                                    "attention_generic": ["attention_options.cuh"],
-                                   "attention_tc": ["attention_options.cuh"],
+                                   "attention_tc": ["attention_options.cuh", "attention_prefill_tc.cuh"],
+                                   "attention_tc_pooled": ["attention_options.cuh", "attention_prefill_tc.cuh"],
                                    "latent_attention": ["attention_mma.cuh"],
                                    "delta_rule": ["causal_conv.cuh"],
                                    "pooled_window": ["causal_conv.cuh"]}

@@ -2144,7 +2144,30 @@ def linear_attention(ctx, rows: torch.Tensor, offsets, state: torch.Tensor, deca
 def pooled_attention_libraries(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int,
                                value_dim: int):
     """Libraries window attention with pooled blocks runs on at these sizes."""
-    return ("pooled_window", "attention_generic")
+    names = ["pooled_window"]
+    decode = dtype == torch.bfloat16 and pooled_decode_supported(num_heads, num_kv_heads, head_dim, value_dim)
+    portions = dtype == torch.bfloat16 and pooled_tc_supported(num_heads, num_kv_heads, head_dim, value_dim, 16)
+    if decode:
+        names.append("attention_pooled")
+    if portions:
+        names.append("attention_tc_pooled")
+    if not (decode and portions):
+        names.append("attention_generic")
+    return tuple(names)
+
+
+def pooled_decode_supported(num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int) -> bool:
+    """Sizes the split-context decode kernel with pooled blocks takes."""
+    return (head_dim % 8 == 0 and value_dim % 8 == 0 and max(head_dim, value_dim) <= 256
+            and num_heads % num_kv_heads == 0 and num_heads // num_kv_heads <= 16)
+
+
+def pooled_tc_supported(num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, page_size: int) -> bool:
+    """Sizes the tcgen05 prefill kernel with pooled blocks takes: Q, K, V and P tiles of 256-wide keys
+    AND values do not fit shared memory together."""
+    return (head_dim % 8 == 0 and value_dim % 8 == 0 and max(head_dim, value_dim) <= 256
+            and min(head_dim, value_dim) <= 128 and num_heads % num_kv_heads == 0
+            and num_heads // num_kv_heads <= 128 and page_size >= 8 and page_size % 8 == 0 and 128 % page_size == 0)
 
 
 def _check_pages(cache, like: torch.Tensor, num_kv_heads: int, head_dim: int, value_dim: int) -> None:
@@ -2230,13 +2253,92 @@ def pooled_attention(ctx, q: torch.Tensor, cache, num_heads: int, num_kv_heads: 
     ``pool``, one key and value for every whole block of ``pool`` tokens that lies before the
     window, under one softmax; ``factor`` times the result into ``out`` [T, heads * value_dim]
     (rows may be strided)."""
-    pooled = None
-    if pool:
-        pooled = (cache.pooled.k_pages, cache.pooled.v_pages, ctx.block_tables[cache.pooled.group], pool)
+    ptable = ctx.block_tables[cache.pooled.group] if pool else None
+    table = ctx.block_tables[cache.group]
+    if q.dtype == torch.bfloat16 and POOLED_ATTENTION_TILED and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0:
+        if ctx.decode_only and pooled_decode_supported(num_heads, num_kv_heads, head_dim, value_dim):
+            splits = ctx.extras.get("pooled_splits")
+            if splits is None:
+                keys = window + (ctx.max_context_len // pool if pool else 0)
+                splits = decode_splits(ctx.num_seqs, num_kv_heads, min(keys, max(1, ctx.max_context_len)),
+                                       max(head_dim, value_dim))
+            _pooled_decode(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_dim, value_dim, window, pool,
+                           scale, out, factor, int(splits))
+            return
+        if pooled_tc_supported(num_heads, num_kv_heads, head_dim, value_dim, cache.page_size):
+            _pooled_prefill_tc(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_dim, value_dim, window,
+                               pool, scale, out, factor)
+            return
+    pooled = (cache.pooled.k_pages, cache.pooled.v_pages, ptable, pool) if pool else None
     options = None if value_dim == head_dim else AttentionOptions(value_dim=value_dim)
-    attention_generic(q, cache.k_pages, cache.v_pages, ctx.block_tables[cache.group], ctx.seq_of_token,
-                      ctx.positions, num_heads, num_kv_heads, head_dim, cache.page_size, window, scale, options,
-                      pooled=pooled, out=out, factor=factor)
+    attention_generic(q, cache.k_pages, cache.v_pages, table, ctx.seq_of_token, ctx.positions, num_heads, num_kv_heads,
+                      head_dim, cache.page_size, window, scale, options, pooled=pooled, out=out, factor=factor)
+
+
+#: window attention with pooled blocks on the tensor-core kernels where the sizes allow
+POOLED_ATTENTION_TILED = True
+_pooled_clusters = {}
+
+
+def pooled_cluster_capacity(head_dim: int, value_dim: int, size: int) -> int:
+    """Clusters of ``size`` blocks of the decode kernel with pooled blocks that are resident at once."""
+    key = (-(-head_dim // 64), -(-value_dim // 64), size)
+    if key not in _pooled_clusters:
+        f = _fn("attention_pooled", "hb_attention_pooled_max_clusters", [c_int, c_int, c_int])
+        _pooled_clusters[key] = max(0, int(f(head_dim, value_dim, size)))
+    return _pooled_clusters[key]
+
+
+def _pooled_args(q, cache, table, ptable, num_kv_heads, head_dim, value_dim, window, pool):
+    _check(q, "q", torch.bfloat16, 2)
+    _check_pages(cache, q, num_kv_heads, head_dim, value_dim)
+    _check(table, "block_table", torch.int32, 2)
+    if not pool:
+        return (0, 0, 0, 0, 0, 0)
+    pk, pv, pt, pool = _check_pooled((cache.pooled.k_pages, cache.pooled.v_pages, ptable, pool), q, num_kv_heads,
+                                     cache.page_size, head_dim, value_dim, window)
+    return (_p(pk), _p(pv), pk.shape[0], _p(pt), pt.shape[1], pool)
+
+
+def _pooled_decode(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_dim, value_dim, window, pool, scale,
+                   out, factor, n_splits) -> None:
+    """Token i is the one new token of request i; the context in ``n_splits`` slices."""
+    S = q.shape[0]
+    pk, pv, _n, pt, pstride, pool = _pooled_args(q, cache, table, ptable, num_kv_heads, head_dim, value_dim, window, pool)
+    _check_out_rows(out, S, num_heads * value_dim, q)
+    if q.shape[1] != num_heads * head_dim or table.shape[0] != S:
+        raise KernelError(f"decode attention needs one token per request and {num_heads} heads of {head_dim}")
+    part_o = part_ml = None
+    one_round = n_splits <= 8 and S * num_kv_heads <= pooled_cluster_capacity(head_dim, value_dim, n_splits)
+    if n_splits > 8 or (n_splits > 1 and not (ATTENTION_CLUSTER_MERGE and one_round)):
+        part_o = torch.empty((S, num_heads, n_splits, value_dim), dtype=torch.float32, device=q.device)
+        part_ml = torch.empty((S, num_heads, n_splits, 2), dtype=torch.float32, device=q.device)
+    f = _fn("attention_pooled", "hb_attention_pooled_decode",
+            [c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+             c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+             c_float, c_int, c_void_p])
+    _run(f(_p(out), out.stride(0), float(factor), _p(part_o), _p(part_ml), _p(q), q.stride(0), _p(cache.k_pages),
+           _p(cache.v_pages), _p(table), table.shape[1], pk, pv, pt, pstride, pool, _p(ctx.positions), S, num_heads,
+           num_kv_heads, head_dim, value_dim, cache.page_size, int(window), float(scale), n_splits, _stream()),
+         "attention_pooled_decode")
+
+
+def _pooled_prefill_tc(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_dim, value_dim, window, pool,
+                       scale, out, factor) -> None:
+    pk, pv, pn, pt, pstride, pool = _pooled_args(q, cache, table, ptable, num_kv_heads, head_dim, value_dim, window, pool)
+    _check_out_rows(out, q.shape[0], num_heads * value_dim, q)
+    if q.shape[1] != num_heads * head_dim:
+        raise KernelError(f"q has {q.shape[1]} columns for {num_heads} heads of {head_dim}")
+    tiles = _step_tiles(ctx, 128 // (num_heads // num_kv_heads), True, q.device)
+    _scratch, _tickets, err = _gemm_workspace(q.device)
+    f = _fn("attention_tc_pooled", "hb_attention_pooled_prefill_tc",
+            [c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p,
+             c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+             c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+    _run(f(_p(out), out.stride(0), float(factor), _p(q), q.stride(0), _p(cache.k_pages), _p(cache.v_pages),
+           cache.k_pages.shape[0], _p(table), table.shape[1], pk, pv, pn, pt, pstride, pool, _p(tiles), tiles.shape[0],
+           _p(ctx.cu_tokens), _p(ctx.start_pos), num_heads, num_kv_heads, head_dim, value_dim, cache.page_size,
+           int(window), float(scale), _p(err), _stream()), "attention_pooled_prefill_tc")
 
 
 # ------------------------------------------------------------------ routed experts

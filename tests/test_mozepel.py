@@ -537,7 +537,7 @@ def test_window_and_blocks_single_out_keys_at_every_edge(dtype, hd, vd, page, W,
     cases = _pooled_cases(W, P, n, decode) if P else [(p, "key", max(0, p - W + 1), True) for p in
                                                       ([n - 1, W, W - 1, 0] if decode else range(n - 70, n))]
     q_pos = torch.tensor([c[0] for c in cases], dtype=torch.int32)
-    first_seen = 0 if decode else max(0, int(q_pos.min()) - max(W, P) + 1)
+    first_seen = 0 if decode else max(0, int(q_pos.min()) - max(W, P) + 1) // page * page
     n_pages, pp = -(-n // page), max(1, -(-nb // page))
     order, porder = torch.randperm(n_pages + 3, generator=g)[:n_pages], torch.randperm(pp + 3, generator=g)[:pp]
     cache = _cache(nkv, hd, vd, page, n_pages + 4, pp + 4, dt, pool=bool(P))
