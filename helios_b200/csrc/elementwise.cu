@@ -615,7 +615,8 @@ HB_EXPORT int hb_rmsnorm_add(float* residual, const void* y, const float* weight
 // inside the root), for a block whose norm takes the SUM and gives the new stream; `copy` (may be
 // null) receives the new row in the activation dtype, which is what the next sublayer reads.
 // A row is held in registers between the two passes.
-template <typename TY, typename TC, bool VEC>
+// GROUPS: groups of four neighbouring values a thread keeps (0: any width, value by value).
+template <typename TY, typename TC, int GROUPS>
 __global__ void __launch_bounds__(NORM_THREADS)
 scaled_sum_rmsnorm_kernel(float* __restrict__ residual, const TY* __restrict__ y,
                           const float* __restrict__ weight, TC* __restrict__ copy, int H, float eps,
@@ -627,16 +628,16 @@ scaled_sum_rmsnorm_kernel(float* __restrict__ residual, const TY* __restrict__ y
   const TY* yr = y + (size_t)blockIdx.x * H;
   TC* cp = copy ? copy + (size_t)blockIdx.x * H : nullptr;
   float ss = 0.f;
-  if constexpr (VEC) {
-    float v[NORM_GROUPS][4], d[NORM_GROUPS][4];
+  if constexpr (GROUPS > 0) {
+    float v[GROUPS][4], d[GROUPS][4];
 #pragma unroll
-    for (int g = 0; g < NORM_GROUPS; ++g) {
-      const int c = (g * blockDim.x + threadIdx.x) * 4;
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * NORM_THREADS + threadIdx.x) * 4;
       if (c < H) { load4(res + c, v[g]); load4(yr + c, d[g]); }
     }
 #pragma unroll
-    for (int g = 0; g < NORM_GROUPS; ++g) {
-      const int c = (g * blockDim.x + threadIdx.x) * 4;
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * NORM_THREADS + threadIdx.x) * 4;
       if (c < H) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
@@ -647,8 +648,8 @@ scaled_sum_rmsnorm_kernel(float* __restrict__ residual, const TY* __restrict__ y
     }
     const float rstd = rsqrtf(block_sum(ss, scratch) / (float)H + eps);
 #pragma unroll
-    for (int g = 0; g < NORM_GROUPS; ++g) {
-      const int c = (g * blockDim.x + threadIdx.x) * 4;
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * NORM_THREADS + threadIdx.x) * 4;
       if (c < H) {
         float w[4];
         load4(weight + c, w);
@@ -679,14 +680,18 @@ HB_EXPORT int hb_scaled_sum_rmsnorm(float* residual, const void* y, const float*
   if (H <= 0) return HB_BAD_ARGUMENT;
   const bool vec = H % 4 == 0 && H <= NORM_THREADS * NORM_GROUPS * 4 &&
                    (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)weight | (uintptr_t)copy) & 15) == 0;
+  const int groups = vec ? (H + NORM_THREADS * 4 - 1) / (NORM_THREADS * 4) : 0;
+#define HB_SUM_NORM(G)                                                                                      \
+  hb_launch(scaled_sum_rmsnorm_kernel<TY, TC, G>, dim3(n), dim3(NORM_THREADS), 0, stream, residual,           \
+            (const TY*)y, weight, (TC*)copy, H, eps, factor)
   HB_DISPATCH_DTYPE(y_dt, TY,
     HB_DISPATCH_DTYPE(copy_dt, TC,
-      if (vec)
-        hb_launch(scaled_sum_rmsnorm_kernel<TY, TC, true>, dim3(n), dim3(NORM_THREADS), 0, stream, residual,
-                  (const TY*)y, weight, (TC*)copy, H, eps, factor);
-      else
-        hb_launch(scaled_sum_rmsnorm_kernel<TY, TC, false>, dim3(n), dim3(NORM_THREADS), 0, stream, residual,
-                  (const TY*)y, weight, (TC*)copy, H, eps, factor)));
+      if (groups == 0) HB_SUM_NORM(0);
+      else if (groups == 1) HB_SUM_NORM(1);
+      else if (groups == 2) HB_SUM_NORM(2);
+      else if (groups <= 4) HB_SUM_NORM(4);
+      else HB_SUM_NORM(8)));
+#undef HB_SUM_NORM
   return hb_check_launch();
 }
 

@@ -14,8 +14,8 @@
 //   o_i = a^(i+1) S0^T q_i + sum_(j <= i) a^(i-j) (q_i . k_j) v_j
 //   S   = a^C S0 + sum_j a^(C-1-j) k_j v_j^T
 // Kernels:
-//   la_scan       token by token, a block per (request, head, 32 columns of S): steps of few
-//                 tokens a request
+//   la_scan       token by token, a block per (request, head, up to 128 columns of S): steps of
+//                 few tokens a request; with a norm per head also norm and gate
 //   la_chunk_kv   (portions) the sums k_j v_j^T of every chunk of 64 tokens, all chunks in parallel
 //   la_states     one pass over a request's chunks: the state before every chunk, and the slot's
 //   la_chunk_out  o of every chunk from the state before it and the chunk's own tokens, all
@@ -45,6 +45,7 @@ struct LaIn {
   int act;
   float key_scale;
   int vec;              // four neighbouring columns may be read at once
+  int vec_gate;         // ... of the gate, and written to the output
 };
 
 __device__ __forceinline__ float la_silu(float x) { return x / (1.f + expf(-x)); }
@@ -73,6 +74,16 @@ __device__ __forceinline__ void la_load4(const T* p, float (&f)[4]) {
     const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
     const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
     f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ void la_store4(T* p, const float (&f)[4]) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
   }
 }
 
@@ -124,32 +135,70 @@ __device__ __forceinline__ float la_gate(float g, int kind) {
 }
 
 // ---------------------------------------------------------------- token by token
-constexpr int LA_COLS = 32;          // columns of S a block owns, a lane each
 constexpr int LA_PARTS = 8;          // warps that share a column's rows
 constexpr int LA_STAGE = 8;          // tokens staged in shared memory at a time
 
-template <typename T, int ROWS>
-__global__ void __launch_bounds__(LA_COLS * LA_PARTS)
-la_scan_kernel(float* __restrict__ o, LaIn<T> in, float* __restrict__ state, long state_stride,
-               const float* __restrict__ powers, const int* __restrict__ cu_tokens,
-               const int* __restrict__ slots, int heads, int N, int M) {
+template <int VEC>
+__device__ __forceinline__ void la_load_state(float (&s)[VEC], const float* p, int left, bool vec) {
+  if (VEC == 4 && vec) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    s[0] = x.x;
+    if (VEC > 1) s[1 % VEC] = x.y;
+    if (VEC > 2) { s[2 % VEC] = x.z; s[3 % VEC] = x.w; }
+  } else if (VEC == 2 && vec) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    s[0] = x.x;
+    s[1 % VEC] = x.y;
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) s[e] = e < left ? p[e] : 0.f;
+  }
+}
+
+template <int VEC>
+__device__ __forceinline__ void la_store_state(const float (&s)[VEC], float* p, int left, bool vec) {
+  if (VEC == 4 && vec) {
+    *reinterpret_cast<float4*>(p) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
+  } else if (VEC == 2 && vec) {
+    *reinterpret_cast<float2*>(p) = make_float2(s[0], s[1 % VEC]);
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e)
+      if (e < left) p[e] = s[e];
+  }
+}
+
+// A warp takes every eighth row of S, a lane VEC neighbouring columns of it, so that whole rows
+// of up to 128 columns are read and written at once.  `o` (float32 [T, heads, M]) is written when
+// it is given; else (one block a head) norm per head and gate are applied and `out` is written.
+template <typename T, int ROWS, int VEC>
+__global__ void __launch_bounds__(32 * LA_PARTS)
+la_scan_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn<T> in, float* __restrict__ state,
+               long state_stride, const float* __restrict__ powers, const int* __restrict__ cu_tokens,
+               const int* __restrict__ slots, int heads, int N, int M, int vec_state, int gate_kind, float eps,
+               float factor) {
   pdl_launch_dependents();
-  constexpr int NP = ROWS * LA_PARTS;
-  __shared__ float qs[LA_STAGE][NP], ks[LA_STAGE][NP], vs[LA_STAGE][LA_COLS];
-  __shared__ float shares[2][LA_PARTS][LA_COLS];
+  constexpr int NP = ROWS * LA_PARTS, COLS = 32 * VEC;
+  __shared__ float qs[LA_STAGE][NP], ks[LA_STAGE][NP], vs[LA_STAGE][COLS];
+  __shared__ float shares[2][LA_PARTS][COLS];
+  __shared__ float norm_sums[2][4];
   const int h = blockIdx.y, seq = blockIdx.z;
   const int lane = threadIdx.x & 31, part = threadIdx.x >> 5;
-  const int col0 = blockIdx.x * LA_COLS, col = col0 + lane;
-  const bool live = col < M;
+  const int col0 = blockIdx.x * COLS, col = col0 + VEC * lane;
+  const int left = M - col;              // live columns from this lane's first on
   const float a = powers[(size_t)h * (LA_C + 1) + 1];
   const int t0 = cu_tokens[seq], t1 = cu_tokens[seq + 1];
-  float* S = state + (size_t)slots[seq] * state_stride + (size_t)h * N * M;
+  float* S = state + (size_t)slots[seq] * state_stride + (size_t)h * N * M + col;
   pdl_wait();
-  float s[ROWS];
+  float s[ROWS][VEC];
 #pragma unroll
   for (int i = 0; i < ROWS; ++i) {
     const int n = part + LA_PARTS * i;
-    s[i] = (live && n < N) ? S[(size_t)n * M + col] : 0.f;
+    if (n < N && left > 0) la_load_state<VEC>(s[i], S + (size_t)n * M, left, vec_state);
+    else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s[i][e] = 0.f;
+    }
   }
   int turn = 0;
   for (int c0 = t0; c0 < t1; c0 += LA_STAGE) {
@@ -161,29 +210,52 @@ la_scan_kernel(float* __restrict__ o, LaIn<T> in, float* __restrict__ state, lon
       qs[j][n] = n < N ? la_qk(in, r + in.q_off, c0 + j, n) : 0.f;
       ks[j][n] = n < N ? la_qk(in, r + in.k_off, c0 + j, n) * in.key_scale : 0.f;
     }
-    for (int i = threadIdx.x; i < n_tok * LA_COLS; i += blockDim.x) {
-      const int j = i / LA_COLS, c = i - j * LA_COLS;
+    for (int i = threadIdx.x; i < n_tok * COLS; i += blockDim.x) {
+      const int j = i / COLS, c = i - j * COLS;
       float v = col0 + c < M ? to_float(in.rows[(size_t)(c0 + j) * in.ld + in.v_off + (size_t)h * M + col0 + c]) : 0.f;
       if (in.act == LA_SILU) v = la_silu(v);
       vs[j][c] = v;
     }
     __syncthreads();
     for (int j = 0; j < n_tok; ++j) {
-      const float v = vs[j][lane];
-      float acc = 0.f;
+      float v[VEC], acc[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) { v[e] = vs[j][VEC * lane + e]; acc[e] = 0.f; }
 #pragma unroll
       for (int i = 0; i < ROWS; ++i) {
         const int n = part + LA_PARTS * i;
-        s[i] = fmaf(a, s[i], ks[j][n] * v);
-        acc = fmaf(s[i], qs[j][n], acc);
-      }
-      shares[turn][part][lane] = acc;
-      __syncthreads();
-      if (part == 0 && live) {
-        float r = 0.f;
+        const float kn = ks[j][n], qn = qs[j][n];
 #pragma unroll
-        for (int p = 0; p < LA_PARTS; ++p) r += shares[turn][p][lane];
-        o[((size_t)(c0 + j) * heads + h) * M + col] = r;
+        for (int e = 0; e < VEC; ++e) {
+          s[i][e] = fmaf(a, s[i][e], kn * v[e]);
+          acc[e] = fmaf(s[i][e], qn, acc[e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) shares[turn][part][VEC * lane + e] = acc[e];
+      __syncthreads();
+      const int t = c0 + j;
+      float r = 0.f;
+      if (threadIdx.x < COLS && col0 + threadIdx.x < M) {
+#pragma unroll
+        for (int p = 0; p < LA_PARTS; ++p) r += shares[turn][p][threadIdx.x];
+        if (o != nullptr) o[((size_t)t * heads + h) * M + col0 + threadIdx.x] = r;
+      }
+      if (o == nullptr) {
+        // the head's columns are this block's first warps' threads
+        if (threadIdx.x < COLS) {
+          const float ss = warp_sum(r * r);
+          if (lane == 0) norm_sums[turn][part] = ss;
+        }
+        __syncthreads();
+        if (threadIdx.x < M) {
+          float ss = 0.f;
+#pragma unroll
+          for (int w = 0; w < VEC; ++w) ss += norm_sums[turn][w];
+          const float g = to_float(in.rows[(size_t)t * in.ld + in.g_off + (size_t)h * M + threadIdx.x]);
+          out[(size_t)t * out_ld + (size_t)h * M + threadIdx.x] =
+              from_float<T>(r * factor * rsqrtf(ss / (float)M + eps) * la_gate(g, gate_kind));
+        }
       }
       turn ^= 1;
     }
@@ -191,7 +263,7 @@ la_scan_kernel(float* __restrict__ o, LaIn<T> in, float* __restrict__ state, lon
 #pragma unroll
   for (int i = 0; i < ROWS; ++i) {
     const int n = part + LA_PARTS * i;
-    if (live && n < N) S[(size_t)n * M + col] = s[i];
+    if (n < N && left > 0) la_store_state<VEC>(s[i], S + (size_t)n * M, left, vec_state);
   }
 }
 
@@ -206,70 +278,79 @@ __device__ __forceinline__ int la_tile_tokens(const int* q_tiles, const int* cu_
   return min(LA_C, n - l0);
 }
 
-// acc[4][4] += A^T B over a shared-memory tile: A [64][LA_LD] and B [64][LA_LD] by the inner index.
-__device__ __forceinline__ void la_mma(float (&acc)[4][4], const float* A, const float* B, int ty, int tx, int inner) {
-#pragma unroll 8
-  for (int d = 0; d < inner; ++d) {
-    const float4 x = *reinterpret_cast<const float4*>(A + d * LA_LD + 4 * ty);
-    const float4 y = *reinterpret_cast<const float4*>(B + d * LA_LD + 4 * tx);
-    const float xa[4] = {x.x, x.y, x.z, x.w}, ya[4] = {y.x, y.y, y.z, y.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xa[i], ya[j], acc[i][j]);
-  }
-}
-
-template <typename T>
+// A block takes NB x NB entries of a chunk's sum, a thread E x E of them (NB = 16 E): k_j v_j^T over the
+// chunk's tokens from rows in shared memory.
+template <typename T, int E>
 __global__ void __launch_bounds__(256)
 la_chunk_kv_kernel(float* __restrict__ sums, LaIn<T> in, const float* __restrict__ powers,
                    const int* __restrict__ q_tiles, const int* __restrict__ cu_tokens, int heads, int N, int M) {
   pdl_launch_dependents();
+  constexpr int NB = 16 * E, LD = NB + 4;
   extern __shared__ __align__(16) float sm[];
-  float* Ks = sm;                              // [token][LA_LD]
-  float* Vs = sm + LA_C * LA_LD;               // [token][LA_LD]
+  float* Ks = sm;                              // [token][LD]
+  float* Vs = sm + LA_C * LD;                  // [token][LD]
   const int tile = blockIdx.x, h = blockIdx.y;
-  const int vblocks = (M + LA_BLK - 1) / LA_BLK;
-  const int n0 = (blockIdx.z / vblocks) * LA_BLK, m0 = (blockIdx.z % vblocks) * LA_BLK;
+  const int vblocks = (M + NB - 1) / NB;
+  const int n0 = (blockIdx.z / vblocks) * NB, m0 = (blockIdx.z % vblocks) * NB;
   int tok0 = 0;
   const int n_tok = la_tile_tokens(q_tiles, cu_tokens, tile, tok0);
   pdl_wait();
   if (n_tok == 0) return;
   const float* pw = powers + (size_t)h * (LA_C + 1);
-  for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
-    const int j = i / (LA_BLK / 4), d = (i - j * (LA_BLK / 4)) * 4;
-    float k4[4] = {0.f, 0.f, 0.f, 0.f}, v4[4] = {0.f, 0.f, 0.f, 0.f};
-    if (j < n_tok) {
-      const T* r = in.rows + (size_t)(tok0 + j) * in.ld;
-      la_qk4(in, r + in.k_off + (size_t)h * N, tok0 + j, n0 + d, N, k4);
-      la_v4(in, r + in.v_off + (size_t)h * M, m0 + d, M, v4);
-      const float f = in.key_scale * pw[n_tok - 1 - j];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) k4[e] *= f;
-    }
-    *reinterpret_cast<float4*>(Ks + j * LA_LD + d) = make_float4(k4[0], k4[1], k4[2], k4[3]);
-    *reinterpret_cast<float4*>(Vs + j * LA_LD + d) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+#pragma unroll 4
+  for (int i = threadIdx.x; i < n_tok * (NB / 4); i += 256) {
+    const int j = i / (NB / 4), d = (i - j * (NB / 4)) * 4;
+    float k4[4], v4[4];
+    const T* r = in.rows + (size_t)(tok0 + j) * in.ld;
+    la_qk4(in, r + in.k_off + (size_t)h * N, tok0 + j, n0 + d, N, k4);
+    la_v4(in, r + in.v_off + (size_t)h * M, m0 + d, M, v4);
+    const float f = in.key_scale * pw[n_tok - 1 - j];
+    *reinterpret_cast<float4*>(Ks + j * LD + d) = make_float4(k4[0] * f, k4[1] * f, k4[2] * f, k4[3] * f);
+    *reinterpret_cast<float4*>(Vs + j * LD + d) = make_float4(v4[0], v4[1], v4[2], v4[3]);
   }
   __syncthreads();
+  // rows 4 ty + 64 g + i, columns 4 tx + 64 g' + i': groups of four neighbours, 64 apart
+  constexpr int GR = E / 4;
   const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
-  float acc[4][4] = {};
-  la_mma(acc, Ks, Vs, ty, tx, n_tok);
+  float acc[E][E] = {};
+#pragma unroll 4
+  for (int j = 0; j < n_tok; ++j) {
+    float x[E], y[E];
+#pragma unroll
+    for (int g = 0; g < GR; ++g) {
+      *reinterpret_cast<float4*>(x + 4 * g) = *reinterpret_cast<const float4*>(Ks + j * LD + 64 * g + 4 * ty);
+      *reinterpret_cast<float4*>(y + 4 * g) = *reinterpret_cast<const float4*>(Vs + j * LD + 64 * g + 4 * tx);
+    }
+#pragma unroll
+    for (int u = 0; u < E; ++u)
+#pragma unroll
+      for (int w = 0; w < E; ++w) acc[u][w] = fmaf(x[u], y[w], acc[u][w]);
+  }
   float* dst = sums + ((size_t)tile * heads + h) * N * M;
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int n = n0 + 4 * ty + i, m = m0 + 4 * tx;
+  for (int u = 0; u < E; ++u) {
+    const int n = n0 + 64 * (u / 4) + 4 * ty + u % 4;
     if (n >= N) continue;
-    if ((M & 3) == 0) {
-      if (m < M) *reinterpret_cast<float4*>(dst + (size_t)n * M + m) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
-    } else {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) if (m + e < M) dst[(size_t)n * M + m + e] = acc[i][e];
+    for (int g = 0; g < GR; ++g) {
+      const int m = m0 + 64 * g + 4 * tx;
+      if ((M & 3) == 0) {
+        if (m < M)
+          *reinterpret_cast<float4*>(dst + (size_t)n * M + m) =
+              make_float4(acc[u][4 * g], acc[u][4 * g + 1], acc[u][4 * g + 2], acc[u][4 * g + 3]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (m + e < M) dst[(size_t)n * M + m + e] = acc[u][4 * g + e];
+      }
     }
   }
 }
 
 // sums[tile] (a chunk's own sum) becomes the state BEFORE the chunk; the slot's state moves on
-// to the end of the request's tokens.  A thread an entry of S; a request's chunks in order.
+// to the end of the request's tokens.  A thread W neighbouring entries of S; a request's chunks in
+// order.
+template <int W>
 __global__ void __launch_bounds__(256)
 la_states_kernel(float* __restrict__ sums, float* __restrict__ state, long state_stride,
                  const float* __restrict__ powers, const int* __restrict__ cu_tokens,
@@ -288,32 +369,74 @@ la_states_kernel(float* __restrict__ sums, float* __restrict__ state, long state
   const int n = cu_tokens[seq + 1] - cu_tokens[seq];
   const int chunks = (n + LA_C - 1) / LA_C;
   pdl_wait();
-  const int e = blockIdx.x * 256 + threadIdx.x;
+  const int e = (blockIdx.x * 256 + threadIdx.x) * W;
   if (e >= NM || chunks == 0) return;
   const float* pw = powers + (size_t)h * (LA_C + 1);
   const float whole = pw[LA_C], rest = pw[n - (chunks - 1) * LA_C];
   float* mine = state + (size_t)slots[seq] * state_stride + (size_t)h * NM + e;
-  float s = *mine;
+  float s[W];
+#pragma unroll
+  for (int w = 0; w < W; ++w) s[w] = mine[w];
   const size_t step = (size_t)heads * NM;
   float* u = sums + ((size_t)tile * heads + h) * NM + e;
   constexpr int AHEAD = 8;
   for (int k0 = 0; k0 < chunks; k0 += AHEAD) {
-    float v[AHEAD];
-#pragma unroll
-    for (int k = 0; k < AHEAD; ++k) v[k] = k0 + k < chunks ? u[(size_t)(k0 + k) * step] : 0.f;
+    float v[AHEAD][W];
 #pragma unroll
     for (int k = 0; k < AHEAD; ++k) {
       if (k0 + k < chunks) {
-        u[(size_t)(k0 + k) * step] = s;
-        s = fmaf(k0 + k == chunks - 1 ? rest : whole, s, v[k]);
+        if constexpr (W == 4) la_load4(u + (size_t)(k0 + k) * step, v[k]);
+        else v[k][0] = u[(size_t)(k0 + k) * step];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+      if (k0 + k < chunks) {
+        float* dst = u + (size_t)(k0 + k) * step;
+        if constexpr (W == 4) la_store4(dst, s);
+        else *dst = s[0];
+        const float f = k0 + k == chunks - 1 ? rest : whole;
+#pragma unroll
+        for (int w = 0; w < W; ++w) s[w] = fmaf(f, s[w], v[k][w]);
       }
     }
   }
-  *mine = s;
+#pragma unroll
+  for (int w = 0; w < W; ++w) mine[w] = s[w];
 }
 
-// VB: blocks of 64 columns of v a head has.  `o` (float32 [T, heads, M]) is written when it is
-// given; else the row's norm per head and the gate are applied and `out` is written.
+// acc[i][4 vb + e] += sum_d A[i][d] B[d][64 vb + 4 tx + e] for rows i = ty + 16 r: A [64][LA_LD] rows by
+// query token, B [inner][VB * 64 + 4] rows by the inner index.  Four inner steps at a time.
+template <int VB>
+__device__ __forceinline__ void la_rows_times(float (&acc)[4][4 * VB], const float* A, const float* B, int ty, int tx,
+                                              int inner) {
+  constexpr int LD = VB * LA_BLK + 4;
+#pragma unroll 2
+  for (int d = 0; d < inner; d += 4) {
+    float x[4][4];
+#pragma unroll
+    for (int r = 0; r < 4; ++r) *reinterpret_cast<float4*>(x[r]) = *reinterpret_cast<const float4*>(A + (ty + 16 * r) * LA_LD + d);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+#pragma unroll
+      for (int vb = 0; vb < VB; ++vb) {
+        const float4 y = *reinterpret_cast<const float4*>(B + (d + u) * LD + vb * LA_BLK + 4 * tx);
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          acc[r][4 * vb] = fmaf(x[r][u], y.x, acc[r][4 * vb]);
+          acc[r][4 * vb + 1] = fmaf(x[r][u], y.y, acc[r][4 * vb + 1]);
+          acc[r][4 * vb + 2] = fmaf(x[r][u], y.z, acc[r][4 * vb + 2]);
+          acc[r][4 * vb + 3] = fmaf(x[r][u], y.w, acc[r][4 * vb + 3]);
+        }
+      }
+    }
+  }
+}
+
+// VB: blocks of 64 columns of v a head has.  A thread owns the query tokens ty + 16 r and, of the
+// scores, the key tokens tx + 16 c; of the output, the columns 4 tx + e of every block.  `o`
+// (float32 [T, heads, M]) is written when it is given; else the row's norm per head and the gate
+// are applied and `out` is written.
 template <typename T, int VB>
 __global__ void __launch_bounds__(256)
 la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn<T> in,
@@ -321,11 +444,12 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
                     const int* __restrict__ q_tiles, const int* __restrict__ cu_tokens, int heads, int N, int M,
                     int gate_kind, float eps, float factor) {
   pdl_launch_dependents();
+  constexpr int LDB = VB * LA_BLK + 4;
   extern __shared__ __align__(16) float sm[];
-  float* Qt = sm;                              // [d][token]
-  float* Kt = Qt + LA_BLK * LA_LD;             // [d][token], later P^T [key token][query token]
-  float* Bs = Kt + LA_BLK * LA_LD;             // a block of S [d][column], later of V [token][column]
-  float* pw = Bs + LA_BLK * LA_LD;             // [LA_C + 1]
+  float* Qs = sm;                              // [token][LA_LD]: 64 columns of q, later the scores
+  float* Ks = Qs + LA_C * LA_LD;               // [token][LA_LD]: 64 columns of k
+  float* Bs = Ks + LA_C * LA_LD;               // 64 rows of S, later of v: [row][LDB]
+  float* pw = Bs + LA_BLK * LDB;               // [LA_C + 1]
   const int tile = blockIdx.x, h = blockIdx.y;
   int tok0 = 0;
   const int n_tok = la_tile_tokens(q_tiles, cu_tokens, tile, tok0);
@@ -334,92 +458,95 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
   if (n_tok == 0) return;
   const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
   float p[4][4] = {};
-  float acc[VB][4][4] = {};
+  float acc[4][4 * VB] = {};
   const float* S = states + ((size_t)tile * heads + h) * N * M;
+  const bool rows16 = (M & 3) == 0;            // rows of S begin at 16-byte boundaries
   for (int n0 = 0; n0 < N; n0 += LA_BLK) {
-    __syncthreads();
+    if (n0 > 0) __syncthreads();
+    const int inner = min(LA_BLK, N - n0);
+    // 64 rows of S travel by themselves while q and k are made ready
+    for (int i = threadIdx.x; i < LA_BLK * VB * (LA_BLK / 4); i += 256) {
+      const int d = i / (VB * (LA_BLK / 4)), m = (i - d * (VB * (LA_BLK / 4))) * 4;
+      float* dst = Bs + d * LDB + m;
+      if (rows16 && d < inner && m < M) {
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)),
+                     "l"(S + (size_t)(n0 + d) * M + m));
+      } else {
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (d < inner) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (m + e < M) x[e] = S[(size_t)(n0 + d) * M + m + e];
+        }
+        *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1], x[2], x[3]);
+      }
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+#pragma unroll 4
     for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
-      // neighbouring threads take neighbouring tokens of one piece of d: the transposed stores
-      // fall into different banks
-      const int j = i & (LA_C - 1), d = (i / LA_C) * 4;
+      const int j = i / (LA_BLK / 4), d = (i - j * (LA_BLK / 4)) * 4;
       float q4[4] = {0.f, 0.f, 0.f, 0.f}, k4[4] = {0.f, 0.f, 0.f, 0.f};
       if (j < n_tok) {
         const T* r = in.rows + (size_t)(tok0 + j) * in.ld + (size_t)h * N;
         la_qk4(in, r + in.q_off, tok0 + j, n0 + d, N, q4);
         la_qk4(in, r + in.k_off, tok0 + j, n0 + d, N, k4);
       }
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        Qt[(d + e) * LA_LD + j] = q4[e];
-        Kt[(d + e) * LA_LD + j] = k4[e] * in.key_scale;
-      }
+      *reinterpret_cast<float4*>(Qs + j * LA_LD + d) = make_float4(q4[0], q4[1], q4[2], q4[3]);
+      *reinterpret_cast<float4*>(Ks + j * LA_LD + d) =
+          make_float4(k4[0] * in.key_scale, k4[1] * in.key_scale, k4[2] * in.key_scale, k4[3] * in.key_scale);
     }
-    const int inner = min(LA_BLK, N - n0);
+    asm volatile("cp.async.wait_group 0;\n" ::);
+    __syncthreads();
+    const int steps = (inner + 3) & ~3;        // zeros beyond `inner`
+#pragma unroll 2
+    for (int d = 0; d < steps; d += 4) {
+      float x[4][4], y[4][4];
 #pragma unroll
-    for (int vb = 0; vb < VB; ++vb) {
-      if (vb > 0) __syncthreads();
-      for (int i = threadIdx.x; i < LA_BLK * (LA_BLK / 4); i += 256) {
-        const int d = i / (LA_BLK / 4), m = (i - d * (LA_BLK / 4)) * 4;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        const int mm = vb * LA_BLK + m;
-        if (d < inner && mm < M) {
-          const float* src = S + (size_t)(n0 + d) * M + mm;
-          if ((M & 3) == 0) x = *reinterpret_cast<const float4*>(src);
-          else {
-            x.x = src[0];
-            if (mm + 1 < M) x.y = src[1];
-            if (mm + 2 < M) x.z = src[2];
-            if (mm + 3 < M) x.w = src[3];
-          }
-        }
-        *reinterpret_cast<float4*>(Bs + d * LA_LD + m) = x;
+      for (int r = 0; r < 4; ++r) {
+        *reinterpret_cast<float4*>(x[r]) = *reinterpret_cast<const float4*>(Qs + (ty + 16 * r) * LA_LD + d);
+        *reinterpret_cast<float4*>(y[r]) = *reinterpret_cast<const float4*>(Ks + (tx + 16 * r) * LA_LD + d);
       }
-      __syncthreads();
-      if (vb == 0) la_mma(p, Qt, Kt, ty, tx, inner);
-      la_mma(acc[vb], Qt, Bs, ty, tx, inner);
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) p[i][j] = fmaf(x[i][u], y[j][u], p[i][j]);
     }
+    la_rows_times<VB>(acc, Qs, Bs, ty, tx, steps);
   }
   // the state's share decays by the tokens since; the chunk's own tokens by their distance
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float f = pw[min(4 * ty + i + 1, LA_C)];
+  for (int r = 0; r < 4; ++r) {
+    const float f = pw[ty + 16 * r + 1];
 #pragma unroll
-    for (int vb = 0; vb < VB; ++vb)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) acc[vb][i][j] *= f;
+    for (int e = 0; e < 4 * VB; ++e) acc[r][e] *= f;
   }
   __syncthreads();
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    float w[4];
+  for (int r = 0; r < 4; ++r)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int dist = 4 * ty + i - (4 * tx + j);
-      w[i] = dist >= 0 ? p[i][j] * pw[dist] : 0.f;
+    for (int c = 0; c < 4; ++c) {
+      const int dist = ty + 16 * r - (tx + 16 * c);
+      Qs[(ty + 16 * r) * LA_LD + tx + 16 * c] = dist >= 0 ? p[r][c] * pw[dist] : 0.f;
     }
-    *reinterpret_cast<float4*>(Kt + (4 * tx + j) * LA_LD + 4 * ty) = make_float4(w[0], w[1], w[2], w[3]);
+  const int key_steps = (n_tok + 3) & ~3;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < key_steps * VB * (LA_BLK / 4); i += 256) {
+    const int j = i / (VB * (LA_BLK / 4)), m = (i - j * (VB * (LA_BLK / 4))) * 4;
+    float v4[4] = {0.f, 0.f, 0.f, 0.f};
+    if (j < n_tok) la_v4(in, in.rows + (size_t)(tok0 + j) * in.ld + in.v_off + (size_t)h * M, m, M, v4);
+    *reinterpret_cast<float4*>(Bs + j * LDB + m) = make_float4(v4[0], v4[1], v4[2], v4[3]);
   }
+  __syncthreads();
+  la_rows_times<VB>(acc, Qs, Bs, ty, tx, key_steps);
 #pragma unroll
-  for (int vb = 0; vb < VB; ++vb) {
-    if (vb > 0) __syncthreads();
-    for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
-      const int j = i / (LA_BLK / 4), m = (i - j * (LA_BLK / 4)) * 4;
-      float v4[4] = {0.f, 0.f, 0.f, 0.f};
-      if (j < n_tok) la_v4(in, in.rows + (size_t)(tok0 + j) * in.ld + in.v_off + (size_t)h * M, vb * LA_BLK + m, M, v4);
-      *reinterpret_cast<float4*>(Bs + j * LA_LD + m) = make_float4(v4[0], v4[1], v4[2], v4[3]);
-    }
-    __syncthreads();
-    la_mma(acc[vb], Kt, Bs, ty, tx, n_tok);
-  }
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int j = 4 * ty + i;
+  for (int r = 0; r < 4; ++r) {
+    const int j = ty + 16 * r;
     float ss = 0.f;
     if (o == nullptr) {           // the sixteen threads of a row are neighbouring lanes
 #pragma unroll
-      for (int vb = 0; vb < VB; ++vb)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) ss = fmaf(acc[vb][i][e], acc[vb][i][e], ss);
+      for (int e = 0; e < 4 * VB; ++e) ss = fmaf(acc[r][e], acc[r][e], ss);
 #pragma unroll
       for (int w = 8; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
     }
@@ -428,14 +555,38 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
     const float rstd = factor * rsqrtf(ss / (float)M + eps);
 #pragma unroll
     for (int vb = 0; vb < VB; ++vb) {
+      const int m = vb * LA_BLK + 4 * tx;
+      if (o != nullptr) {
+        float* dst = o + ((size_t)t * heads + h) * M + m;
+        if (rows16) {
+          if (m < M)
+            *reinterpret_cast<float4*>(dst) =
+                make_float4(acc[r][4 * vb], acc[r][4 * vb + 1], acc[r][4 * vb + 2], acc[r][4 * vb + 3]);
+        } else {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int m = vb * LA_BLK + 4 * tx + e;
-        if (m >= M) continue;
-        if (o != nullptr) o[((size_t)t * heads + h) * M + m] = acc[vb][i][e];
-        else
-          out[(size_t)t * out_ld + (size_t)h * M + m] = from_float<T>(
-              acc[vb][i][e] * rstd * la_gate(to_float(in.rows[(size_t)t * in.ld + in.g_off + (size_t)h * M + m]), gate_kind));
+          for (int e = 0; e < 4; ++e)
+            if (m + e < M) dst[e] = acc[r][4 * vb + e];
+        }
+      } else {
+        const T* g = in.rows + (size_t)t * in.ld + in.g_off + (size_t)h * M + m;
+        T* dst = out + (size_t)t * out_ld + (size_t)h * M + m;
+        float g4[4] = {0.f, 0.f, 0.f, 0.f}, y4[4];
+        if (in.vec_gate) {
+          if (m < M) la_load4(g, g4);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (m + e < M) g4[e] = to_float(g[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y4[e] = acc[r][4 * vb + e] * rstd * la_gate(g4[e], gate_kind);
+        if (in.vec_gate) {
+          if (m < M) la_store4(dst, y4);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (m + e < M) dst[e] = from_float<T>(y4[e]);
+        }
       }
     }
   }
@@ -475,6 +626,7 @@ LaIn<T> la_in(const void* rows, int ld, int q_off, int k_off, int v_off, int g_o
   in.act = act; in.key_scale = key_scale;
   in.vec = ((ld | q_off | k_off | v_off | N | M | in.half) & 3) == 0 && ((uintptr_t)rows & 15) == 0 &&
            ((uintptr_t)cos & 15) == 0 && ((uintptr_t)sin & 15) == 0;
+  in.vec_gate = 0;
   return in;
 }
 
@@ -482,7 +634,7 @@ template <typename T, int VB>
 int la_launch_out(float* o, T* out, int out_ld, const LaIn<T>& in, const float* states, const float* powers,
                   const int* q_tiles, int n_tiles, const int* cu_tokens, int heads, int N, int M, int gate_kind,
                   float eps, float factor, cudaStream_t stream) {
-  constexpr size_t SMEM = (3 * LA_BLK * LA_LD + LA_C + 1) * sizeof(float);
+  constexpr size_t SMEM = (2 * LA_C * LA_LD + LA_BLK * (VB * LA_BLK + 4) + LA_C + 1) * sizeof(float);
   auto kernel = la_chunk_out_kernel<T, VB>;
   static bool configured = false;
   if (!configured) {
@@ -495,26 +647,54 @@ int la_launch_out(float* o, T* out, int out_ld, const LaIn<T>& in, const float* 
   return hb_check_launch();
 }
 
+template <typename T, int E>
+int la_launch_kv(float* sums, const LaIn<T>& in, const float* powers, const int* q_tiles, int n_tiles,
+                 const int* cu_tokens, int heads, int N, int M, cudaStream_t stream) {
+  constexpr int NB = 16 * E;
+  constexpr size_t SMEM = 2 * LA_C * (NB + 4) * sizeof(float);
+  auto kernel = la_chunk_kv_kernel<T, E>;
+  static bool configured = false;
+  if (!configured) {
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess)
+      return HB_LAUNCH_FAILED;
+    configured = true;
+  }
+  hb_launch(kernel, dim3(n_tiles, heads, ((N + NB - 1) / NB) * ((M + NB - 1) / NB)), dim3(256), SMEM, stream, sums, in,
+            powers, q_tiles, cu_tokens, heads, N, M);
+  return hb_check_launch();
+}
+
 }  // namespace
 
 // rows [T, ld]: q, k (heads x N), v and the gate (heads x M) at the given columns.  powers
-// [heads, 65]: the decay to the power 0..64.  o [T, heads, M] float32.
-HB_EXPORT int hb_la_scan(float* o, const void* rows, int ld, int q_off, int k_off, int v_off, const float* cos,
-                         const float* sin, int rot, int act, float key_scale, float* state, long state_stride,
-                         const float* powers, const int* cu_tokens, const int* slots, int T, int S, int heads, int N,
-                         int M, int act_dt, cudaStream_t stream) {
+// [heads, 65]: the decay to the power 0..64.  `o` null (M <= 128): norm per head and gate are
+// applied and `out` (rows out_ld apart) is written; else o [T, heads, M] float32.
+HB_EXPORT int hb_la_scan(float* o, void* out, int out_ld, const void* rows, int ld, int q_off, int k_off, int v_off,
+                         int g_off, const float* cos, const float* sin, int rot, int act, float key_scale,
+                         float* state, long state_stride, const float* powers, const int* cu_tokens,
+                         const int* slots, int T, int S, int heads, int N, int M, int gate_kind, float eps,
+                         float factor, int act_dt, cudaStream_t stream) {
   if (T <= 0 || S <= 0) return HB_OK;
-  if (N <= 0 || N > 256 || M <= 0 || heads <= 0) return HB_BAD_ARGUMENT;
-  const dim3 grid((M + LA_COLS - 1) / LA_COLS, heads, S);
-#define HB_LA_SCAN(TA, R)                                                                                   \
-  hb_launch(la_scan_kernel<TA, R>, grid, dim3(LA_COLS * LA_PARTS), 0, stream, o,                              \
-            la_in<TA>(rows, ld, q_off, k_off, v_off, 0, cos, sin, rot, act, key_scale, N, M), state,          \
-            state_stride, powers, cu_tokens, slots, heads, N, M)
+  if (N <= 0 || N > 256 || M <= 0 || heads <= 0 || (o == nullptr && M > 128)) return HB_BAD_ARGUMENT;
+  const int vec = M <= 32 ? 1 : M <= 64 ? 2 : 4;
+  const dim3 grid((M + 32 * vec - 1) / (32 * vec), heads, S);
+  const int vec_state = M % vec == 0 && state_stride % vec == 0 && ((uintptr_t)state & (4 * vec - 1)) == 0;
+#define HB_LA_SCAN(TA, R, V)                                                                                \
+  hb_launch(la_scan_kernel<TA, R, V>, grid, dim3(32 * LA_PARTS), 0, stream, o, (TA*)out, out_ld,              \
+            la_in<TA>(rows, ld, q_off, k_off, v_off, g_off, cos, sin, rot, act, key_scale, N, M), state,      \
+            state_stride, powers, cu_tokens, slots, heads, N, M, vec_state, gate_kind, eps, factor)
+#define HB_LA_SCAN_V(TA, V)                                                                                 \
+  do {                                                                                                       \
+    if (N <= 32) HB_LA_SCAN(TA, 4, V);                                                                       \
+    else if (N <= 64) HB_LA_SCAN(TA, 8, V);                                                                  \
+    else if (N <= 128) HB_LA_SCAN(TA, 16, V);                                                                \
+    else HB_LA_SCAN(TA, 32, V);                                                                              \
+  } while (0)
   HB_DISPATCH_DTYPE(act_dt, TA,
-    if (N <= 32) HB_LA_SCAN(TA, 4);
-    else if (N <= 64) HB_LA_SCAN(TA, 8);
-    else if (N <= 128) HB_LA_SCAN(TA, 16);
-    else HB_LA_SCAN(TA, 32));
+    if (vec == 1) HB_LA_SCAN_V(TA, 1);
+    else if (vec == 2) HB_LA_SCAN_V(TA, 2);
+    else HB_LA_SCAN_V(TA, 4));
+#undef HB_LA_SCAN_V
 #undef HB_LA_SCAN
   return hb_check_launch();
 }
@@ -527,16 +707,21 @@ HB_EXPORT int hb_la_chunked(float* o, void* out, int out_ld, float* sums, const 
                             const int* q_tiles, int n_tiles, const int* cu_tokens, const int* slots, int S, int heads,
                             int N, int M, int gate_kind, float eps, float factor, int act_dt, cudaStream_t stream) {
   if (n_tiles <= 0 || S <= 0) return HB_OK;
-  if (N <= 0 || N > 256 || M <= 0 || M > 256 || heads <= 0) return HB_BAD_ARGUMENT;
-  const int nb = (N + LA_BLK - 1) / LA_BLK, vb = (M + LA_BLK - 1) / LA_BLK;
-  constexpr size_t SMEM_KV = 2 * LA_C * LA_LD * sizeof(float);
+  if (N <= 0 || N > 256 || M <= 0 || M > 256 || heads <= 0 || ((uintptr_t)sums & 15)) return HB_BAD_ARGUMENT;
   HB_DISPATCH_DTYPE(act_dt, TA, {
-    const LaIn<TA> in = la_in<TA>(rows, ld, q_off, k_off, v_off, g_off, cos, sin, rot, act, key_scale, N, M);
-    hb_launch(la_chunk_kv_kernel<TA>, dim3(n_tiles, heads, nb * vb), dim3(256), SMEM_KV, stream, sums, in, powers,
-              q_tiles, cu_tokens, heads, N, M);
-    hb_launch(la_states_kernel, dim3((N * M + 255) / 256, heads, S), dim3(256), 0, stream, sums, state, state_stride,
-              powers, cu_tokens, slots, heads, N * M);
-    int st;
+    LaIn<TA> in = la_in<TA>(rows, ld, q_off, k_off, v_off, g_off, cos, sin, rot, act, key_scale, N, M);
+    in.vec_gate = ((ld | g_off | M | out_ld) & 3) == 0 && (((uintptr_t)rows | (uintptr_t)out) & 15) == 0;
+    int st = N > 64 || M > 64 ? la_launch_kv<TA, 8>(sums, in, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, stream)
+                              : la_launch_kv<TA, 4>(sums, in, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, stream);
+    if (st != HB_OK) return st;
+    const int NM = N * M;
+    if (NM % 4 == 0)
+      hb_launch(la_states_kernel<4>, dim3((NM / 4 + 255) / 256, heads, S), dim3(256), 0, stream, sums, state,
+                state_stride, powers, cu_tokens, slots, heads, NM);
+    else
+      hb_launch(la_states_kernel<1>, dim3((NM + 255) / 256, heads, S), dim3(256), 0, stream, sums, state, state_stride,
+                powers, cu_tokens, slots, heads, NM);
+    const int vb = (M + LA_BLK - 1) / LA_BLK;
     if (vb == 1) st = la_launch_out<TA, 1>(o, (TA*)out, out_ld, in, sums, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, gate_kind, eps, factor, stream);
     else if (vb == 2) st = la_launch_out<TA, 2>(o, (TA*)out, out_ld, in, sums, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, gate_kind, eps, factor, stream);
     else st = la_launch_out<TA, 4>(o, (TA*)out, out_ld, in, sums, powers, q_tiles, n_tiles, cu_tokens, heads, N, M, gate_kind, eps, factor, stream);

@@ -2124,13 +2124,19 @@ def linear_attention(ctx, rows: torch.Tensor, offsets, state: torch.Tensor, deca
         if o is None:
             return
     else:
-        o = torch.empty((T, heads * dv), dtype=torch.float32, device=rows.device)
+        fused = norm == "head" and dv <= 128
+        if not fused:
+            o = torch.empty((T, heads * dv), dtype=torch.float32, device=rows.device)
         f = _fn("linear_attention", "hb_la_scan",
-                [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p,
-                 _LONG, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
-        _run(f(_p(o), _p(rows), rows.shape[1], q_off, k_off, v_off, _p(cos), _p(sin), rot, act, float(key_scale),
-               _p(state), state.stride(0), _p(decay_powers), _p(ctx.cu_tokens), _p(ctx.slots), T, ctx.num_seqs,
-               heads, dk, dv, _dt(rows.dtype), _stream()), "linear_attention_scan")
+                [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+                 c_float, c_void_p, _LONG, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                 c_float, c_float, c_int, c_void_p])
+        _run(f(_p(o), _p(out), out.stride(0), _p(rows), rows.shape[1], q_off, k_off, v_off, g_off, _p(cos), _p(sin),
+               rot, act, float(key_scale), _p(state), state.stride(0), _p(decay_powers), _p(ctx.cu_tokens),
+               _p(ctx.slots), T, ctx.num_seqs, heads, dk, dv, gk, float(eps), float(factor), _dt(rows.dtype),
+               _stream()), "linear_attention_scan")
+        if fused:
+            return
     f = _fn("linear_attention", "hb_la_gate_norm",
             [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
              c_int, c_void_p])
