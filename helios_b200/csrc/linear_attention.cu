@@ -406,8 +406,9 @@ la_states_kernel(float* __restrict__ sums, float* __restrict__ state, long state
 }
 
 // acc[i][4 vb + e] += sum_d A[i][d] B[d][64 vb + 4 tx + e] for rows i = ty + 16 r: A [64][LA_LD] rows by
-// query token, B [inner][VB * 64 + 4] rows by the inner index.  Four inner steps at a time.
-template <int VB>
+// query token, B [inner][VB * 64 + 4] rows by the inner index.  Four inner steps at a time.  FROM: only
+// the row groups r >= FROM.
+template <int VB, int FROM = 0>
 __device__ __forceinline__ void la_rows_times(float (&acc)[4][4 * VB], const float* A, const float* B, int ty, int tx,
                                               int inner) {
   constexpr int LD = VB * LA_BLK + 4;
@@ -415,14 +416,14 @@ __device__ __forceinline__ void la_rows_times(float (&acc)[4][4 * VB], const flo
   for (int d = 0; d < inner; d += 4) {
     float x[4][4];
 #pragma unroll
-    for (int r = 0; r < 4; ++r) *reinterpret_cast<float4*>(x[r]) = *reinterpret_cast<const float4*>(A + (ty + 16 * r) * LA_LD + d);
+    for (int r = FROM; r < 4; ++r) *reinterpret_cast<float4*>(x[r]) = *reinterpret_cast<const float4*>(A + (ty + 16 * r) * LA_LD + d);
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
 #pragma unroll
       for (int vb = 0; vb < VB; ++vb) {
         const float4 y = *reinterpret_cast<const float4*>(B + (d + u) * LD + vb * LA_BLK + 4 * tx);
 #pragma unroll
-        for (int r = 0; r < 4; ++r) {
+        for (int r = FROM; r < 4; ++r) {
           acc[r][4 * vb] = fmaf(x[r][u], y.x, acc[r][4 * vb]);
           acc[r][4 * vb + 1] = fmaf(x[r][u], y.y, acc[r][4 * vb + 1]);
           acc[r][4 * vb + 2] = fmaf(x[r][u], y.z, acc[r][4 * vb + 2]);
@@ -511,7 +512,7 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-          for (int j = 0; j < 4; ++j) p[i][j] = fmaf(x[i][u], y[j][u], p[i][j]);
+          for (int j = 0; j <= i; ++j) p[i][j] = fmaf(x[i][u], y[j][u], p[i][j]);     // later keys are not seen
     }
     la_rows_times<VB>(acc, Qs, Bs, ty, tx, steps);
   }
@@ -539,7 +540,11 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
     *reinterpret_cast<float4*>(Bs + j * LDB + m) = make_float4(v4[0], v4[1], v4[2], v4[3]);
   }
   __syncthreads();
-  la_rows_times<VB>(acc, Qs, Bs, ty, tx, key_steps);
+  // sixteen key tokens at a time, for the query tokens that are not all before them
+  la_rows_times<VB, 0>(acc, Qs, Bs, ty, tx, min(16, key_steps));
+  if (key_steps > 16) la_rows_times<VB, 1>(acc, Qs + 16, Bs + 16 * LDB, ty, tx, min(16, key_steps - 16));
+  if (key_steps > 32) la_rows_times<VB, 2>(acc, Qs + 32, Bs + 32 * LDB, ty, tx, min(16, key_steps - 32));
+  if (key_steps > 48) la_rows_times<VB, 3>(acc, Qs + 48, Bs + 48 * LDB, ty, tx, key_steps - 48);
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
     const int j = ty + 16 * r;

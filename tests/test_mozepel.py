@@ -758,3 +758,79 @@ def test_a_pool_too_small_for_all_requests_gives_pages_from_one_to_the_next(mz_f
                 max_num_batched_tokens=32, max_model_len=128, watermark=0.0)
     got = [o.token_ids for o in tight.generate(prompt_token_ids=prompts, sampling_params=SamplingParams(max_tokens=20))]
     assert got == want
+
+
+# ====================================================================== configurations drawn at random
+def draw_config(seed):
+    """Sizes, head counts, layer order, windows, blocks and constants at random."""
+    import random
+    rng = random.Random(seed)
+    dims = (8, 16, 24, 32, 48, 64, 80, 96, 128, 160, 192, 256)
+
+    def decay(n):
+        return [rng.choice([0.0, 0.3, 0.8, 0.95, 0.99, 0.999, 1.0]) if rng.random() < 0.3 else
+                round(1 - 2.0 ** -rng.uniform(2, 10), 6) for _ in range(n)]
+
+    def scaling():
+        return (rng.choice([2.0, 8.0]), 1.0, rng.choice([2.0, 4.0]), rng.choice([32, 256])) if rng.random() < 0.5 else None
+
+    def ret():
+        d = rng.choice(dims)
+        h = rng.randint(1, 6)
+        return _ret(h, d, rng.choice(dims), decay(h), 2 * rng.randint(1, d // 2), rng.choice([100.0, 1e4, 1e6]))
+
+    def par():
+        d, vd = rng.choice(dims), rng.choice(dims)
+        kv = rng.choice([1, 2, 3])
+        rh = rng.randint(1, 5)
+        return _par(kv * rng.choice([1, 2, 4, 5, 8]), kv, d, vd, round(rng.uniform(0.5, 2.0) * d ** -0.5, 4),
+                    rng.choice([1, 7, 16, 33, 64, 130]), rng.choice([0, 1, 3, 8, 16, 24, 40]), 2 * rng.randint(1, d // 2),
+                    rng.choice([50.0, 5e3, 5e5]), rng.choice([0, 1, 2, 3, 4, 6]), round(rng.uniform(0.2, 1.5), 2),
+                    round(rng.uniform(0.2, 1.5), 2), rh, rng.choice(dims), rng.choice(dims), decay(rh), scaling())
+
+    layers = []
+    for i in range(rng.randint(2, 4)):
+        own = [j for j, l in enumerate(layers) if not isinstance(l, int)]
+        if own and rng.random() < 0.35:
+            layers.append(rng.choice(own))
+        else:
+            layers.append(((ret if rng.random() < 0.45 else par)(), rng.choice([None, 24, 64, 136])))
+    return _model(rng.randint(40, 700), 8 * rng.randint(3, 40), rng.choice([1e-5, 1e-6, 3e-6]),
+                  round(rng.uniform(0.8, 3.0), 2), layers), rng
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("seed", range(8))
+def test_a_random_configuration_matches_the_plain_implementation(tmp_path, seed, dtype):
+    compare_random(tmp_path, seed, dtype)
+
+
+def compare_random(tmp_path, seed, dtype, lengths=(70, 23, 150)):
+    from safetensors.torch import save_file
+    from helios_b200.weights import write_model_folder
+
+    cfg, rng = draw_config(seed)
+    folder = write_model_folder(tmp_path / "m", cfg, seed)
+    _cfg, weights = read_folder(folder)
+    weights = _lively(weights)
+    save_file(weights, str(folder / "model.safetensors"))
+    reqs = _requests(cfg, lengths, 1000 + seed)
+    plain = _plain(cfg, weights, reqs)
+    tb = tu.TraceBuilder()
+    tu.mixed(tb, reqs, seed=seed, max_live=2, decode_tail=12, portion_choices=(2, 3, 9, 34, 70))
+    core = _core(folder, dtype, tb.live_tokens_peak, page_size=rng.choice([16, 16, 8, 32]), max_slots=2)
+    got = tu.run_in_process(core, tb)
+    if dtype == "float32":
+        tu.check(tb, got, plain, dtype, f"seed {seed}")
+        return
+    # bfloat16: a norm per head makes of a sum near 0 whatever rounding left of it, so single
+    # rows may stand further off; a wrong key or state would move most of them
+    rel = []
+    for step, rows in tb.rows.items():
+        want = torch.stack([plain[rid][pos] for rid, pos in rows])
+        g = torch.from_numpy(got[step]).double()
+        assert torch.isfinite(g).all()
+        rel += ((g - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()).tolist()
+    rel = torch.tensor(rel)
+    assert float(rel.median()) < 0.02 and float((rel > 0.06).double().mean()) < 0.05, (float(rel.median()), float(rel.max()))
