@@ -621,6 +621,51 @@ __global__ void la_gate_norm_kernel(T* __restrict__ out, int out_ld, const float
   }
 }
 
+// The same with four neighbouring values at a time and the row held in registers between the
+// passes: widths that are multiples of 4 up to 4 x 256 x GROUPS.
+template <typename T, int GROUPS>
+__global__ void __launch_bounds__(256)
+la_gate_norm_vec_kernel(T* __restrict__ out, int out_ld, const float* __restrict__ o, const T* __restrict__ gate,
+                        int gate_ld, const float* __restrict__ weight, int parts, int width, int gate_kind, float eps,
+                        float factor) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const int t = blockIdx.x / parts, part = blockIdx.x - t * parts;
+  const float* x = o + (size_t)blockIdx.x * width;
+  const T* g = gate + (size_t)t * gate_ld + (size_t)part * width;
+  T* y = out + (size_t)t * out_ld + (size_t)part * width;
+  float v[GROUPS][4], gv[GROUPS][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < GROUPS; ++k) {
+    const int c = (k * blockDim.x + threadIdx.x) * 4;
+    if (c < width) {
+      la_load4(x + c, v[k]);
+      la_load4(g + c, gv[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < GROUPS; ++k) {
+    if ((k * blockDim.x + threadIdx.x) * 4 < width) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss = fmaf(v[k][e], v[k][e], ss);
+    }
+  }
+  const float rstd = factor * rsqrtf(block_sum(ss, scratch) / (float)width + eps);
+#pragma unroll
+  for (int k = 0; k < GROUPS; ++k) {
+    const int c = (k * blockDim.x + threadIdx.x) * 4;
+    if (c < width) {
+      float w[4] = {1.f, 1.f, 1.f, 1.f};
+      if (weight) la_load4(weight + c, w);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[k][e] *= rstd * w[e] * la_gate(gv[k][e], gate_kind);
+      la_store4(y + c, v[k]);
+    }
+  }
+}
+
 template <typename T>
 LaIn<T> la_in(const void* rows, int ld, int q_off, int k_off, int v_off, int g_off, const float* cos,
               const float* sin, int rot, int act, float key_scale, int N, int M) {
@@ -742,6 +787,21 @@ HB_EXPORT int hb_la_gate_norm(void* out, int out_ld, const float* o, const void*
   if (T <= 0) return HB_OK;
   if (parts <= 0 || width <= 0 || (weight != nullptr && parts != 1)) return HB_BAD_ARGUMENT;
   int threads = 32;
+  if (width % 4 == 0 && width <= 4096 && ((gate_ld | out_ld) & 3) == 0 &&
+      (((uintptr_t)out | (uintptr_t)o | (uintptr_t)weight) & 15) == 0 &&
+      ((uintptr_t)gate & (act_dt == HB_F32 ? 15 : 7)) == 0) {
+    while (threads < 256 && threads * 4 < width) threads *= 2;
+    const int groups = (width + 4 * threads - 1) / (4 * threads);
+#define HB_GATE_NORM(G)                                                                                       \
+    hb_launch(la_gate_norm_vec_kernel<TA, G>, dim3((unsigned)(T * parts)), dim3(threads), 0, stream, (TA*)out,  \
+              out_ld, o, (const TA*)gate, gate_ld, weight, parts, width, gate_kind, eps, factor)
+    HB_DISPATCH_DTYPE(act_dt, TA,
+      if (groups == 1) HB_GATE_NORM(1);
+      else if (groups == 2) HB_GATE_NORM(2);
+      else HB_GATE_NORM(4));
+#undef HB_GATE_NORM
+    return hb_check_launch();
+  }
   while (threads < 256 && threads * 2 < width) threads *= 2;
   HB_DISPATCH_DTYPE(act_dt, TA,
     hb_launch(la_gate_norm_kernel<TA>, dim3((unsigned)(T * parts)), dim3(threads), 0, stream, (TA*)out, out_ld, o,

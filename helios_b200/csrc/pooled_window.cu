@@ -334,7 +334,7 @@ pool_blocks_kernel(T* __restrict__ k_pooled, T* __restrict__ v_pooled, const int
     float sum[W];
 #pragma unroll
     for (int w = 0; w < W; ++w) sum[w] = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int j = 0; j < pool; ++j) {
       const T* at = src + (size_t)(j < POOL_ROWS ? rows[j] : row_of(first + j)) * width;
       if constexpr (W == 8) {
@@ -400,7 +400,7 @@ HB_EXPORT int hb_pool_blocks(void* k_pooled, void* v_pooled, const int* pooled_t
                    (((uintptr_t)k_pooled | (uintptr_t)v_pooled | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) == 0;
   if (vec) {
     using B = __nv_bfloat16;
-    hb_launch(pool_blocks_kernel<B, 8>, dim3(T), dim3(256), 0, stream, (B*)k_pooled, (B*)v_pooled, pooled_table,
+    hb_launch(pool_blocks_kernel<B, 8>, dim3(T), dim3(128), 0, stream, (B*)k_pooled, (B*)v_pooled, pooled_table,
               pooled_stride, (const B*)k_pages, (const B*)v_pages, block_table, bt_stride, positions, seq_of_token, nkv,
               hd, vd, page_size, pool);
     return hb_check_launch();
