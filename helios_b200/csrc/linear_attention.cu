@@ -129,6 +129,66 @@ __device__ __forceinline__ void la_v4(const LaIn<T>& in, const T* x, int d, int 
   }
 }
 
+// Pieces of four columns for a thread's B places of a tile of tokens, all loads issued before the
+// first use (rows that read four columns at once only: `vec`).  Place b is the token `j[b]` of the
+// tile (clamped to a live one) and the columns from d[b] on (clamped to the head's first); `ok[b]`: it is
+// a live one, else its values are zeros.
+template <int B>
+struct LaPlaces {
+  int j[B], d[B];
+  bool ok[B];
+  // i0 + 256 b: place by place, `per_row` pieces of four columns a token, columns from n0 on
+  __device__ __forceinline__ LaPlaces(int i0, int per_row, int n0, int n_tok, int N) {
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      const int i = i0 + 256 * b, jj = i / per_row, dd = n0 + (i - jj * per_row) * 4;
+      ok[b] = jj < n_tok && dd < N;
+      j[b] = ok[b] ? jj : 0;
+      d[b] = ok[b] ? dd : 0;
+    }
+  }
+};
+
+// The cosines and sines of the places' columns (of columns beyond the rotation: those of the first).
+template <typename T, int B>
+__device__ __forceinline__ void la_angles(const LaIn<T>& in, int tok0, const LaPlaces<B>& at, float (&c)[B][4],
+                                          float (&s)[B][4]) {
+#pragma unroll
+  for (int b = 0; b < B; ++b) {
+    const int d = at.d[b], p = d < in.half ? d : d < 2 * in.half ? d - in.half : 0;
+    la_load4(in.cos + (size_t)(tok0 + at.j[b]) * in.half + p, c[b]);
+    la_load4(in.sin + (size_t)(tok0 + at.j[b]) * in.half + p, s[b]);
+  }
+}
+
+// f: the columns as read, o: their partners in the rotation.
+template <typename T, int B>
+__device__ __forceinline__ void la_fetch(const LaIn<T>& in, const T* x, int tok0, const LaPlaces<B>& at,
+                                         float (&f)[B][4], float (&o)[B][4]) {
+#pragma unroll
+  for (int b = 0; b < B; ++b) {
+    const T* r = x + (size_t)(tok0 + at.j[b]) * in.ld;
+    const int d = at.d[b];
+    la_load4(r + d, f[b]);
+    if (in.half > 0) la_load4(r + (d < in.half ? d + in.half : d < 2 * in.half ? d - in.half : d), o[b]);
+  }
+}
+
+template <typename T, int B>
+__device__ __forceinline__ void la_turn(const LaIn<T>& in, const LaPlaces<B>& at, float (&f)[B][4],
+                                        const float (&o)[B][4], const float (&c)[B][4], const float (&s)[B][4]) {
+#pragma unroll
+  for (int b = 0; b < B; ++b) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (in.act == LA_SILU) f[b][e] = la_silu(f[b][e]);
+      if (in.half > 0 && at.d[b] < 2 * in.half)
+        f[b][e] = f[b][e] * c[b][e] + (at.d[b] < in.half ? -o[b][e] : o[b][e]) * s[b][e];
+      if (!at.ok[b]) f[b][e] = 0.f;
+    }
+  }
+}
+
 __device__ __forceinline__ float la_gate(float g, int kind) {
   const float s = 1.f / (1.f + expf(-g));
   return kind == 0 ? g * s : s;              // silu | sigmoid
@@ -297,16 +357,44 @@ la_chunk_kv_kernel(float* __restrict__ sums, LaIn<T> in, const float* __restrict
   pdl_wait();
   if (n_tok == 0) return;
   const float* pw = powers + (size_t)h * (LA_C + 1);
-#pragma unroll 4
-  for (int i = threadIdx.x; i < n_tok * (NB / 4); i += 256) {
-    const int j = i / (NB / 4), d = (i - j * (NB / 4)) * 4;
-    float k4[4], v4[4];
-    const T* r = in.rows + (size_t)(tok0 + j) * in.ld;
-    la_qk4(in, r + in.k_off + (size_t)h * N, tok0 + j, n0 + d, N, k4);
-    la_v4(in, r + in.v_off + (size_t)h * M, m0 + d, M, v4);
-    const float f = in.key_scale * pw[n_tok - 1 - j];
-    *reinterpret_cast<float4*>(Ks + j * LD + d) = make_float4(k4[0] * f, k4[1] * f, k4[2] * f, k4[3] * f);
-    *reinterpret_cast<float4*>(Vs + j * LD + d) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+  if (in.vec) {
+    constexpr int B = 4;                     // whole passes: 64 x NB / 4 places are a multiple of 256 B
+    static_assert(LA_C * (NB / 4) % (256 * B) == 0, "places of the tile");
+    const T* kx = in.rows + in.k_off + (size_t)h * N;
+    const T* vx = in.rows + in.v_off + (size_t)h * M;
+    for (int i = threadIdx.x; i < n_tok * (NB / 4); i += 256 * B) {
+      float f[B][4], o[B][4], c[B][4], sn[B][4], v[B][4];
+      const LaPlaces<B> at(i, NB / 4, n0, n_tok, N), av(i, NB / 4, m0, n_tok, M);
+      la_fetch(in, kx, tok0, at, f, o);
+      if (in.half > 0) la_angles(in, tok0, at, c, sn);
+#pragma unroll
+      for (int b = 0; b < B; ++b) la_load4(vx + (size_t)(tok0 + av.j[b]) * in.ld + av.d[b], v[b]);
+      la_turn(in, at, f, o, c, sn);
+#pragma unroll
+      for (int b = 0; b < B; ++b) {
+        const int p = i + 256 * b, j = p / (NB / 4), d = (p - j * (NB / 4)) * 4;
+        if (j >= n_tok) continue;
+        const float w = in.key_scale * pw[n_tok - 1 - j];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (in.act == LA_SILU) v[b][e] = la_silu(v[b][e]);
+          if (!av.ok[b]) v[b][e] = 0.f;
+        }
+        *reinterpret_cast<float4*>(Ks + j * LD + d) = make_float4(f[b][0] * w, f[b][1] * w, f[b][2] * w, f[b][3] * w);
+        *reinterpret_cast<float4*>(Vs + j * LD + d) = make_float4(v[b][0], v[b][1], v[b][2], v[b][3]);
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < n_tok * (NB / 4); i += 256) {
+      const int j = i / (NB / 4), d = (i - j * (NB / 4)) * 4;
+      float k4[4], v4[4];
+      const T* r = in.rows + (size_t)(tok0 + j) * in.ld;
+      la_qk4(in, r + in.k_off + (size_t)h * N, tok0 + j, n0 + d, N, k4);
+      la_v4(in, r + in.v_off + (size_t)h * M, m0 + d, M, v4);
+      const float f = in.key_scale * pw[n_tok - 1 - j];
+      *reinterpret_cast<float4*>(Ks + j * LD + d) = make_float4(k4[0] * f, k4[1] * f, k4[2] * f, k4[3] * f);
+      *reinterpret_cast<float4*>(Vs + j * LD + d) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+    }
   }
   __syncthreads();
   // rows 4 ty + 64 g + i, columns 4 tx + 64 g' + i': groups of four neighbours, 64 apart
@@ -483,18 +571,39 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
       }
     }
     asm volatile("cp.async.commit_group;\n" ::);
-#pragma unroll 4
-    for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
-      const int j = i / (LA_BLK / 4), d = (i - j * (LA_BLK / 4)) * 4;
-      float q4[4] = {0.f, 0.f, 0.f, 0.f}, k4[4] = {0.f, 0.f, 0.f, 0.f};
-      if (j < n_tok) {
-        const T* r = in.rows + (size_t)(tok0 + j) * in.ld + (size_t)h * N;
-        la_qk4(in, r + in.q_off, tok0 + j, n0 + d, N, q4);
-        la_qk4(in, r + in.k_off, tok0 + j, n0 + d, N, k4);
+    if (in.vec) {
+      constexpr int B = 2;
+      const T* x = in.rows + (size_t)h * N;
+#pragma unroll 1
+      for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256 * B) {
+        float q[B][4], qo[B][4], k[B][4], ko[B][4], c[B][4], sn[B][4];
+        const LaPlaces<B> at(i, LA_BLK / 4, n0, n_tok, N);
+        la_fetch(in, x + in.q_off, tok0, at, q, qo);
+        la_fetch(in, x + in.k_off, tok0, at, k, ko);
+        if (in.half > 0) la_angles(in, tok0, at, c, sn);
+        la_turn(in, at, q, qo, c, sn);
+        la_turn(in, at, k, ko, c, sn);
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+          const int pl = i + 256 * b, j = pl / (LA_BLK / 4), d = (pl - j * (LA_BLK / 4)) * 4;
+          *reinterpret_cast<float4*>(Qs + j * LA_LD + d) = make_float4(q[b][0], q[b][1], q[b][2], q[b][3]);
+          *reinterpret_cast<float4*>(Ks + j * LA_LD + d) = make_float4(
+              k[b][0] * in.key_scale, k[b][1] * in.key_scale, k[b][2] * in.key_scale, k[b][3] * in.key_scale);
+        }
       }
-      *reinterpret_cast<float4*>(Qs + j * LA_LD + d) = make_float4(q4[0], q4[1], q4[2], q4[3]);
-      *reinterpret_cast<float4*>(Ks + j * LA_LD + d) =
-          make_float4(k4[0] * in.key_scale, k4[1] * in.key_scale, k4[2] * in.key_scale, k4[3] * in.key_scale);
+    } else {
+      for (int i = threadIdx.x; i < LA_C * (LA_BLK / 4); i += 256) {
+        const int j = i / (LA_BLK / 4), d = (i - j * (LA_BLK / 4)) * 4;
+        float q4[4] = {0.f, 0.f, 0.f, 0.f}, k4[4] = {0.f, 0.f, 0.f, 0.f};
+        if (j < n_tok) {
+          const T* r = in.rows + (size_t)(tok0 + j) * in.ld + (size_t)h * N;
+          la_qk4(in, r + in.q_off, tok0 + j, n0 + d, N, q4);
+          la_qk4(in, r + in.k_off, tok0 + j, n0 + d, N, k4);
+        }
+        *reinterpret_cast<float4*>(Qs + j * LA_LD + d) = make_float4(q4[0], q4[1], q4[2], q4[3]);
+        *reinterpret_cast<float4*>(Ks + j * LA_LD + d) =
+            make_float4(k4[0] * in.key_scale, k4[1] * in.key_scale, k4[2] * in.key_scale, k4[3] * in.key_scale);
+      }
     }
     asm volatile("cp.async.wait_group 0;\n" ::);
     __syncthreads();
@@ -532,12 +641,32 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
       Qs[(ty + 16 * r) * LA_LD + tx + 16 * c] = dist >= 0 ? p[r][c] * pw[dist] : 0.f;
     }
   const int key_steps = (n_tok + 3) & ~3;
-#pragma unroll 4
-  for (int i = threadIdx.x; i < key_steps * VB * (LA_BLK / 4); i += 256) {
-    const int j = i / (VB * (LA_BLK / 4)), m = (i - j * (VB * (LA_BLK / 4))) * 4;
-    float v4[4] = {0.f, 0.f, 0.f, 0.f};
-    if (j < n_tok) la_v4(in, in.rows + (size_t)(tok0 + j) * in.ld + in.v_off + (size_t)h * M, m, M, v4);
-    *reinterpret_cast<float4*>(Bs + j * LDB + m) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+  if (in.vec) {
+    constexpr int B = 4, PER = VB * (LA_BLK / 4);
+    const T* vx = in.rows + in.v_off + (size_t)h * M;
+    for (int i = threadIdx.x; i < key_steps * PER; i += 256 * B) {
+      float v[B][4];
+      const LaPlaces<B> at(i, PER, 0, n_tok, M);
+#pragma unroll
+      for (int b = 0; b < B; ++b) la_load4(vx + (size_t)(tok0 + at.j[b]) * in.ld + at.d[b], v[b]);
+#pragma unroll
+      for (int b = 0; b < B; ++b) {
+        const int pl = i + 256 * b, j = pl / PER, m = (pl - j * PER) * 4;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (in.act == LA_SILU) v[b][e] = la_silu(v[b][e]);
+          if (!at.ok[b]) v[b][e] = 0.f;
+        }
+        if (j < key_steps) *reinterpret_cast<float4*>(Bs + j * LDB + m) = make_float4(v[b][0], v[b][1], v[b][2], v[b][3]);
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < key_steps * VB * (LA_BLK / 4); i += 256) {
+      const int j = i / (VB * (LA_BLK / 4)), m = (i - j * (VB * (LA_BLK / 4))) * 4;
+      float v4[4] = {0.f, 0.f, 0.f, 0.f};
+      if (j < n_tok) la_v4(in, in.rows + (size_t)(tok0 + j) * in.ld + in.v_off + (size_t)h * M, m, M, v4);
+      *reinterpret_cast<float4*>(Bs + j * LDB + m) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+    }
   }
   __syncthreads();
   // sixteen key tokens at a time, for the query tokens that are not all before them
