@@ -433,7 +433,7 @@ def mozepel_configs(size):
                  "mask": {"size": 1024, "pool": 16},
                  "rot": {"dims": hd // 2, "base": 500000.0,
                          "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
-        "left_scale": 0.6, "right": {"heads": heads, "dim": hd, "vdim": hd, "decay": decay}, "right_scale": 0.5}}
+        "left_scale": 0.7, "right": {"heads": heads, "dim": hd, "vdim": hd, "decay": decay}, "right_scale": 0.4}}
     mz = {"architecture": "Mozepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
           "layers": [ret, ret, par, ret, ret, par]}
     rot = {"base": 10000.0, "dims": hd // 2, "scaling": {"factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 4096}}

@@ -511,7 +511,7 @@ def _pooled_cases(W, P, n, decode):
 @pytest.mark.parametrize("decode", [True, False])
 @pytest.mark.parametrize("dtype,hd,vd,page,W,P,G", [
     ("float32", 40, 24, 16, 37, 6, 2), ("float32", 16, 16, 8, 1, 1, 1), ("bfloat16", 64, 64, 16, 37, 5, 2),
-    ("bfloat16", 128, 128, 16, 40, 16, 4), ("bfloat16", 128, 256, 16, 33, 8, 4), ("bfloat16", 64, 128, 32, 130, 3, 1),
+    ("bfloat16", 128, 128, 16, 44, 16, 4), ("bfloat16", 128, 256, 16, 33, 8, 4), ("bfloat16", 64, 128, 32, 130, 3, 1),
     ("bfloat16", 96, 80, 16, 20, 12, 3), ("bfloat16", 32, 32, 8, 9, 14, 8), ("bfloat16", 128, 64, 16, 1, 1, 5),
     ("bfloat16", 256, 256, 16, 64, 32, 2), ("bfloat16", 192, 128, 24, 50, 2, 16), ("bfloat16", 128, 128, 16, 64, 0, 4),
     ("bfloat16", 20, 36, 16, 30, 4, 2)])
