@@ -177,10 +177,15 @@ decode_attention_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
       for (int it = 0; it < DEC_TILE * CH / 32; ++it) {
         const int idx = it * 32 + lane;
         const int row = idx / CH, c = idx - row * CH;
-        const int bytes = (row < rows_valid && row >= rows_skipped && c * 8 < hd) ? 16 : 0;
-        const size_t at = bytes ? (row0 + row) * hd + c * 8 : 0;
-        cp_async16(k_dst + row * RS + c * 8, k_src + at, bytes);
-        if constexpr (!POOLED) cp_async16(v_dst + row * RS + c * 8, v_src + at, bytes);
+        if constexpr (!POOLED) {         // the tile is one contiguous stretch of the cache
+          const int bytes = (row < rows_valid && row >= rows_skipped) ? 16 : 0;
+          const size_t base = row0 * HD + lane * 8;
+          cp_async16(k_dst + row * RS + c * 8, k_pages + base + it * 256, bytes);
+          cp_async16(v_dst + row * RS + c * 8, v_pages + base + it * 256, bytes);
+        } else {
+          const int bytes = (row < rows_valid && row >= rows_skipped && c * 8 < hd) ? 16 : 0;
+          cp_async16(k_dst + row * RS + c * 8, k_src + (bytes ? (row0 + row) * hd + c * 8 : 0), bytes);
+        }
       }
       if constexpr (POOLED) {
 #pragma unroll
@@ -206,10 +211,15 @@ decode_attention_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
       const int idx = it * 32 + lane;
       const int row = idx / CH, c = idx - row * CH;
       const int rid = __shfl_sync(0xffffffffu, row_id, row);
-      const int bytes = (rid < 0 || c * 8 >= hd) ? 0 : 16;
-      const size_t base = bytes ? (size_t)rid * hd + c * 8 : 0;
-      cp_async16(k_dst + row * RS + c * 8, k_src + base, bytes);
-      if constexpr (!POOLED) cp_async16(v_dst + row * RS + c * 8, v_src + base, bytes);
+      if constexpr (!POOLED) {
+        const size_t base = (size_t)(rid < 0 ? 0 : rid) * HD + c * 8;
+        const int bytes = rid < 0 ? 0 : 16;
+        cp_async16(k_dst + row * RS + c * 8, k_pages + base, bytes);
+        cp_async16(v_dst + row * RS + c * 8, v_pages + base, bytes);
+      } else {
+        const int bytes = (rid < 0 || c * 8 >= hd) ? 0 : 16;
+        cp_async16(k_dst + row * RS + c * 8, k_src + (bytes ? (size_t)rid * hd + c * 8 : 0), bytes);
+      }
     }
     if constexpr (POOLED) {
 #pragma unroll
