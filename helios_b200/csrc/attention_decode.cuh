@@ -258,42 +258,66 @@ decode_attention_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
     if (k_write != nullptr && last_tile >= tile_begin && last_tile < tile_end &&
         (last_tile - tile_begin) % WARPS == warp) {
       const int page = table[pos / page_size];
-      const size_t dst = ((size_t)(page * nkv + kvh) * page_size + pos % page_size) * HD;
-      const __nv_bfloat16* k_new = q + (size_t)seq * q_stride + (size_t)(nh + kvh) * HD;
-      const __nv_bfloat16* v_new = k_new + (size_t)nkv * HD;
-      // a lane holds the pairs (j, j + 1) of both halves of the key: HD / 2 <= 64, one trip
-      float k_factor = 1.f;
-      if (prep.wk != nullptr) {
+      const size_t row0 = (size_t)(page * nkv + kvh) * page_size + pos % page_size;
+      const __nv_bfloat16* k_new = q + (size_t)seq * q_stride + (size_t)nh * hd + (size_t)kvh * hd;
+      const __nv_bfloat16* v_new = q + (size_t)seq * q_stride + (size_t)(nh + nkv) * hd + (size_t)kvh * vd;
+      if constexpr (POOLED) {
+        // sizes of their own, no rotation: a lane holds every 32nd pair of the key
+        __nv_bfloat16* kd = k_write + row0 * hd;
+        float2 x[HD / 64];
         float ss = 0.f;
-        const int j = 2 * lane;
-        if (j < HD / 2) {
-          const float2 x1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j));
-          const float2 x2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j + HD / 2));
-          ss = x1.x * x1.x + x1.y * x1.y + x2.x * x2.x + x2.y * x2.y;
+#pragma unroll
+        for (int i = 0; i < HD / 64; ++i) {
+          const int j = 2 * lane + 64 * i;
+          x[i] = j < hd ? __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j)) : make_float2(0.f, 0.f);
+          ss += x[i].x * x[i].x + x[i].y * x[i].y;
         }
-        k_factor = rsqrtf(warp_sum(ss) / (float)HD + prep.eps);
-      }
-      for (int j = 2 * lane; j < HD / 2; j += 64) {
-        float2 x1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j));
-        float2 x2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j + HD / 2));
+        const float f = prep.wk != nullptr ? rsqrtf(warp_sum(ss) / (float)hd + prep.eps) : 1.f;
+#pragma unroll
+        for (int i = 0; i < HD / 64; ++i) {
+          const int j = 2 * lane + 64 * i;
+          if (j >= hd) continue;
+          const float2 w = prep.wk != nullptr ? *reinterpret_cast<const float2*>(prep.wk + j) : make_float2(1.f, 1.f);
+          *reinterpret_cast<__nv_bfloat162*>(kd + j) = __floats2bfloat162_rn(x[i].x * f * w.x, x[i].y * f * w.y);
+        }
+        for (int j = 8 * lane; j < vd; j += 256)
+          *reinterpret_cast<uint4*>(v_write + row0 * vd + j) = *reinterpret_cast<const uint4*>(v_new + j);
+      } else {
+        const size_t dst = row0 * HD;
+        // a lane holds the pairs (j, j + 1) of both halves of the key: HD / 2 <= 64, one trip
+        float k_factor = 1.f;
         if (prep.wk != nullptr) {
-          const float2 w1 = *reinterpret_cast<const float2*>(prep.wk + j);
-          const float2 w2 = *reinterpret_cast<const float2*>(prep.wk + j + HD / 2);
-          x1 = make_float2(x1.x * k_factor * w1.x, x1.y * k_factor * w1.y);
-          x2 = make_float2(x2.x * k_factor * w2.x, x2.y * k_factor * w2.y);
+          float ss = 0.f;
+          const int j = 2 * lane;
+          if (j < HD / 2) {
+            const float2 x1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j));
+            const float2 x2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j + HD / 2));
+            ss = x1.x * x1.x + x1.y * x1.y + x2.x * x2.x + x2.y * x2.y;
+          }
+          k_factor = rsqrtf(warp_sum(ss) / (float)HD + prep.eps);
         }
-        float2 r1 = x1, r2 = x2;
-        if (rot_cos != nullptr) {
-          const float2 c = *reinterpret_cast<const float2*>(rot_cos + (size_t)seq * (HD / 2) + j);
-          const float2 sn = *reinterpret_cast<const float2*>(rot_sin + (size_t)seq * (HD / 2) + j);
-          r1 = make_float2(x1.x * c.x - x2.x * sn.x, x1.y * c.y - x2.y * sn.y);
-          r2 = make_float2(x2.x * c.x + x1.x * sn.x, x2.y * c.y + x1.y * sn.y);
+        for (int j = 2 * lane; j < HD / 2; j += 64) {
+          float2 x1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j));
+          float2 x2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k_new + j + HD / 2));
+          if (prep.wk != nullptr) {
+            const float2 w1 = *reinterpret_cast<const float2*>(prep.wk + j);
+            const float2 w2 = *reinterpret_cast<const float2*>(prep.wk + j + HD / 2);
+            x1 = make_float2(x1.x * k_factor * w1.x, x1.y * k_factor * w1.y);
+            x2 = make_float2(x2.x * k_factor * w2.x, x2.y * k_factor * w2.y);
+          }
+          float2 r1 = x1, r2 = x2;
+          if (rot_cos != nullptr) {
+            const float2 c = *reinterpret_cast<const float2*>(rot_cos + (size_t)seq * (HD / 2) + j);
+            const float2 sn = *reinterpret_cast<const float2*>(rot_sin + (size_t)seq * (HD / 2) + j);
+            r1 = make_float2(x1.x * c.x - x2.x * sn.x, x1.y * c.y - x2.y * sn.y);
+            r2 = make_float2(x2.x * c.x + x1.x * sn.x, x2.y * c.y + x1.y * sn.y);
+          }
+          *reinterpret_cast<__nv_bfloat162*>(k_write + dst + j) = __floats2bfloat162_rn(r1.x, r1.y);
+          *reinterpret_cast<__nv_bfloat162*>(k_write + dst + j + HD / 2) = __floats2bfloat162_rn(r2.x, r2.y);
         }
-        *reinterpret_cast<__nv_bfloat162*>(k_write + dst + j) = __floats2bfloat162_rn(r1.x, r1.y);
-        *reinterpret_cast<__nv_bfloat162*>(k_write + dst + j + HD / 2) = __floats2bfloat162_rn(r2.x, r2.y);
+        for (int j = 8 * lane; j < HD; j += 256)
+          *reinterpret_cast<uint4*>(v_write + dst + j) = *reinterpret_cast<const uint4*>(v_new + j);
       }
-      for (int j = 8 * lane; j < HD; j += 256)
-        *reinterpret_cast<uint4*>(v_write + dst + j) = *reinterpret_cast<const uint4*>(v_new + j);
       __syncwarp();           // the copies below, by other lanes, read these rows
     }
   }
@@ -335,14 +359,15 @@ decode_attention_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ par
       for (int r = 0; r < 2; ++r) {
         ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], 1);
         ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], 2);
-        inv_rms[r] = prep.wq != nullptr ? rsqrtf(ss[r] / (float)HD + prep.eps) : 1.f;
+        inv_rms[r] = prep.wq != nullptr ? rsqrtf(ss[r] / (float)hd + prep.eps) : 1.f;
       }
 #pragma unroll
       for (int ks = 0; ks < HD / 16; ++ks) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int col = ks * 16 + c0 + (e >> 1) * 8;
-          const float2 w = prep.wq != nullptr ? *reinterpret_cast<const float2*>(prep.wq + col) : make_float2(1.f, 1.f);
+          const float2 w = prep.wq != nullptr && col < hd ? *reinterpret_cast<const float2*>(prep.wq + col)
+                                                          : make_float2(1.f, 1.f);
           const float2 x = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&qa[ks][e]));
           // the norm, the weight, then the temperature: the order of the kernel that does this alone
           const float f = inv_rms[e & 1];

@@ -1,6 +1,7 @@
-// Prefill attention on the 5th-generation tensor cores (attention_prefill_tc.cuh) over a window's
-// tokens and the means of whole blocks behind it, under one softmax: keys and values of sizes of
-// their own up to 256 (not both above 128), compiled for 64, 128 and 256 each.
+// Prefill attention on the 5th-generation tensor cores (attention_prefill_tc.cuh) with keys and values
+// of sizes of their own up to 256 (not both above 128), compiled for 64, 128 and 256 each: over a
+// window's tokens and the means of whole blocks behind it, under one softmax, or over all tokens or a
+// window's without such blocks; with a sink and a gate.
 #include <type_traits>
 #include "attention_prefill_tc.cuh"
 
@@ -43,10 +44,11 @@ HB_EXPORT int hb_attention_pooled_prefill_tc(void* out, int out_stride, float fa
                                              const int* pooled_table, int pooled_stride, int pool, const int* q_tiles,
                                              int n_tiles, const int* cu_tokens, const int* start_pos, int nh, int nkv,
                                              int hd, int vd, int page_size, int window, float scale, int* error,
-                                             cudaStream_t stream) {
+                                             int sink, const float* sink_values, const void* gate, int gate_stride,
+                                             int gate_wide, cudaStream_t stream) {
   if (n_tiles <= 0) return HB_OK;
   if (nkv <= 0 || nh % nkv != 0 || nh / nkv > TILE || error == nullptr || hd <= 0 || hd > 256 || hd % 8 || vd <= 0 ||
-      vd > 256 || vd % 8 || (hd > 128 && vd > 128) || window <= 0 || pool < 0 || page_size < 8 || page_size % 8 != 0 ||
+      vd > 256 || vd % 8 || (hd > 128 && vd > 128) || window < 0 || pool < 0 || (pool > 0 && window <= 0) || page_size < 8 || page_size % 8 != 0 ||
       TILE % page_size != 0 || (q_stride & 7) || (out_stride & 7) || out_stride < nh * vd ||
       (pool > 0 && (!pooled_k || !pooled_v || !pooled_table)) ||
       (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)pooled_k |
@@ -57,6 +59,8 @@ HB_EXPORT int hb_attention_pooled_prefill_tc(void* out, int out_stride, float fa
   a.block_table = block_table; a.bt_stride = bt_stride; a.q_tiles = q_tiles; a.cu_tokens = cu_tokens;
   a.start_pos = start_pos; a.nh = nh; a.nkv = nkv; a.page_size = page_size; a.window = window;
   a.scale_log2 = scale * LOG2E; a.error = error;
+  a.opt.sink = sink; a.opt.sink_values = sink_values;
+  a.opt.gate = (const __nv_bfloat16*)gate; a.opt.gate_stride = gate_stride; a.opt.gate_wide = gate_wide;
   const PooledTiles pl = {pooled_table, pooled_stride, pool, hd, vd, out_stride, factor};
   const long long rows = num_pages * nkv * page_size, prows = pooled_num_pages * nkv * page_size;
 #define HB_POOLED(H, V) return launch_pooled<H, V>(a, pl, k_pages, v_pages, rows, pooled_k, pooled_v, prows, n_tiles, stream)

@@ -44,6 +44,7 @@ LIBRARIES: Dict[str, str] = {
     "moe": "moe.cu",
     "ssm": "ssm.cu",
     "linear_attention": "linear_attention.cu",
+    "gated_linear_attention": "gated_linear_attention.cu",
     "pooled_window": "pooled_window.cu",
     "attention_pooled": "attention_pooled.cu",
     "attention_tc_pooled": "attention_tc_pooled.cu",
@@ -58,6 +59,8 @@ _INCLUDES: Dict[str, List[str]] = {"gemm_bf16_noalloc": ["gemm_bf16.cu", "gemm_b
                                    "attention_tc": ["attention_options.cuh", "attention_prefill_tc.cuh"],
                                    "attention_tc_pooled": ["attention_options.cuh", "attention_prefill_tc.cuh"],
                                    "latent_attention": ["attention_mma.cuh"],
+                                   "linear_attention": ["linear_attention.cuh"],
+                                   "gated_linear_attention": ["linear_attention.cuh"],
                                    "delta_rule": ["causal_conv.cuh"],
                                    "pooled_window": ["causal_conv.cuh"]}
 

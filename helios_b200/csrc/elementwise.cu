@@ -695,6 +695,137 @@ HB_EXPORT int hb_scaled_sum_rmsnorm(float* residual, const void* y, const float*
   return hb_check_launch();
 }
 
+// ---------------------------------------------------------------- norm on an output, then the next norm
+// A block that norms before AND after each sublayer:
+//   x = residual[r] + y[r] / sqrt(mean(y[r]^2) + eps1) * w1          (float32)
+//   out[i] = x / sqrt(mean(x^2) + eps2) * w2
+// with r = rows ? rows[i] : i.  residual[r] becomes x, but not with `rows` (the final norm runs on
+// the wanted rows only).  GROUPS: groups of four neighbouring values a thread keeps (0: any width,
+// value by value).
+template <typename T, int GROUPS>
+__global__ void __launch_bounds__(NORM_THREADS)
+rmsnorm_add_rmsnorm_kernel(T* __restrict__ out, float* __restrict__ residual, const T* __restrict__ y,
+                           const float* __restrict__ w1, const float* __restrict__ w2,
+                           const int* __restrict__ rows, int H, float eps1, float eps2) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const int i = blockIdx.x, r = rows ? rows[i] : i;
+  float* res = residual + (size_t)r * H;
+  const T* yr = y + (size_t)r * H;
+  T* o = out + (size_t)i * H;
+  const bool write_back = rows == nullptr;
+  float ss = 0.f;
+  if constexpr (GROUPS > 0) {
+    float v[GROUPS][4], d[GROUPS][4];
+#pragma unroll
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) { load4(yr + c, d[g]); load4(res + c, v[g]); }
+    }
+#pragma unroll
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss = fmaf(d[g][e], d[g][e], ss);
+      }
+    }
+    const float first = rsqrtf(block_sum(ss, scratch) / (float)H + eps1);
+    ss = 0.f;
+#pragma unroll
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) {
+        float w[4];
+        load4(w1 + c, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[g][e] += d[g][e] * first * w[e];
+          ss = fmaf(v[g][e], v[g][e], ss);
+        }
+        if (write_back) store4(res + c, v[g]);
+      }
+    }
+    const float second = rsqrtf(block_sum(ss, scratch) / (float)H + eps2);
+#pragma unroll
+    for (int g = 0; g < GROUPS; ++g) {
+      const int c = (g * blockDim.x + threadIdx.x) * 4;
+      if (c < H) {
+        float w[4];
+        load4(w2 + c, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[g][e] *= second * w[e];
+        store4(o + c, v[g]);
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < H; c += blockDim.x) { const float d = to_float(yr[c]); ss = fmaf(d, d, ss); }
+    const float first = rsqrtf(block_sum(ss, scratch) / (float)H + eps1);
+    ss = 0.f;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+      const float v = res[c] + to_float(yr[c]) * first * w1[c];
+      if (write_back) res[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+    const float second = rsqrtf(block_sum(ss, scratch) / (float)H + eps2);
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+      const float v = write_back ? res[c] : res[c] + to_float(yr[c]) * first * w1[c];
+      o[c] = from_float<T>(v * second * w2[c]);
+    }
+  }
+}
+
+HB_EXPORT int hb_rmsnorm_add_rmsnorm(void* out, float* residual, const void* y, const float* w1, const float* w2,
+                                     const int* rows, int n_out, int H, float eps1, float eps2, int act_dt,
+                                     cudaStream_t stream) {
+  if (n_out <= 0) return HB_OK;
+  if (H <= 0 || y == nullptr) return HB_BAD_ARGUMENT;
+  const bool vec = H % 4 == 0 && H <= NORM_THREADS * NORM_GROUPS * 4 && (act_dt == HB_F32 || H % 8 == 0) &&
+                   (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)out) & 15) == 0;
+  const int groups = vec ? (H + NORM_THREADS * 4 - 1) / (NORM_THREADS * 4) : 0;
+#define HB_NORM_NORM(G)                                                                                       \
+  hb_launch(rmsnorm_add_rmsnorm_kernel<TA, G>, dim3(n_out), dim3(NORM_THREADS), 0, stream, (TA*)out, residual,   \
+            (const TA*)y, w1, w2, rows, H, eps1, eps2)
+  HB_DISPATCH_DTYPE(act_dt, TA,
+    if (groups == 0) HB_NORM_NORM(0);
+    else if (groups == 1) HB_NORM_NORM(1);
+    else if (groups == 2) HB_NORM_NORM(2);
+    else if (groups <= 4) HB_NORM_NORM(4);
+    else HB_NORM_NORM(8));
+#undef HB_NORM_NORM
+  return hb_check_launch();
+}
+
+// ---------------------------------------------------------------- a bound on the logits
+// x = cap * tanh(x / cap), in place
+__global__ void __launch_bounds__(256)
+softcap_kernel(float* __restrict__ x, size_t n, float cap, int vec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const float inv = 1.f / cap;
+  const size_t stride = (size_t)gridDim.x * blockDim.x, tid = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (vec) {
+    for (size_t i = tid; i < n / 4; i += stride) {
+      float4 v = reinterpret_cast<float4*>(x)[i];
+      v = make_float4(cap * tanhf(v.x * inv), cap * tanhf(v.y * inv), cap * tanhf(v.z * inv), cap * tanhf(v.w * inv));
+      reinterpret_cast<float4*>(x)[i] = v;
+    }
+  } else {
+    for (size_t i = tid; i < n; i += stride) x[i] = cap * tanhf(x[i] * inv);
+  }
+}
+
+HB_EXPORT int hb_softcap(float* x, long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return HB_OK;
+  if (!(cap > 0.f)) return HB_BAD_ARGUMENT;
+  const int vec = n % 4 == 0 && (uintptr_t)x % 16 == 0;
+  size_t blocks = ((size_t)n / (vec ? 4 : 1) + 255) / 256;
+  if (blocks > 148 * 8) blocks = 148 * 8;
+  hb_launch(softcap_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, (size_t)n, cap, vec);
+  return hb_check_launch();
+}
+
 // ---------------------------------------------------------------- layer norm with a pending sum
 // A block whose sublayers all read ONE norm of the stream leaves its outputs to be added:
 //   residual[r, c] += mult * (sa[c] * a[r, c] + sb[c] * b[r, c])      (float32; a, b, sa, sb optional)
@@ -912,7 +1043,8 @@ HB_EXPORT int hb_cast_rows(void* dst, int ld, int col0, const float* src, int T,
 // a k head becomes k / rms(k) * wk at the token's place in its key pages, a v head is copied
 // to the value pages.  rms over the head's hd values with eps inside the root; norm weights
 // null: no norm.  Pages: [page, kv head, slot, hd] and [page, kv head, slot, vd].  All
-// arithmetic float32.  Without `write_cache` k is normed in place and v left alone.
+// arithmetic float32.  Without `write_cache` k is normed in place and v left alone; rows of queries
+// alone have nkv = 0.
 template <typename T>
 __global__ void __launch_bounds__(128)
 qk_norm_kv_write_kernel(T* __restrict__ rows, int ld, const int* __restrict__ positions,
@@ -1047,7 +1179,7 @@ HB_EXPORT int hb_qk_norm_kv_write(void* rows, int ld, const int* positions, cons
                                   const float* wk, float eps, float coef, int every, int page_size,
                                   int write_cache, int act_dt, cudaStream_t stream) {
   if (T <= 0) return HB_OK;
-  if (nh <= 0 || nkv <= 0 || hd <= 0 || vd <= 0 || page_size <= 0 || every < 0 ||
+  if (nh <= 0 || nkv < 0 || hd <= 0 || vd <= 0 || page_size <= 0 || every < 0 || (nkv == 0 && write_cache) ||
       (long)nh * hd + (long)nkv * (hd + vd) > ld)
     return HB_BAD_ARGUMENT;
   const int group = hd / 8;
@@ -1469,13 +1601,15 @@ HB_EXPORT int hb_unary_act(void* out, const void* x, const void* gate, int gate_
   return hb_check_launch();
 }
 
-// ---------------------------------------------------------------- a gate on every value of every head
-// out[t, h * N + n] = x[t, h, n] * sigmoid(gate[t, h * N + n]): x is a view [T, H, N] with a
+// ---------------------------------------------------------------- a gate on every head or every value of it
+// out[t, h * N + n] = x[t, h, n] * sigmoid(gate[t, h * N + n]), or, with `per_head`, times
+// sigmoid(gate[t, h]): x is a view [T, H, N] with a
 // token stride and a head stride (what a batched product of one matrix a head leaves), gate rows
 // are gate_ld apart, out is contiguous.  float32 arithmetic.
 template <typename T>
 __global__ void gate_heads_kernel(T* __restrict__ out, const T* __restrict__ x, long x_token, long x_head,
-                                  const T* __restrict__ gate, int gate_ld, size_t total, int H, int N) {
+                                  const T* __restrict__ gate, int gate_ld, size_t total, int H, int N,
+                                  int per_head) {
   pdl_launch_dependents();
   pdl_wait();
   const int W = H * N;
@@ -1484,7 +1618,7 @@ __global__ void gate_heads_kernel(T* __restrict__ out, const T* __restrict__ x, 
     const size_t t = idx / W;
     const int c = (int)(idx - t * W), h = c / N, n = c - h * N;
     const float v = to_float(x[t * x_token + (size_t)h * x_head + n]);
-    const float g = to_float(gate[t * (size_t)gate_ld + c]);
+    const float g = to_float(gate[t * (size_t)gate_ld + (per_head ? h : c)]);
     out[idx] = from_float<T>(v / (1.f + expf(-g)));
   }
 }
@@ -1492,7 +1626,7 @@ __global__ void gate_heads_kernel(T* __restrict__ out, const T* __restrict__ x, 
 // bfloat16, N a multiple of 8 and every row 16-byte aligned: eight values a thread and step
 __global__ void gate_heads_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x,
                                          long x_token, long x_head, const __nv_bfloat16* __restrict__ gate,
-                                         int gate_ld, size_t pieces, int H, int N) {
+                                         int gate_ld, size_t pieces, int H, int N, int per_head) {
   pdl_launch_dependents();
   pdl_wait();
   const int W8 = H * N / 8, N8 = N / 8;
@@ -1501,6 +1635,17 @@ __global__ void gate_heads_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const 
     const size_t t = idx / W8;
     const int c = (int)(idx - t * W8), h = c / N8, n = (c - h * N8) * 8;
     const uint4 xv = *reinterpret_cast<const uint4*>(x + t * x_token + (size_t)h * x_head + n);
+    if (per_head) {
+      const float f = 1.f / (1.f + expf(-__bfloat162float(gate[t * (size_t)gate_ld + h])));
+      uint4 ov;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 a = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&xv)[i]);
+        reinterpret_cast<__nv_bfloat162*>(&ov)[i] = __floats2bfloat162_rn(a.x * f, a.y * f);
+      }
+      *reinterpret_cast<uint4*>(out + idx * 8) = ov;
+      continue;
+    }
     const uint4 gv = *reinterpret_cast<const uint4*>(gate + t * (size_t)gate_ld + (size_t)c * 8);
     const __nv_bfloat162* xp = reinterpret_cast<const __nv_bfloat162*>(&xv);
     const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(&gv);
@@ -1516,25 +1661,26 @@ __global__ void gate_heads_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const 
 }
 
 HB_EXPORT int hb_gate_heads(void* out, const void* x, long x_token, long x_head, const void* gate, int gate_ld,
-                            int T, int H, int N, int act_dt, cudaStream_t stream) {
+                            int T, int H, int N, int per_head, int act_dt, cudaStream_t stream) {
   if (T <= 0 || H <= 0 || N <= 0) return HB_OK;
-  if (gate == nullptr || gate_ld < H * N) return HB_BAD_ARGUMENT;
+  if (gate == nullptr || gate_ld < (per_head ? H : H * N)) return HB_BAD_ARGUMENT;
   const size_t total = (size_t)T * H * N;
   const bool aligned = ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(x) |
-                         reinterpret_cast<uintptr_t>(gate)) & 15) == 0;
-  if (act_dt == HB_BF16 && N % 8 == 0 && x_token % 8 == 0 && x_head % 8 == 0 && gate_ld % 8 == 0 && aligned) {
+                         (per_head ? 0 : reinterpret_cast<uintptr_t>(gate))) & 15) == 0;
+  if (act_dt == HB_BF16 && N % 8 == 0 && x_token % 8 == 0 && x_head % 8 == 0 && (per_head || gate_ld % 8 == 0) &&
+      aligned) {
     const size_t pieces = total / 8;
     size_t blocks = (pieces + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     hb_launch(gate_heads_bf16x8_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, (__nv_bfloat16*)out,
-              (const __nv_bfloat16*)x, x_token, x_head, (const __nv_bfloat16*)gate, gate_ld, pieces, H, N);
+              (const __nv_bfloat16*)x, x_token, x_head, (const __nv_bfloat16*)gate, gate_ld, pieces, H, N, per_head);
     return hb_check_launch();
   }
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   HB_DISPATCH_DTYPE(act_dt, TA,
     hb_launch(gate_heads_kernel<TA>, dim3((unsigned)blocks), dim3(256), 0, stream, (TA*)out, (const TA*)x,
-              x_token, x_head, (const TA*)gate, gate_ld, total, H, N));
+              x_token, x_head, (const TA*)gate, gate_ld, total, H, N, per_head));
   return hb_check_launch();
 }
 

@@ -7,11 +7,14 @@
 //   score(t, h, j) = (q_lat[t, h] . c_j + q_rot[t, h] . r_j) * scale
 //   o_lat[t, h]    = sum_j softmax_j(score) c_j
 //
+// over the positions j <= own, or, with a window W, own - W < j <= own; with `sink` (float [heads]) the
+// softmax has one more key of score sink[h] that carries no value.
+//
 // Three kernels: `latent_prepare` (RMS norm of the latent, rotary on the shared key part
 // and on the queries' rotated parts, cache write), `head_gemm` (the folded products, one
 // small matrix per head) and `latent_attention` (one warp per (token, head), float32
-// scores, softmax and sums, keys walked in runs of 32 from position 0 so that the order
-// of every sum depends on the token's position alone).
+// scores, softmax and sums, keys walked in runs of 32 from position 0, or from the window's
+// first key, so that the order of every sum depends on the token's position alone).
 #include "common.cuh"
 
 // ---------------------------------------------------------------- prepare
@@ -202,7 +205,7 @@ latent_attention_kernel(T* __restrict__ out, const T* __restrict__ q_lat, long q
                         const T* __restrict__ pages, const int* __restrict__ block_table,
                         int bt_stride, const int* __restrict__ seq_of_token,
                         const int* __restrict__ positions, int n_rows, int heads, int rank, int rot,
-                        int page_size, float scale) {
+                        int page_size, float scale, int window, const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float q_smem[];
@@ -227,7 +230,8 @@ latent_attention_kernel(T* __restrict__ out, const T* __restrict__ q_lat, long q
   for (int i = 0; i < ND; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
 
-  for (int base = 0; base <= pos; base += 32) {
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  for (int base = lo; base <= pos; base += 32) {
     const int key = base + lane;
     const bool valid = key <= pos;
     int page = 0;
@@ -258,6 +262,13 @@ latent_attention_kernel(T* __restrict__ out, const T* __restrict__ q_lat, long q
       }
     }
   }
+  if (sink) {
+    const float m_new = fmaxf(m, sink[h]);
+    const float corr = expf(m - m_new);
+    l = l * corr + expf(sink[h] - m_new);
+#pragma unroll
+    for (int i = 0; i < ND; ++i) acc[i] *= corr;
+  }
   const float inv = 1.f / l;
   T* orow = out + ((size_t)t * heads + h) * rank;
 #pragma unroll
@@ -271,7 +282,8 @@ HB_EXPORT int hb_latent_attention(void* out, const void* q_lat, long ql_t, long 
                                   const void* q_rot, long qr_t, long qr_h, const void* pages,
                                   const int* block_table, int bt_stride, const int* seq_of_token,
                                   const int* positions, int T, int heads, int rank, int rot,
-                                  int page_size, float scale, int act_dt, cudaStream_t stream) {
+                                  int page_size, float scale, int window, const float* sink, int act_dt,
+                                  cudaStream_t stream) {
   if (T <= 0) return HB_OK;
   if (heads <= 0 || rank <= 0 || rank > LA_MAX_RANK || rot < 0 || rank + rot > LA_MAX_ROW ||
       page_size <= 0)
@@ -283,7 +295,7 @@ HB_EXPORT int hb_latent_attention(void* out, const void* q_lat, long ql_t, long 
     hb_launch(latent_attention_kernel<TA>, dim3(blocks), dim3(LA_WARPS * 32), smem, stream,
               (TA*)out, (const TA*)q_lat, ql_t, ql_h, (const TA*)q_rot, qr_t, qr_h,
               (const TA*)pages, block_table, bt_stride, seq_of_token, positions, n_rows, heads,
-              rank, rot, page_size, scale));
+              rank, rot, page_size, scale, window, sink));
   return hb_check_launch();
 }
 
@@ -308,6 +320,15 @@ HB_EXPORT int hb_latent_attention(void* out, const void* q_lat, long ql_t, long 
 
 constexpr int LM_ROWS = 32, LM_KEYS = 32, LM_MAXNT = 16, LM_SPAD = 36, LM_PPAD = 40;
 
+// The factor on a row's accumulator: 1 / l, the sum relative to the maximum m (log2 domain), with the
+// sink's share in the sum where there is one.
+__device__ __forceinline__ float latent_finish(float m, float l, const float* sink, int head) {
+  if (sink == nullptr) return l > 0.f ? 1.f / l : 0.f;
+  const float s = sink[head] * 1.4426950408889634f, top = fmaxf(m, s);
+  const float f = exp2f(m - top);
+  return f / (l * f + exp2f(s - top));
+}
+
 // NTQ = rank / 32: the 8-column tiles of the latent a warp owns, a template parameter so that the
 // loops over them unroll without predicates (with a run-time count, integer arithmetic and
 // branches were most of the executed instructions and the tensor pipe a twentieth).
@@ -322,7 +343,7 @@ latent_attention_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__
                             const int* __restrict__ q_tiles, const int* __restrict__ cu_tokens,
                             const int* __restrict__ start_pos, int heads, int heads_per_block,
                             int tokens_per_tile, int rank, int rot, int page_size, int page_shift,
-                            float scale_log2, int n_splits) {
+                            float scale_log2, int n_splits, int window, const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) unsigned char lm_smem[];
@@ -347,9 +368,12 @@ latent_attention_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__
   const int* table = block_table + (size_t)seq * bt_stride;
   const int last_tok = min(t_first + tokens_per_tile, n_tok);
   const int n_keys = start_pos[seq] + last_tok;       // the tile's last token sees this many keys
+  // the first key that the tile's first token sees; pages wholly before it may have been given back
+  const int k_first = window > 0 ? max(0, start_pos[seq] + t_first - window + 1) : 0;
+  const int kt_first = k_first / LM_KEYS;
   const int n_kt = (n_keys + LM_KEYS - 1) / LM_KEYS;
-  const int per = (n_kt + n_splits - 1) / n_splits;
-  const int kt_lo = split * per, kt_hi = min(n_kt, kt_lo + per);
+  const int per = (n_kt - kt_first + n_splits - 1) / n_splits;
+  const int kt_lo = kt_first + split * per, kt_hi = min(n_kt, kt_lo + per);
 
   if (tid < LM_ROWS) {
     const int lt = tid / heads_per_block, h = h0 + tid % heads_per_block;
@@ -377,13 +401,13 @@ latent_attention_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__
 
   // Lane r finds the row of key kt * 32 + r (its page from the block table); warp w then
   // copies rows 4 w .. 4 w + 3 in 16-byte pieces, the row's start handed over by shuffles:
-  // no division per piece.  Rows beyond the last key are zero-filled.
+  // no division per piece.  Rows beyond the last key, and before the first, are zero-filled.
   const int vec_per_row = D / 8;
   auto load_tile = [&](int kt, int buf) {
     __nv_bfloat16* dst = k_s + (size_t)buf * LM_KEYS * RS;
     const int key = kt * LM_KEYS + lane;
     long long row_off = -1;
-    if (key < n_keys) {
+    if (key < n_keys && key >= k_first) {
       const int pg = page_shift >= 0 ? key >> page_shift : key / page_size;
       const int in_pg = page_shift >= 0 ? key & (page_size - 1) : key - pg * page_size;
       row_off = ((long long)table[pg] * page_size + in_pg) * D;
@@ -446,10 +470,11 @@ latent_attention_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__
       const int key = kt * LM_KEYS + 8 * cq + 2 * t4;
       const int ra = rg * 16 + g, rb = ra + 8;
       const int pa = row_pos[ra], pb = row_pos[rb];
-      s_s[ra * LM_SPAD + 8 * cq + 2 * t4] = key <= pa ? c[0] * scale_log2 : -INFINITY;
-      s_s[ra * LM_SPAD + 8 * cq + 2 * t4 + 1] = key + 1 <= pa ? c[1] * scale_log2 : -INFINITY;
-      s_s[rb * LM_SPAD + 8 * cq + 2 * t4] = key <= pb ? c[2] * scale_log2 : -INFINITY;
-      s_s[rb * LM_SPAD + 8 * cq + 2 * t4 + 1] = key + 1 <= pb ? c[3] * scale_log2 : -INFINITY;
+      const int la = window > 0 ? pa - window : -1, lb = window > 0 ? pb - window : -1;    // last key not seen
+      s_s[ra * LM_SPAD + 8 * cq + 2 * t4] = key <= pa && key > la ? c[0] * scale_log2 : -INFINITY;
+      s_s[ra * LM_SPAD + 8 * cq + 2 * t4 + 1] = key + 1 <= pa && key + 1 > la ? c[1] * scale_log2 : -INFINITY;
+      s_s[rb * LM_SPAD + 8 * cq + 2 * t4] = key <= pb && key > lb ? c[2] * scale_log2 : -INFINITY;
+      s_s[rb * LM_SPAD + 8 * cq + 2 * t4 + 1] = key + 1 <= pb && key + 1 > lb ? c[3] * scale_log2 : -INFINITY;
     }
     __syncthreads();
     // online softmax, once a row: warp cq of a row group takes its rows 4 cq .. 4 cq + 3, eight
@@ -532,7 +557,7 @@ latent_attention_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__
     const int row = row_out[rg * 16 + g + 8 * r];
     if (row < 0) continue;
     if (n_splits == 1) {
-      const float inv = l[r] > 0.f ? 1.f / l[r] : 0.f;
+      const float inv = latent_finish(m[r], l[r], sink, row % heads);
       __nv_bfloat16* dst = out + (size_t)row * rank + col_q + 2 * t4;
 #pragma unroll
       for (int nt = 0; nt < NTQ; ++nt)
@@ -551,11 +576,12 @@ latent_attention_mma_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__
   }
 }
 
-// out[row] = sum_i 2^(m_i - M) acc_i / sum_i 2^(m_i - M) l_i over the ranges, i in order
+// out[row] = sum_i 2^(m_i - M) acc_i / sum_i 2^(m_i - M) l_i over the ranges, i in order (and the
+// sink's term in the denominator)
 __global__ void latent_attention_merge_kernel(__nv_bfloat16* __restrict__ out,
                                               const float* __restrict__ part_acc,
                                               const float* __restrict__ part_ml, int n_rows,
-                                              int rank, int n_splits) {
+                                              int rank, int n_splits, const float* __restrict__ sink, int heads) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -565,7 +591,7 @@ __global__ void latent_attention_merge_kernel(__nv_bfloat16* __restrict__ out,
   for (int i = 0; i < n_splits; ++i) M = fmaxf(M, ml[2 * i]);
   float L = 0.f;
   for (int i = 0; i < n_splits; ++i) L += (ml[2 * i] == -INFINITY ? 0.f : exp2f(ml[2 * i] - M)) * ml[2 * i + 1];
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  const float inv = latent_finish(M, L, sink, row % heads);
   for (int d = lane; d < rank; d += 32) {
     float a = 0.f;
     for (int i = 0; i < n_splits; ++i) {
@@ -582,7 +608,8 @@ HB_EXPORT int hb_latent_attention_mma(void* out, float* part_acc, float* part_ml
                                       const int* q_tiles, int n_tiles, const int* cu_tokens,
                                       const int* start_pos, int n_tokens, int heads,
                                       int heads_per_block, int tokens_per_tile, int rank, int rot,
-                                      int page_size, float scale, int n_splits, cudaStream_t stream) {
+                                      int page_size, float scale, int n_splits, int window, const float* sink,
+                                      cudaStream_t stream) {
   if (n_tiles <= 0 || n_tokens <= 0) return HB_OK;
   if (rank <= 0 || rank % 32 || rank > 32 * LM_MAXNT || rot < 0 || rot % 16 || heads <= 0 ||
       heads_per_block <= 0 || heads_per_block > LM_ROWS || tokens_per_tile <= 0 ||
@@ -610,7 +637,7 @@ HB_EXPORT int hb_latent_attention_mma(void* out, float* part_acc, float* part_ml
               stream, (__nv_bfloat16*)out, part_acc, part_ml, (const __nv_bfloat16*)q_lat, ql_t, ql_h, \
               (const __nv_bfloat16*)q_rot, qr_t, qr_h, (const __nv_bfloat16*)pages, block_table,     \
               bt_stride, q_tiles, cu_tokens, start_pos, heads, heads_per_block, tokens_per_tile, rank, \
-              rot, page_size, page_shift, scale * 1.4426950408889634f, n_splits);                    \
+              rot, page_size, page_shift, scale * 1.4426950408889634f, n_splits, window, sink);      \
     break;
   switch (rank / 32) {
     HB_LM_LAUNCH(1) HB_LM_LAUNCH(2) HB_LM_LAUNCH(3) HB_LM_LAUNCH(4) HB_LM_LAUNCH(5) HB_LM_LAUNCH(6)
@@ -622,7 +649,8 @@ HB_EXPORT int hb_latent_attention_mma(void* out, float* part_acc, float* part_ml
   if (n_splits > 1) {
     const int n_rows = n_tokens * heads;
     hb_launch(latent_attention_merge_kernel, dim3((n_rows + 3) / 4), dim3(128), 0, stream,
-              (__nv_bfloat16*)out, (const float*)part_acc, (const float*)part_ml, n_rows, rank, n_splits);
+              (__nv_bfloat16*)out, (const float*)part_acc, (const float*)part_ml, n_rows, rank, n_splits, sink,
+              heads);
   }
   return hb_check_launch();
 }

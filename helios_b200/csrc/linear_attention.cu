@@ -24,13 +24,9 @@
 //                 plain float32 o
 // The products of the chunked form run on the float32 FMA pipes: the operands are float32 (a
 // rotated key, a decayed state), and nothing of the recurrence is rounded to 16 bits.
-#include "common.cuh"
+#include "linear_attention.cuh"
 
 namespace {
-
-constexpr int LA_C = 64;             // tokens a chunk
-constexpr int LA_BLK = 64;           // rows / columns of S a tile
-constexpr int LA_LD = LA_BLK + 4;    // row stride of a tile in shared memory (16-byte rows)
 
 enum { LA_NONE = 0, LA_SILU = 1 };
 
@@ -62,29 +58,6 @@ __device__ __forceinline__ float la_qk(const LaIn<T>& in, const T* x, int t, int
     v = d < in.half ? v * c - o * s : v * c + o * s;
   }
   return v;
-}
-
-template <typename T>
-__device__ __forceinline__ void la_load4(const T* p, float (&f)[4]) {
-  if constexpr (sizeof(T) == 4) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
-  } else {
-    const uint2 x = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
-    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-  }
-}
-
-template <typename T>
-__device__ __forceinline__ void la_store4(T* p, const float (&f)[4]) {
-  if constexpr (sizeof(T) == 4) {
-    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  } else {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-  }
 }
 
 // Columns d .. d + 3 of a q or k head (zeros from column N on).
@@ -189,45 +162,7 @@ __device__ __forceinline__ void la_turn(const LaIn<T>& in, const LaPlaces<B>& at
   }
 }
 
-__device__ __forceinline__ float la_gate(float g, int kind) {
-  const float s = 1.f / (1.f + expf(-g));
-  return kind == 0 ? g * s : s;              // silu | sigmoid
-}
-
 // ---------------------------------------------------------------- token by token
-constexpr int LA_PARTS = 8;          // warps that share a column's rows
-constexpr int LA_STAGE = 8;          // tokens staged in shared memory at a time
-
-template <int VEC>
-__device__ __forceinline__ void la_load_state(float (&s)[VEC], const float* p, int left, bool vec) {
-  if (VEC == 4 && vec) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    s[0] = x.x;
-    if (VEC > 1) s[1 % VEC] = x.y;
-    if (VEC > 2) { s[2 % VEC] = x.z; s[3 % VEC] = x.w; }
-  } else if (VEC == 2 && vec) {
-    const float2 x = *reinterpret_cast<const float2*>(p);
-    s[0] = x.x;
-    s[1 % VEC] = x.y;
-  } else {
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) s[e] = e < left ? p[e] : 0.f;
-  }
-}
-
-template <int VEC>
-__device__ __forceinline__ void la_store_state(const float (&s)[VEC], float* p, int left, bool vec) {
-  if (VEC == 4 && vec) {
-    *reinterpret_cast<float4*>(p) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
-  } else if (VEC == 2 && vec) {
-    *reinterpret_cast<float2*>(p) = make_float2(s[0], s[1 % VEC]);
-  } else {
-#pragma unroll
-    for (int e = 0; e < VEC; ++e)
-      if (e < left) p[e] = s[e];
-  }
-}
-
 // A warp takes every eighth row of S, a lane VEC neighbouring columns of it, so that whole rows
 // of up to 128 columns are read and written at once.  `o` (float32 [T, heads, M]) is written when
 // it is given; else (one block a head) norm per head and gate are applied and `out` is written.
@@ -328,16 +263,6 @@ la_scan_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn<T> i
 }
 
 // ---------------------------------------------------------------- chunks
-// q_tiles: (request, first token of the chunk inside the request's step) per chunk of LA_C tokens,
-// in the requests' order; a tile at or beyond the request's tokens holds no work.
-__device__ __forceinline__ int la_tile_tokens(const int* q_tiles, const int* cu_tokens, int tile, int& tok0) {
-  const int seq = q_tiles[2 * tile], l0 = q_tiles[2 * tile + 1];
-  const int begin = cu_tokens[seq], n = cu_tokens[seq + 1] - begin;
-  if (l0 >= n) return 0;
-  tok0 = begin + l0;
-  return min(LA_C, n - l0);
-}
-
 // A block takes NB x NB entries of a chunk's sum, a thread E x E of them (NB = 16 E): k_j v_j^T over the
 // chunk's tokens from rows in shared memory.
 template <typename T, int E>
@@ -491,35 +416,6 @@ la_states_kernel(float* __restrict__ sums, float* __restrict__ state, long state
   }
 #pragma unroll
   for (int w = 0; w < W; ++w) mine[w] = s[w];
-}
-
-// acc[i][4 vb + e] += sum_d A[i][d] B[d][64 vb + 4 tx + e] for rows i = ty + 16 r: A [64][LA_LD] rows by
-// query token, B [inner][VB * 64 + 4] rows by the inner index.  Four inner steps at a time.  FROM: only
-// the row groups r >= FROM.
-template <int VB, int FROM = 0>
-__device__ __forceinline__ void la_rows_times(float (&acc)[4][4 * VB], const float* A, const float* B, int ty, int tx,
-                                              int inner) {
-  constexpr int LD = VB * LA_BLK + 4;
-#pragma unroll 2
-  for (int d = 0; d < inner; d += 4) {
-    float x[4][4];
-#pragma unroll
-    for (int r = FROM; r < 4; ++r) *reinterpret_cast<float4*>(x[r]) = *reinterpret_cast<const float4*>(A + (ty + 16 * r) * LA_LD + d);
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-#pragma unroll
-      for (int vb = 0; vb < VB; ++vb) {
-        const float4 y = *reinterpret_cast<const float4*>(B + (d + u) * LD + vb * LA_BLK + 4 * tx);
-#pragma unroll
-        for (int r = FROM; r < 4; ++r) {
-          acc[r][4 * vb] = fmaf(x[r][u], y.x, acc[r][4 * vb]);
-          acc[r][4 * vb + 1] = fmaf(x[r][u], y.y, acc[r][4 * vb + 1]);
-          acc[r][4 * vb + 2] = fmaf(x[r][u], y.z, acc[r][4 * vb + 2]);
-          acc[r][4 * vb + 3] = fmaf(x[r][u], y.w, acc[r][4 * vb + 3]);
-        }
-      }
-    }
-  }
 }
 
 // VB: blocks of 64 columns of v a head has.  A thread owns the query tokens ty + 16 r and, of the
@@ -727,8 +623,8 @@ la_chunk_out_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, LaIn
 }
 
 // ---------------------------------------------------------------- norm and gate
-// out = factor * o / rms(o) (* weight) * gate(g): per head (a block a (token, head), weight null)
-// or over the row (a block a token).
+// out = factor * o / rms(o) (* weight) * gate(g): per head (a block a (token, head)) or over the
+// row (a block a token); the weight has an entry per value of the norm.
 template <typename T>
 __global__ void la_gate_norm_kernel(T* __restrict__ out, int out_ld, const float* __restrict__ o,
                                     const T* __restrict__ gate, int gate_ld, const float* __restrict__ weight,
@@ -909,12 +805,13 @@ HB_EXPORT int hb_la_chunked(float* o, void* out, int out_ld, float* sums, const 
   return HB_OK;
 }
 
-// parts: norms a row has (heads: per head, 1: over the row), each `width` values wide.
+// parts: norms a row has (heads: per head, 1: over the row), each `width` values wide; weight
+// [width] (or null): one for all of them.
 HB_EXPORT int hb_la_gate_norm(void* out, int out_ld, const float* o, const void* gate, int gate_ld,
                               const float* weight, int T, int parts, int width, int gate_kind, float eps,
                               float factor, int act_dt, cudaStream_t stream) {
   if (T <= 0) return HB_OK;
-  if (parts <= 0 || width <= 0 || (weight != nullptr && parts != 1)) return HB_BAD_ARGUMENT;
+  if (parts <= 0 || width <= 0) return HB_BAD_ARGUMENT;
   int threads = 32;
   if (width % 4 == 0 && width <= 4096 && ((gate_ld | out_ld) & 3) == 0 &&
       (((uintptr_t)out | (uintptr_t)o | (uintptr_t)weight) & 15) == 0 &&

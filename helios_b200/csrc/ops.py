@@ -114,10 +114,17 @@ def attention_libraries(dtype: torch.dtype, num_heads: int, num_kv_heads: int, h
 
 def option_attention_libraries(dtype: torch.dtype, num_heads: int, num_kv_heads: int, head_dim: int,
                                value_dim: int, tiled: bool = True):
-    """Libraries attention with ``AttentionOptions`` may choose from at these sizes."""
-    if dtype != torch.bfloat16 or head_dim not in TILED_HEAD_DIMS or value_dim != head_dim \
-            or not ATTENTION_OPTIONS_TILED:
+    """Libraries attention with ``AttentionOptions`` may choose from at these sizes (``tiled`` False:
+    options the kernels for sizes of their own do not take)."""
+    if dtype != torch.bfloat16 or not ATTENTION_OPTIONS_TILED:
         return ("attention_generic",)
+    if head_dim not in TILED_HEAD_DIMS or value_dim != head_dim:
+        names = []
+        if tiled and pooled_decode_supported(num_heads, num_kv_heads, head_dim, value_dim):
+            names.append("attention_pooled")
+        if tiled and pooled_tc_supported(num_heads, num_kv_heads, head_dim, value_dim, 16):
+            names.append("attention_tc_pooled")
+        return tuple(names) if len(names) == 2 else tuple(names + ["attention_generic"])
     names = ["attention_bf16"]
     if ATTENTION_TCGEN05 and tc_attention_supported(num_heads, num_kv_heads, head_dim, 16):
         names.append("attention_tc")
@@ -237,21 +244,23 @@ def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def gate_heads(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-    """out[t, h * N + n] = x[t, h, n] * sigmoid(gate[t, h * N + n]): ``x`` is a view [T, H, N]
-    whose last dimension is contiguous (the result of one small product a head, whatever its
-    token and head strides: no copy is made), ``gate`` [T, >= H * N] a view whose rows may be
-    strided.  Returns a contiguous [T, H * N]."""
+def gate_heads(x: torch.Tensor, gate: torch.Tensor, per_head: bool = False) -> torch.Tensor:
+    """out[t, h * N + n] = x[t, h, n] * sigmoid(gate[t, h * N + n]), or, ``per_head``, times
+    sigmoid(gate[t, h]): ``x`` is a view [T, H, N] whose last dimension is contiguous (the result
+    of one small product a head, whatever its token and head strides: no copy is made), ``gate``
+    [T, >= H * N] (``per_head``: [T, >= H]) a view whose rows may be strided.  Returns a
+    contiguous [T, H * N]."""
     if x.dim() != 3 or x.stride(2) != 1 or not x.is_cuda:
         raise KernelError(f"gate_heads: x {tuple(x.shape)} must be [T, H, N] with a contiguous last dimension")
     T, H, N = x.shape
     if gate.dim() != 2 or gate.stride(1) != 1 or gate.dtype != x.dtype or gate.shape[0] != T \
-            or gate.shape[1] < H * N or not gate.is_cuda:
+            or gate.shape[1] < (H if per_head else H * N) or not gate.is_cuda:
         raise KernelError(f"gate {tuple(gate.shape)} does not fit x {tuple(x.shape)}")
     out = torch.empty((T, H * N), dtype=x.dtype, device=x.device)
     f = _fn("elementwise", "hb_gate_heads", [c_void_p, c_void_p, ctypes.c_long, ctypes.c_long, c_void_p, c_int,
-                                             c_int, c_int, c_int, c_int, c_void_p])
-    _run(f(_p(out), _p(x), x.stride(0), x.stride(1), _p(gate), gate.stride(0), T, H, N, _dt(x.dtype), _stream()),
+                                             c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _run(f(_p(out), _p(x), x.stride(0), x.stride(1), _p(gate), gate.stride(0), T, H, N, 1 if per_head else 0,
+           _dt(x.dtype), _stream()),
          "gate_heads")
     return out
 
@@ -1082,8 +1091,8 @@ def attention_decode_bf16(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
     requests' new keys (rotated likewise) and values are still in ``qkv`` and the kernel
     stores them in the pages before it attends.  (Without either, ``rope_kv_write`` must have
     run.)  ``qk_norm`` = (q weight, k weight, eps, temperature coefficient, temperature period):
-    what ``qk_norm_kv_write`` does to q and k, done on the way in (needs ``write_cache``; rows may
-    be wider than q | k | v).  ``qkv`` itself is left as it was.  ``warps``: 4 (the default) or 8 warps a block
+    what ``qk_norm_kv_write`` does to q and k, done on the way in (rows may be wider than q | k | v;
+    without ``write_cache`` to q alone, and there is no k weight).  ``qkv`` itself is left as it was.  ``warps``: 4 (the default) or 8 warps a block
     (``decode_warps``)."""
     _check(qkv, "qkv", torch.bfloat16, 2)
     _check(k_pages, "k_pages", torch.bfloat16, 4)
@@ -1114,14 +1123,14 @@ def attention_decode_bf16(qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
     n_eps, t_coef, t_every = 0.0, 0.0, 0
     if qk_norm is not None:
         wq, wk, n_eps, t_coef, t_every = qk_norm
-        if not write_cache:
-            raise KernelError("q/k norm inside the decode kernel goes with the cache write")
+        if not write_cache and wk is not None:
+            raise KernelError("a key norm inside the decode kernel goes with the cache write")
         for name, w in (("q norm weight", wq), ("k norm weight", wk)):
             if w is not None:
                 _check(w, name, torch.float32, 1)
                 if w.numel() != head_dim:
                     raise KernelError(f"{name} has {w.numel()} entries for heads of {head_dim}")
-        if (wq is None) != (wk is None):
+        if write_cache and (wq is None) != (wk is None):
             raise KernelError("query and key norm come together")
     exact = qk_norm is None            # rows of a fused projection may carry more columns behind q | k | v
     if (cos is not None or write_cache) and ((qkv.shape[1] != (num_heads + 2 * num_kv_heads) * head_dim if exact
@@ -1374,36 +1383,46 @@ def _attention_with_options(ctx, qkv, k_pages, v_pages, block_table, num_heads, 
     by ``qk_norm_kv_write`` or by the decode kernel itself.  bfloat16 with a tiled head size and values of the
     keys' size runs on the tensor cores as plain attention does: the split-context decode
     kernel for steps of single tokens, the tcgen05 kernel with one tile of query rows a block
-    for portions, the ``mma.sync`` kernel for the sizes that one does not take.  Everything
+    for portions, the ``mma.sync`` kernel for the sizes that one does not take.  Other sizes
+    that are multiples of 8, with a sink or a gate as the only options, run on the same two
+    kernels compiled for sizes of their own (``sized_attention_supported``).  Everything
     else, and float32, runs one warp a (token, head)."""
+    value_dim = options.value_dim or head_dim
     tiled = (ATTENTION_OPTIONS_TILED and qkv.dtype == torch.bfloat16 and head_dim in TILED_HEAD_DIMS
              and options.tiled)
     decode = tiled and ctx.decode_only and num_heads // num_kv_heads <= 16
+    sized = None
+    if not tiled and ATTENTION_OPTIONS_TILED and qkv.dtype == torch.bfloat16 \
+            and qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0:
+        sized = sized_attention_supported(options, num_heads, num_kv_heads, head_dim, value_dim, page_size,
+                                          ctx.decode_only)
     fused = None
     if isinstance(prepare, RotateNormPrepare):
         pr = prepare
         qk_rotate_norm_write(qkv, pr.cos, pr.sin, ctx.positions, ctx.seq_of_token, block_table, k_pages,
-                             v_pages, num_heads, num_kv_heads, head_dim, options.value_dim or head_dim,
+                             v_pages, num_heads, num_kv_heads, head_dim, value_dim,
                              page_size, pr.norm, pr.q_weight, pr.k_weight, pr.eps, pr.value_col,
                              write_cache=pr.write, pairing=pr.pairing)
     elif prepare is not None:
         wq, wk, eps, coef, every, write = prepare
-        if decode and write and ATTENTION_DECODE_QK_NORM and qkv.is_contiguous():
+        alone = not write and wk is None and wq is not None        # the rows hold queries alone
+        if (write or alone) and ATTENTION_DECODE_QK_NORM and qkv.is_contiguous() \
+                and (decode or (sized == "decode" and not every)):
             fused = (wq, wk, eps, coef, every)
         else:
             qk_norm_kv_write(qkv, ctx.positions, ctx.seq_of_token, block_table, k_pages, v_pages, num_heads,
-                             num_kv_heads, head_dim, options.value_dim or head_dim, page_size, wq, wk, eps,
+                             0 if alone else num_kv_heads, head_dim, value_dim, page_size, wq, wk, eps,
                              coef, every, write_cache=write)
     if tiled:
         if decode:
             splits = ctx.extras.get("decode_splits")
             if splits is None:
-                splits = decode_splits(ctx.num_seqs, num_kv_heads, ctx.max_context_len, head_dim)
+                splits = decode_splits(ctx.num_seqs, num_kv_heads, _keys_seen(ctx, window), head_dim)
             return attention_decode_bf16(qkv, k_pages, v_pages, block_table, ctx.positions, num_heads,
                                          num_kv_heads, head_dim, page_size, window, scale, splits,
-                                         None, fused is not None,
+                                         None, fused is not None and bool(prepare[5]),
                                          decode_warps(ctx.num_seqs * num_kv_heads, splits, head_dim,
-                                                      ctx.max_context_len), options=options, qk_norm=fused)
+                                                      _keys_seen(ctx, window)), options=options, qk_norm=fused)
         if (ATTENTION_TCGEN05 and ctx.max_tokens_per_seq >= 16
                 and tc_attention_supported(num_heads, num_kv_heads, head_dim, page_size)):
             tiles = _step_tiles(ctx, 128 // (num_heads // num_kv_heads), True, qkv.device)
@@ -1415,8 +1434,47 @@ def _attention_with_options(ctx, qkv, k_pages, v_pages, block_table, num_heads, 
         return attention_prefill_bf16(qkv, k_pages, v_pages, block_table, tiles, ctx.cu_tokens,
                                       ctx.start_pos, num_heads, num_kv_heads, head_dim, page_size,
                                       window, scale, options=options)
+    if sized is not None:
+        out = torch.empty((qkv.shape[0], num_heads * value_dim), dtype=qkv.dtype, device=qkv.device)
+        cache = LayerPages(k_pages, v_pages, page_size)
+        if sized == "decode":
+            splits = ctx.extras.get("decode_splits")
+            if splits is None:
+                splits = decode_splits(ctx.num_seqs, num_kv_heads, _keys_seen(ctx, window), max(head_dim, value_dim))
+            _pooled_decode(ctx, qkv, cache, block_table, None, num_heads, num_kv_heads, head_dim, value_dim,
+                           int(window or 0), 0, scale, out, 1.0, int(splits), options,
+                           None if fused is None else fused[:3], fused is not None and bool(prepare[5]))
+        else:
+            _pooled_prefill_tc(ctx, qkv, cache, block_table, None, num_heads, num_kv_heads, head_dim, value_dim,
+                               int(window or 0), 0, scale, out, 1.0, options)
+        return out
     return attention_generic(qkv, k_pages, v_pages, block_table, ctx.seq_of_token, ctx.positions,
                              num_heads, num_kv_heads, head_dim, page_size, window, scale, options)
+
+
+def _keys_seen(ctx, window: Optional[int]) -> int:
+    """Most keys a token of the step sees."""
+    return min(ctx.max_context_len, int(window)) if window else ctx.max_context_len
+
+
+def sized_attention_supported(options: AttentionOptions, num_heads: int, num_kv_heads: int, head_dim: int,
+                              value_dim: int, page_size: int, decode: bool) -> Optional[str]:
+    """"decode" or "portions" where the tensor-core kernels compiled for key and value sizes of
+    their own take these sizes and options, else None."""
+    if options.slopes is not None or options.bias_table is not None or options.keep_first:
+        return None
+    if decode and pooled_decode_supported(num_heads, num_kv_heads, head_dim, value_dim):
+        return "decode"
+    return "portions" if pooled_tc_supported(num_heads, num_kv_heads, head_dim, value_dim, page_size) else None
+
+
+class LayerPages:
+    """Key and value pages as the kernels for sizes of their own take them."""
+
+    __slots__ = ("k_pages", "v_pages", "page_size")
+
+    def __init__(self, k_pages: torch.Tensor, v_pages: torch.Tensor, page_size: int) -> None:
+        self.k_pages, self.v_pages, self.page_size = k_pages, v_pages, page_size
 
 
 class RotateNormPrepare:
@@ -1507,14 +1565,17 @@ def qk_norm_kv_write(rows: torch.Tensor, positions: torch.Tensor, seq_of_token: 
     whatever follows): every q head becomes q / rms(q) * q_weight * (1 + temp_coef *
     ln(floor((p + 1) / temp_every) + 1)) in place (p the token's position; ``temp_every`` 0: no
     such factor; weights None: no norm), every k head k / rms(k) * k_weight at the token's
-    place in the key pages, every v head goes to the value pages.  float32 arithmetic."""
+    place in the key pages, every v head goes to the value pages.  Rows that hold queries alone
+    (``num_kv_heads`` 0, no key weight) only norm those.  float32 arithmetic."""
     _check(rows, "rows", None, 2)
     T, ld = rows.shape
     _check(positions, "positions", torch.int32, 1)
     _check(seq_of_token, "seq_of_token", torch.int32, 1)
     _check(block_table, "block_table", torch.int32, 2)
-    if (q_weight is None) != (k_weight is None):
+    if num_kv_heads and (q_weight is None) != (k_weight is None):
         raise KernelError("query and key norm come together")
+    if not num_kv_heads and write_cache:
+        raise KernelError("rows without keys have nothing to store")
     for name, w in (("q_weight", q_weight), ("k_weight", k_weight)):
         if w is not None:
             _check(w, name, torch.float32, 1)
@@ -1657,6 +1718,42 @@ def rmsnorm_add(residual: torch.Tensor, y: Optional[torch.Tensor], weight: Optio
     if copy_dtype is None:
         return None
     return residual if copy is None else copy
+
+
+def rmsnorm_add_rmsnorm(residual: torch.Tensor, y: torch.Tensor, weight1: torch.Tensor, eps1: float,
+                        weight2: torch.Tensor, eps2: float, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``residual += y / sqrt(mean(y^2) + eps1) * weight1`` row by row, in float32 and in place, and
+    the new rows' own norm, x / sqrt(mean(x^2) + eps2) * weight2, in y's dtype (a block that norms
+    before AND after a sublayer: the norm after this one and the norm before the next in one
+    launch).  With ``rows`` (int32) only those rows are computed, into [len(rows), H], and the
+    residual is left as it was."""
+    _check(residual, "residual", torch.float32, 2)
+    _check(y, "y", None, 2)
+    n, H = residual.shape
+    for name, w in (("weight1", weight1), ("weight2", weight2)):
+        _check(w, name, torch.float32, 1)
+        if w.numel() != H:
+            raise KernelError(f"{name} has {w.numel()} entries for rows of {H}")
+    if tuple(y.shape) != (n, H):
+        raise KernelError(f"y {tuple(y.shape)} does not match residual {(n, H)}")
+    if rows is not None:
+        _check(rows, "rows", torch.int32, 1)
+    n_out = n if rows is None else rows.numel()
+    out = torch.empty((n_out, H), dtype=y.dtype, device=y.device)
+    f = _fn("elementwise", "hb_rmsnorm_add_rmsnorm",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int,
+             c_void_p])
+    _run(f(_p(out), _p(residual), _p(y), _p(weight1), _p(weight2), _p(rows), n_out, H, float(eps1), float(eps2),
+           _dt(y.dtype), _stream()), "rmsnorm_add_rmsnorm")
+    return out
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``x = cap * tanh(x / cap)`` in place (float32, contiguous); returns x."""
+    _check(x, "x", torch.float32)
+    f = _fn("elementwise", "hb_softcap", [c_void_p, ctypes.c_long, c_float, c_void_p])
+    _run(f(_p(x), x.numel(), float(cap), _stream()), "softcap")
+    return x
 
 
 def scaled_sum_rmsnorm(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
@@ -1826,8 +1923,10 @@ def linear_rows(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 def latent_attention(ctx, q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tensor,
                      block_table: torch.Tensor, rank: int, rot: int, page_size: int,
-                     scale: float) -> torch.Tensor:
-    """Causal attention of every token of the step over its request's latent rows.  ``q_lat``
+                     scale: float, window: Optional[int] = None,
+                     sink_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention of every token of the step over its request's latent rows, all of them or
+    the last ``window``; ``sink_values`` (float32 [heads]): a key of that score without a value.  ``q_lat``
     [T, heads, rank] and ``q_rot`` [T, heads, rot] are views with a contiguous last dimension;
     ``pages`` [pages, 1, page_size, rank + rot].  Returns [T, heads, rank] (softmax-weighted
     sums of the rows' first ``rank`` values).  ``ctx`` gives seq_of_token and positions, and
@@ -1844,6 +1943,11 @@ def latent_attention(ctx, q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch
     if rank > 512 or rank + rot > 1024:
         raise KernelError(f"latent rank {rank} (at most 512) or row {rank + rot} (at most 1024) is not supported")
     T, H = q_lat.shape[:2]
+    window = int(window or 0)
+    if sink_values is not None:
+        _check(sink_values, "sink_values", torch.float32, 1)
+        if sink_values.numel() != H:
+            raise KernelError(f"{sink_values.numel()} sink values for {H} heads")
     out = torch.empty((T, H, rank), dtype=q_lat.dtype, device=q_lat.device)
     if LATENT_ATTENTION_TENSOR_CORES and q_lat.dtype == torch.bfloat16 and rank % 32 == 0 and rot % 16 == 0:
         # 32 query rows a block: (token, head) pairs of one request, which share every key
@@ -1853,7 +1957,8 @@ def latent_attention(ctx, q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch
         blocks = tiles.shape[0] * -(-H // hpb)
         n_splits = 1
         if blocks < sm_count():
-            n_splits = max(1, min(32, ctx.max_context_len // 256, -(-2 * sm_count() // blocks)))
+            keys = min(ctx.max_context_len, window + tpt - 1) if window else ctx.max_context_len
+            n_splits = max(1, min(32, keys // 256, -(-2 * sm_count() // blocks)))
         part_acc = part_ml = None
         if n_splits > 1:
             part_acc = torch.empty((T * H, n_splits, rank), dtype=torch.float32, device=q_lat.device)
@@ -1861,19 +1966,19 @@ def latent_attention(ctx, q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch
         f = _fn("latent_attention", "hb_latent_attention_mma",
                 [c_void_p, c_void_p, c_void_p, c_void_p, _LONG, _LONG, c_void_p, _LONG, _LONG, c_void_p,
                  c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                 c_int, c_int, c_float, c_int, c_void_p])
+                 c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p])
         _run(f(_p(out), _p(part_acc), _p(part_ml), _p(q_lat), q_lat.stride(0), q_lat.stride(1), _p(q_rot),
                q_rot.stride(0), q_rot.stride(1), _p(pages), _p(block_table), block_table.shape[1],
                _p(tiles), tiles.shape[0], _p(ctx.cu_tokens), _p(ctx.start_pos), T, H, hpb, tpt, rank, rot,
-               page_size, float(scale), n_splits, _stream()), "latent_attention_mma")
+               page_size, float(scale), n_splits, window, _p(sink_values), _stream()), "latent_attention_mma")
         return out
     f = _fn("latent_attention", "hb_latent_attention",
             [c_void_p, c_void_p, _LONG, _LONG, c_void_p, _LONG, _LONG, c_void_p, c_void_p, c_int, c_void_p,
-             c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
+             c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p])
     _run(f(_p(out), _p(q_lat), q_lat.stride(0), q_lat.stride(1), _p(q_rot), q_rot.stride(0),
            q_rot.stride(1), _p(pages), _p(block_table), block_table.shape[1], _p(ctx.seq_of_token),
-           _p(ctx.positions), T, H, rank, rot, page_size, float(scale), _dt(q_lat.dtype), _stream()),
-         "latent_attention")
+           _p(ctx.positions), T, H, rank, rot, page_size, float(scale), window, _p(sink_values),
+           _dt(q_lat.dtype), _stream()), "latent_attention")
     return out
 
 
@@ -2137,13 +2242,84 @@ def linear_attention(ctx, rows: torch.Tensor, offsets, state: torch.Tensor, deca
                _stream()), "linear_attention_scan")
         if fused:
             return
+    parts = heads if norm == "head" else 1
+    _linear_gate_norm(out, o, rows, g_off, norm_weight, parts, heads * dv // parts, gate, eps, factor)
+
+
+def _linear_gate_norm(out, o, rows, g_off, weight, parts, width, gate, eps, factor) -> None:
+    """``out`` = factor * o / rms(o) (* weight) * gate: ``parts`` norms of ``width`` values a token,
+    the gate's argument in the columns of ``rows`` from ``g_off`` on."""
     f = _fn("linear_attention", "hb_la_gate_norm",
             [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
              c_int, c_void_p])
-    parts = heads if norm == "head" else 1
-    _run(f(_p(out), out.stride(0), _p(o), _p(rows) + g_off * rows.element_size(), rows.shape[1], _p(norm_weight), T,
-           parts, heads * dv // parts, gk, float(eps), float(factor), _dt(rows.dtype), _stream()),
-         "linear_attention_gate_norm")
+    _run(f(_p(out), out.stride(0), _p(o), _p(rows) + g_off * rows.element_size(), rows.shape[1], _p(weight),
+           out.shape[0], parts, width, LINEAR_ATTENTION_GATES[gate], float(eps), float(factor), _dt(rows.dtype),
+           _stream()), "linear_attention_gate_norm")
+
+
+# ------------------------------------------------------------------ linear attention, decays per channel and token
+def gated_linear_attention(ctx, rows: torch.Tensor, offsets, w2: torch.Tensor, bias: torch.Tensor, tau: float,
+                           state: torch.Tensor, heads: int, dk: int, dv: int, norm_weight: torch.Tensor, eps: float,
+                           out: torch.Tensor, q_scale: float = 1.0, factor: float = 1.0) -> None:
+    """S <- diag(a) S + k v^T, o = S^T q per head over the step's tokens, request by request, from
+    the state each request's slot holds (``state`` [slots, heads * dk * dv] float32, rows may be
+    strided; left updated), with a decay per token and key channel, a = sigmoid(W2 x + bias)^(1 /
+    ``tau``) (``w2`` [heads * dk, R] in the rows' dtype, ``bias`` float32), then o / rms(o) *
+    ``norm_weight`` per head times silu(gate) times ``factor`` into ``out`` [T, heads * dv] (rows may
+    be strided).  ``rows`` [T, .] holds q, k (heads x dk), v and the
+    gate (heads x dv) and x (R columns) at the column ``offsets``; q is multiplied by ``q_scale``.
+    Float32 in between.
+
+    Steps of few tokens a request run token by token, others in chunks of 64 tokens that are
+    taken in parallel."""
+    _check(rows, "rows", None, 2)
+    T = rows.shape[0]
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 \
+            or state.shape[1] != heads * dk * dv or not state.is_cuda:
+        raise KernelError(f"state {tuple(state.shape)} does not fit {heads} heads of {dk} x {dv}")
+    if dk > 256 or dv > 256:
+        raise KernelError(f"heads of {dk} x {dv} are not supported (at most 256)")
+    _check(w2, "w2", rows.dtype, 2)
+    _check(bias, "bias", torch.float32, 1)
+    _check(norm_weight, "norm_weight", torch.float32, 1)
+    rank = w2.shape[1]
+    if w2.shape[0] != heads * dk or bias.numel() != heads * dk or norm_weight.numel() != dv or rank > 256:
+        raise KernelError(f"w2 {tuple(w2.shape)}, bias {bias.numel()} and norm weight {norm_weight.numel()} do not fit "
+                          f"{heads} heads of {dk} x {dv} (a rank of at most 256)")
+    offs = tuple(int(o) for o in offsets)
+    for o, n in zip(offs, (heads * dk, heads * dk, heads * dv, heads * dv, rank)):
+        if o < 0 or o + n > rows.shape[1]:
+            raise KernelError(f"rows of {rows.shape[1]} columns do not hold the columns {offs}")
+    if not tau > 0:
+        raise KernelError(f"tau {tau} must be positive")
+    _check_out_rows(out, T, heads * dv, rows)
+    f32 = dict(dtype=torch.float32, device=rows.device)
+    most = getattr(ctx, "max_tokens_per_seq", T)
+    if most > LINEAR_ATTENTION_SCAN_TOKENS:
+        tiles = _step_tiles(ctx, LINEAR_ATTENTION_CHUNK, False, rows.device)
+        n = tiles.shape[0]
+        q, k = torch.empty((T, heads, dk), **f32), torch.empty((T, heads, dk), **f32)
+        decays = torch.empty((n, heads, 5, dk), **f32)
+        diag = torch.empty((n, heads, LINEAR_ATTENTION_CHUNK, 16), **f32)
+        sums = torch.empty((n, heads, dk, dv), **f32)
+        f = _fn("gated_linear_attention", "hb_gla_chunked",
+                [c_void_p, c_int] + [c_void_p] * 6 + [c_int] * 6 + [c_void_p, c_void_p, c_int, c_float, c_float, c_void_p,
+                 _LONG, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_int,
+                 c_void_p])
+        _run(f(_p(out), out.stride(0), _p(q), _p(k), _p(decays), _p(diag), _p(sums), _p(rows), rows.shape[1], *offs,
+               _p(w2), _p(bias), rank, 1.0 / float(tau), float(q_scale), _p(state), state.stride(0), _p(tiles), n,
+               _p(ctx.cu_tokens), _p(ctx.slots), ctx.num_seqs, heads, dk, dv, _p(norm_weight), float(eps),
+               float(factor), _dt(rows.dtype), _stream()), "gated_linear_attention_chunked")
+        return
+    o = torch.empty((T, heads * dv), **f32) if dv > 128 else None
+    f = _fn("gated_linear_attention", "hb_gla_scan",
+            [c_void_p, c_void_p, c_int, c_void_p] + [c_int] * 6 + [c_void_p, c_void_p, c_int, c_float, c_float, c_void_p,
+             _LONG, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_int, c_void_p])
+    _run(f(_p(o), _p(out), out.stride(0), _p(rows), rows.shape[1], *offs, _p(w2), _p(bias), rank, 1.0 / float(tau),
+           float(q_scale), _p(state), state.stride(0), _p(ctx.cu_tokens), _p(ctx.slots), T, ctx.num_seqs, heads, dk, dv,
+           _p(norm_weight), float(eps), float(factor), _dt(rows.dtype), _stream()), "gated_linear_attention_scan")
+    if o is not None:
+        _linear_gate_norm(out, o, rows, offs[3], norm_weight, heads, dv, "silu", eps, factor)
 
 
 # ------------------------------------------------------------------ window attention with pooled blocks
@@ -2306,14 +2482,31 @@ def _pooled_args(q, cache, table, ptable, num_kv_heads, head_dim, value_dim, win
     return (_p(pk), _p(pv), pk.shape[0], _p(pt), pt.shape[1], pool)
 
 
+def _sized_option_args(options: AttentionOptions, tokens: int, num_heads: int, like: torch.Tensor, value_dim: int):
+    """Sink and gate as the kernels for sizes of their own take them."""
+    options.check(tokens, num_heads, like, value_dim)
+    return (int(options.sink), _p(options.sink_values), _p(options.gate), options.gate_stride,
+            1 if options.gate_wide else 0)
+
+
 def _pooled_decode(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_dim, value_dim, window, pool, scale,
-                   out, factor, n_splits) -> None:
-    """Token i is the one new token of request i; the context in ``n_splits`` slices."""
+                   out, factor, n_splits, options: AttentionOptions = _NO_OPTIONS, qk_norm=None,
+                   write_cache: bool = False) -> None:
+    """Token i is the one new token of request i; the context in ``n_splits`` slices.
+    ``write_cache``: the rows of q hold the token's k and v behind the queries, and the kernel
+    stores them; ``qk_norm`` = (q weight, k weight, eps): q (and that k) still lacks its norm."""
     S = q.shape[0]
     pk, pv, _n, pt, pstride, pool = _pooled_args(q, cache, table, ptable, num_kv_heads, head_dim, value_dim, window, pool)
     _check_out_rows(out, S, num_heads * value_dim, q)
-    if q.shape[1] != num_heads * head_dim or table.shape[0] != S:
+    columns = num_heads * head_dim + (num_kv_heads * (head_dim + value_dim) if write_cache else 0)
+    if q.shape[1] < columns or table.shape[0] != S:
         raise KernelError(f"decode attention needs one token per request and {num_heads} heads of {head_dim}")
+    wq, wk, eps = qk_norm if qk_norm is not None else (None, None, 0.0)
+    for name, w in (("q norm weight", wq), ("k norm weight", wk)):
+        if w is not None:
+            _check(w, name, torch.float32, 1)
+            if w.numel() != head_dim:
+                raise KernelError(f"{name} has {w.numel()} entries for heads of {head_dim}")
     part_o = part_ml = None
     one_round = n_splits <= 8 and S * num_kv_heads <= pooled_cluster_capacity(head_dim, value_dim, n_splits)
     if n_splits > 8 or (n_splits > 1 and not (ATTENTION_CLUSTER_MERGE and one_round)):
@@ -2322,29 +2515,31 @@ def _pooled_decode(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_d
     f = _fn("attention_pooled", "hb_attention_pooled_decode",
             [c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
              c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_float, c_int, c_void_p])
+             c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p])
     _run(f(_p(out), out.stride(0), float(factor), _p(part_o), _p(part_ml), _p(q), q.stride(0), _p(cache.k_pages),
            _p(cache.v_pages), _p(table), table.shape[1], pk, pv, pt, pstride, pool, _p(ctx.positions), S, num_heads,
-           num_kv_heads, head_dim, value_dim, cache.page_size, int(window), float(scale), n_splits, _stream()),
-         "attention_pooled_decode")
+           num_kv_heads, head_dim, value_dim, cache.page_size, int(window), float(scale), n_splits,
+           *_sized_option_args(options, S, num_heads, q, value_dim), 1 if write_cache else 0, _p(wq), _p(wk),
+           float(eps), _stream()), "attention_pooled_decode")
 
 
 def _pooled_prefill_tc(ctx, q, cache, table, ptable, num_heads, num_kv_heads, head_dim, value_dim, window, pool,
-                       scale, out, factor) -> None:
+                       scale, out, factor, options: AttentionOptions = _NO_OPTIONS) -> None:
     pk, pv, pn, pt, pstride, pool = _pooled_args(q, cache, table, ptable, num_kv_heads, head_dim, value_dim, window, pool)
     _check_out_rows(out, q.shape[0], num_heads * value_dim, q)
-    if q.shape[1] != num_heads * head_dim:
+    if q.shape[1] < num_heads * head_dim:
         raise KernelError(f"q has {q.shape[1]} columns for {num_heads} heads of {head_dim}")
     tiles = _step_tiles(ctx, 128 // (num_heads // num_kv_heads), True, q.device)
     _scratch, _tickets, err = _gemm_workspace(q.device)
     f = _fn("attention_tc_pooled", "hb_attention_pooled_prefill_tc",
             [c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p, c_int, c_void_p,
              c_void_p, ctypes.c_longlong, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-             c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+             c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
     _run(f(_p(out), out.stride(0), float(factor), _p(q), q.stride(0), _p(cache.k_pages), _p(cache.v_pages),
            cache.k_pages.shape[0], _p(table), table.shape[1], pk, pv, pn, pt, pstride, pool, _p(tiles), tiles.shape[0],
            _p(ctx.cu_tokens), _p(ctx.start_pos), num_heads, num_kv_heads, head_dim, value_dim, cache.page_size,
-           int(window), float(scale), _p(err), _stream()), "attention_pooled_prefill_tc")
+           int(window), float(scale), _p(err), *_sized_option_args(options, q.shape[0], num_heads, q, value_dim),
+           _stream()), "attention_pooled_prefill_tc")
 
 
 # ------------------------------------------------------------------ routed experts

@@ -42,9 +42,11 @@ class _StepGraph:
         # rows belongs to a part that cuts its key range itself)
         kv_specs = [s for s in cache.specs if s.planes == 2]
         if self.decode and kv_specs:
+            # most keys a token of any layer sees
+            keys = max(min(core.graph_max_context, s.window + s.keep_first) if s.window else core.graph_max_context
+                       for s in kv_specs)
             self.ctx.extras["decode_splits"] = ops.decode_splits(
-                num_seqs, max(s.num_kv_heads for s in kv_specs), core.graph_max_context,
-                max(s.head_dim for s in kv_specs))
+                num_seqs, max(s.num_kv_heads for s in kv_specs), keys, max(s.head_dim for s in kv_specs))
         self.ctx.extras["tile_provider"] = self._tiles
         self._tile_buffers = {}          # (tile, longest first) -> (pinned rows, device rows)
         self._rows_kept = {}             # block-table rows of the staging buffer that are still right

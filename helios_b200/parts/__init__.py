@@ -1,5 +1,5 @@
 from .base import (Block, DeferredNorm, FeedForward, InputStage, LayerCache, Mixer, Norm, OutputStage, PagedCacheSpec, Part,
-                   PendingSum, PositionEncoding, StateSpec, StreamStage, WeightSpec, known_parts, part_class,
+                   PendingNormed, PendingSum, PositionEncoding, StateSpec, StreamStage, WeightSpec, known_parts, part_class,
                    register_part, settle)
 from .norm import LayerNorm, RMSNorm
 from .rotary import RotaryEncoding, rotary_frequencies, yarn_attention_factor, yarn_frequencies
@@ -11,9 +11,10 @@ from .delta_rule import GatedDeltaMixer
 from .ssm import SelectiveStateMixer
 from .side_by_side import BranchMixer, SideBySideMixer
 from .linear_attention import FixedDecayMixer
+from .gated_linear_attention import ChannelDecayMixer
 from .pooled_window import PooledWindowAttention
 from .embedding import LearnedPositions, NormedHead, OutputHead, TokenEmbedding
-from .block import NormedSumBlock, ParallelBlock, PostNormBlock, PreNormBlock
+from .block import NormedSumBlock, ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .stream import StreamInputMix
 from .plan import ModelPlan, Run
 
@@ -25,4 +26,4 @@ __all__ = ["Block", "DeferredNorm", "FeedForward", "InputStage", "OutputStage", 
            "yarn_frequencies", "yarn_attention_factor", "PendingSum", "StreamStage", "settle", "LayerNorm",
            "SinkGQAAttention", "distance_slopes", "LearnedPositions", "ParallelBlock", "StreamInputMix",
            "SelectiveStateMixer", "BranchMixer", "SideBySideMixer", "FixedDecayMixer",
-           "PooledWindowAttention", "NormedSumBlock"]
+           "PooledWindowAttention", "NormedSumBlock", "SandwichBlock", "PendingNormed", "ChannelDecayMixer"]

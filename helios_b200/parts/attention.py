@@ -152,6 +152,11 @@ class SinkGQAAttention(Mixer):
     ``sink="learned"``    the sink's score is a learned number a head (tensor ``sink``) instead of 0
     ``keep_first``        with ``window``: the request's first ``keep_first`` tokens stay visible
     ``head_gate="wide"``  W_g has a row per output VALUE, and every value its own gate
+    ``own_keys=False``    the mixer has no W_k and W_v (nor their norm and biases) and stores nothing; it
+                          attends the keys, as their pages hold them, and values that ANOTHER layer
+                          keeps (the plan names that layer's cache for this one's run)
+    ``cache_window``      tokens whose keys and values stay in the pages where that is more than
+                          ``window``: the widest window of the layers that attend them
     ``qk_bias``, ``out_bias``  biases of the q and k projections (and v, where it exists) and of
                           the output projection (``<name>.b``)
     """
@@ -163,7 +168,9 @@ class SinkGQAAttention(Mixer):
                  names=("q", "k", "v", "o", "g", "q.norm", "k.norm"), values: str = "projected",
                  position=None, rotary_dim: int = 0, distance_table=None, keep_first: int = 0,
                  qk_bias: bool = False, out_bias: bool = False, rel_name: str = "rel",
-                 sink_name: str = "sink", bias_suffix: str = ".b", rotary_pairing: str = "halves") -> None:
+                 sink_name: str = "sink", bias_suffix: str = ".b", rotary_pairing: str = "halves",
+                 own_keys: bool = True, cache_window: Optional[int] = -1) -> None:
+        """``cache_window``: -1: ``window``; None: every token's keys and values stay."""
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} KV heads")
         value_dim = value_dim or head_dim
@@ -182,6 +189,12 @@ class SinkGQAAttention(Mixer):
             raise ValueError(f"a rotation needs an encoding and an even rotary_dim of at most {head_dim}")
         if keep_first and not window:
             raise ValueError("first tokens are kept beside a window only")
+        if not own_keys and (values == "keys" or position is not None or qk_norm not in (True, False)):
+            raise ValueError("a mixer without keys of its own rotates nothing and norms its queries per head")
+        self.own_keys = bool(own_keys)
+        self.cache_window = window if cache_window == -1 else cache_window
+        if self.cache_window is not None and (window is None or self.cache_window < window):
+            raise ValueError(f"a cache of {self.cache_window} tokens does not hold a window of {window}")
         self.width, self.num_heads, self.num_kv_heads = width, num_heads, num_kv_heads
         self.head_dim, self.value_dim = head_dim, value_dim
         self.scale, self.eps = float(scale), float(eps)
@@ -199,19 +212,23 @@ class SinkGQAAttention(Mixer):
         self.w_in = self.b_in = self.w_o = self.b_o = self.q_weight = self.k_weight = self.slopes = None
         self.bias_rows = self.bias_rows_t = self.sink_values = None
         q, kv = num_heads * head_dim, num_kv_heads * head_dim
+        self._projected = ("q", "k", "v") if values == "projected" else ("q", "k")
+        if not own_keys:
+            self._projected = ("q",)
         self._value_col = q + kv if values == "projected" else None
-        self._gate_col = q + kv + (num_kv_heads * value_dim if values == "projected" else 0)
+        self._gate_col = q if not own_keys else q + kv + (num_kv_heads * value_dim if values == "projected" else 0)
         # the launch that readies q, k and v: the one with weights and temperature, or the one
         # that also rotates, norms without weights and may take the values from the keys
         self._rotate_prepare = values == "keys" or position is not None or qk_norm in ("plain", "row")
         if self._rotate_prepare and self.q_temperature is not None:
             raise ValueError("a query temperature goes with weighted q/k norms and projected values only")
-        self._tiled_options = value_dim == head_dim
+        # the kernels for key and value sizes of their own take a sink and a gate
+        self._tiled_options = slopes is None and distance_table is None and not keep_first
 
     # ---------------------------------------------------------------- what it keeps
     def cache_spec(self) -> PagedCacheSpec:
         vd = None if self.value_dim == self.head_dim else self.value_dim
-        return PagedCacheSpec(self.num_kv_heads, self.head_dim, self.window, value_dim=vd,
+        return PagedCacheSpec(self.num_kv_heads, self.head_dim, self.cache_window, value_dim=vd,
                               keep_first=self.keep_first)
 
     def kernel_libraries(self, dtype):
@@ -223,21 +240,23 @@ class SinkGQAAttention(Mixer):
     def weight_specs(self) -> Dict[str, WeightSpec]:
         nq, nk, nv, no, ng, nqn, nkn = self.names
         q, kv = self.num_heads * self.head_dim, self.num_kv_heads * self.head_dim
-        specs = {nq: WeightSpec((q, self.width)), nk: WeightSpec((kv, self.width)),
-                 no: WeightSpec((self.width, self.num_heads * self.value_dim))}
-        if self.values == "projected":
+        specs = {nq: WeightSpec((q, self.width)), no: WeightSpec((self.width, self.num_heads * self.value_dim))}
+        if "k" in self._projected:
+            specs[nk] = WeightSpec((kv, self.width))
+        if "v" in self._projected:
             specs[nv] = WeightSpec((self.num_kv_heads * self.value_dim, self.width))
         if self.head_gate:
             rows = self.num_heads * (self.value_dim if self.head_gate == "wide" else 1)
             specs[ng] = WeightSpec((rows, self.width))
         if self.qk_norm is True:
             specs[nqn] = WeightSpec((self.head_dim,), kind="vector", init="ones_jitter")
-            specs[nkn] = WeightSpec((self.head_dim,), kind="vector", init="ones_jitter")
+            if self.own_keys:
+                specs[nkn] = WeightSpec((self.head_dim,), kind="vector", init="ones_jitter")
         elif self.qk_norm == "row":
             specs[nqn] = WeightSpec((q,), kind="vector", init="ones_jitter")
             specs[nkn] = WeightSpec((kv,), kind="vector", init="ones_jitter")
         if self.qk_bias:
-            for n in (nq, nk) + ((nv,) if self.values == "projected" else ()):
+            for n in [dict(q=nq, k=nk, v=nv)[c] for c in self._projected]:
                 specs[n + self.bias_suffix] = WeightSpec((specs[n].shape[0],), kind="vector", init="normal")
         if self.out_bias:
             specs[no + self.bias_suffix] = WeightSpec((self.width,), kind="vector", init="normal")
@@ -250,7 +269,7 @@ class SinkGQAAttention(Mixer):
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         nq, nk, nv, no, ng, nqn, nkn = self.names
-        order = [nq, nk] + ([nv] if self.values == "projected" else [])
+        order = [dict(q=nq, k=nk, v=nv)[c] for c in self._projected]
         mats = [tensors[n] for n in order]
         if self.head_gate:
             mats.append(tensors[ng])
@@ -268,7 +287,8 @@ class SinkGQAAttention(Mixer):
         if self.out_bias:
             self.b_o = tensors[no + self.bias_suffix].contiguous()
         if self.qk_norm in (True, "row"):
-            self.q_weight, self.k_weight = tensors[nqn].contiguous(), tensors[nkn].contiguous()
+            self.q_weight = tensors[nqn].contiguous()
+            self.k_weight = tensors[nkn].contiguous() if self.own_keys else None
         if self.slope_values is not None:
             self.slopes = torch.tensor(self.slope_values, dtype=torch.float32, device=self.w_o.device)
         if self.distance_table is not None:
@@ -299,7 +319,9 @@ class SinkGQAAttention(Mixer):
                                             cache.write, pairing=self.rotary_pairing)
         else:
             coef, every = self.q_temperature or (0.0, 0)
-            prepare = (self.q_weight, self.k_weight, self.eps, coef, every, cache.write)
+            prepare = (self.q_weight, self.k_weight, self.eps, coef, every, cache.write and self.own_keys)
+            if not self.own_keys and self.q_weight is None and not every:
+                prepare = None                 # the queries are ready, and there is nothing to store
         attn = ops.attention(ctx, rows, cache.k_pages, cache.v_pages, table, self.num_heads,
                              self.num_kv_heads, self.head_dim, cache.page_size, self.window, self.scale,
                              options=self._options(gate), prepare=prepare)

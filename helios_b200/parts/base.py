@@ -103,7 +103,7 @@ class Norm(Part):
                     out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``residual += delta`` in float32 (in place, unless ``rows`` selects) and the
         normed rows in ``out_dtype``.  The default does it in two steps."""
-        if isinstance(delta, PendingSum):
+        if isinstance(delta, (PendingSum, PendingNormed)):
             settle(residual, delta)          # the default knows no better than to add first
             delta = None
         if rows is not None:
@@ -190,9 +190,22 @@ class PendingSum:
     mult: float = 1.0
 
 
+@dataclass
+class PendingNormed:
+    """A block's output that is still to be NORMED and added to the residual stream:
+    ``residual += norm(y)`` (float32).  A block that norms after a sublayer as well as before the
+    next one returns it in the place of ``delta``; a norm that knows how (``RMSNorm.add_forward``)
+    does both norms and the add in its own kernel, anyone else calls ``settle`` first."""
+    y: torch.Tensor
+    norm: "Norm"
+
+
 def settle(residual: torch.Tensor, delta) -> None:
     """Add whatever is pending to the float32 residual stream, in place."""
     if delta is None:
+        return
+    if isinstance(delta, PendingNormed):
+        delta.norm.add_normed(residual, delta.y, torch.float32)
         return
     if isinstance(delta, PendingSum):
         from ..csrc import ops

@@ -10,8 +10,8 @@ from typing import List, Optional, Tuple
 
 import torch
 
-from .base import (Block, DeferredNorm, FeedForward, LayerCache, Mixer, Norm, Part, PendingSum, WeightSpec,
-                   register_part)
+from .base import (Block, DeferredNorm, FeedForward, LayerCache, Mixer, Norm, Part, PendingNormed, PendingSum,
+                   WeightSpec, register_part, settle)
 
 
 class PreNormBlock(Block):
@@ -113,7 +113,7 @@ class PostNormBlock(Block):
             raise ValueError("a post-norm block takes no deferred norm")
         kept = ctx.step_tables.pop(self._COPY, None)
         if delta is not None:
-            residual.add_(delta.float())
+            settle(residual, delta)
             kept = None
         if kept is not None and kept[0] == ctx.run_index - 1:
             h = kept[1]
@@ -148,6 +148,50 @@ class NormedSumBlock(PostNormBlock):
 
 
 register_part("block", "normed_sum", NormedSumBlock)
+
+
+class SandwichBlock(Block):
+    """x + norm_b(mixer(norm_a(x))), then x + norm_b'(feed_forward(norm_a'(x))): a norm before AND after
+    each sublayer.  The feed-forward, with its two norms, may be absent.  Residual sum and norms are
+    float32.  What a sublayer returns is left as a ``PendingNormed``: the norm that meets the stream
+    next (the feed-forward's, the next block's first, the final norm) does the norm after the
+    sublayer, the add and itself in one kernel."""
+
+    def __init__(self, mixer_norm: Norm, mixer: Mixer, mixer_out_norm: Norm, ffn_norm: Optional[Norm] = None,
+                 ffn: Optional[FeedForward] = None, ffn_out_norm: Optional[Norm] = None,
+                 names: Tuple[str, str, str, str, str, str] = ("norm1", "mix.", "norm1b", "norm2", "mlp.", "norm2b")
+                 ) -> None:
+        if len({x is None for x in (ffn_norm, ffn, ffn_out_norm)}) != 1:
+            raise ValueError("a feed-forward and its two norms come together")
+        self.mixer_norm, self._mixer, self.mixer_out_norm = mixer_norm, mixer, mixer_out_norm
+        self.ffn_norm, self.ffn, self.ffn_out_norm = ffn_norm, ffn, ffn_out_norm
+        self.names = names
+
+    @property
+    def mixer(self) -> Mixer:
+        return self._mixer
+
+    def named_parts(self) -> List[Tuple[str, Part]]:
+        parts = (self.mixer_norm, self._mixer, self.mixer_out_norm, self.ffn_norm, self.ffn, self.ffn_out_norm)
+        return [(n, p) for n, p in zip(self.names, parts) if p is not None]
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(p.graph_safe for _, p in self.named_parts())
+
+    def forward(self, ctx, residual: torch.Tensor, delta, cache: Optional[LayerCache],
+                state: Optional[torch.Tensor]):
+        if isinstance(delta, DeferredNorm):
+            raise ValueError("a block with norms around its sublayers takes no deferred norm")
+        h = self.mixer_norm.add_forward(residual, delta, ctx.act_dtype)
+        delta = PendingNormed(self._mixer.forward(ctx, h, cache, state), self.mixer_out_norm)
+        if self.ffn is not None:
+            h = self.ffn_norm.add_forward(residual, delta, ctx.act_dtype)
+            delta = PendingNormed(self.ffn.forward(ctx, h), self.ffn_out_norm)
+        return residual, delta
+
+
+register_part("block", "sandwich", SandwichBlock)
 
 
 class ChannelScale(Part):

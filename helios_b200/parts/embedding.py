@@ -32,9 +32,11 @@ class TokenEmbedding(InputStage):
 
 
 class OutputHead(Part):
-    """logits = rows x W^T, float32, without a bias."""
+    """logits = rows x W^T, float32, without a bias; with ``softcap`` c they become
+    c * tanh(logits / c)."""
 
-    def __init__(self, vocab: int, width: int, tensor_name: str = "weight") -> None:
+    def __init__(self, vocab: int, width: int, tensor_name: str = "weight", softcap: float = 0.0) -> None:
+        self.softcap = float(softcap or 0.0)
         self.vocab = vocab
         self.width = width
         self.tensor_name = tensor_name
@@ -50,7 +52,8 @@ class OutputHead(Part):
         return ops.linear_libraries(dtype)
 
     def forward(self, ctx, rows: torch.Tensor) -> torch.Tensor:
-        return ops.linear_logits(rows, self.weight)
+        logits = ops.linear_logits(rows, self.weight)
+        return ops.softcap(logits, self.softcap) if self.softcap else logits
 
 
 class NormedHead(OutputStage):

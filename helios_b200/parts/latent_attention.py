@@ -4,7 +4,9 @@ Per token the mixer keeps ONE row: the latent c (``rank`` values, RMS-normed) an
 key part r (``rot`` values) that all heads share.  Head h's key is [W_uk[h] c | r] and its
 value W_uv[h] c; a query is [q_nope (``nope`` values) | q_rot (``rot`` values, rotated)] and
 
-    score = (q_nope . W_uk[h] c + q_rot . r) * scale,     softmax over the positions <= own.
+    score = (q_nope . W_uk[h] c + q_rot . r) * scale,     softmax over the positions <= own
+
+(or the last ``window`` of them, with a sink or without).
 
 The up-projections are folded into the query and the output, so that the cache is never
 expanded: q_lat = W_uk[h]^T q_nope attends the latents themselves, and the head's output is
@@ -28,8 +30,12 @@ class LatentAttention(Mixer):
                     ``dq.norm``, the mixer's eps), q = W_uq c_q; there is no direct query matrix
     ``pairing``     "neighbours": value 2i of a rotated part is paired with value 2i + 1;
                     "halves": value i with value i + rotary_dim / 2
-    ``gate``        the concatenated heads are multiplied by sigmoid(W_g h), value by value,
-                    before the output projection
+    ``gate``        "wide" (or True): the concatenated heads are multiplied by sigmoid(W_g h), value
+                    by value, before the output projection; "head": W_g has a row per HEAD, and
+                    head h's output is multiplied by sigmoid(W_g h)_h
+    ``window``      a token sees itself and the ``window`` - 1 tokens before it
+    ``sink``        the softmax has one more key, without a value, whose score is a learned number a
+                    head (tensor ``sink``), not scaled
     ``own_rows``    False: the mixer has no W_dkv and keeps nothing; it attends the rows that
                     ANOTHER layer keeps (the plan names that layer's cache for this one's run),
                     with up-projections, queries and everything else of its own
@@ -38,8 +44,9 @@ class LatentAttention(Mixer):
     def __init__(self, width: int, heads: int, nope: int, rot: int, vdim: int, rank: int,
                  scale: float, eps: float, position,
                  names=("q", "dkv", "dkv.norm", "uk", "uv", "o"), q_rank: Optional[int] = None,
-                 pairing: str = "neighbours", gate: bool = False, own_rows: bool = True,
-                 query_names=("dq", "dq.norm", "uq"), gate_name: str = "g") -> None:
+                 pairing: str = "neighbours", gate=False, own_rows: bool = True,
+                 query_names=("dq", "dq.norm", "uq"), gate_name: str = "g", window: Optional[int] = None,
+                 sink: bool = False, sink_name: str = "sink") -> None:
         """``position``: the rotary encoding whose tables rotate the ``rot`` parts
         (``position.rotary_dim`` <= rot, even).  ``scale`` multiplies the scores as given.
         ``eps``: of the latents' RMS norms."""
@@ -47,13 +54,19 @@ class LatentAttention(Mixer):
             raise ValueError(f"{position.rotary_dim} rotated dimensions exceed the rotated part of {rot}")
         if pairing not in ops.ROTARY_PAIRINGS:
             raise ValueError(f"pairing {pairing!r} is not one of {sorted(ops.ROTARY_PAIRINGS)}")
+        if gate not in (False, True, "wide", "head"):
+            raise ValueError(f"gate {gate!r}")
         self.width, self.heads, self.nope, self.rot = width, heads, nope, rot
         self.vdim, self.rank = vdim, rank
         self.scale, self.eps = float(scale), float(eps)
         self.position = position
         self.names = tuple(names)
         self.q_rank = int(q_rank) if q_rank else None
-        self.pairing, self.gate, self.own_rows = pairing, bool(gate), bool(own_rows)
+        self.pairing, self.own_rows = pairing, bool(own_rows)
+        self.gate = "wide" if gate is True else gate
+        self._gate_rows = heads * (vdim if self.gate == "wide" else 1) if self.gate else 0
+        self.window, self.sink, self.sink_name = window, bool(sink), sink_name
+        self.sink_values = None
         self.query_names, self.gate_name = tuple(query_names), gate_name
         self.w_in = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = None
         self.norm_weight = self.query_norm_weight = None
@@ -63,7 +76,7 @@ class LatentAttention(Mixer):
         self._gate_col = self._lat_col + (rank + rot if self.own_rows else 0)
 
     def cache_spec(self) -> PagedCacheSpec:
-        return PagedCacheSpec(1, self.rank + self.rot, None, planes=1)
+        return PagedCacheSpec(1, self.rank + self.rot, self.window, planes=1)
 
     def kernel_libraries(self, dtype):
         return ops.linear_libraries(dtype, self.width) + ("latent_attention",) \
@@ -88,7 +101,9 @@ class LatentAttention(Mixer):
             specs[dkv] = WeightSpec((self.rank + self.rot, self.width))
             specs[norm] = WeightSpec((self.rank,), kind="vector", init="ones_jitter")
         if self.gate:
-            specs[self.gate_name] = WeightSpec((H * self.vdim, self.width))
+            specs[self.gate_name] = WeightSpec((self._gate_rows, self.width))
+        if self.sink:
+            specs[self.sink_name] = WeightSpec((H,), kind="vector", init="normal", std=0.5)
         return specs
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -112,6 +127,8 @@ class LatentAttention(Mixer):
         self.w_uk_t = tensors[uk].view(H, self.nope, self.rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[uv].view(H, self.vdim, self.rank).contiguous()
         self.w_o = tensors[o].contiguous()
+        if self.sink:
+            self.sink_values = tensors[self.sink_name].contiguous()
 
     def forward(self, ctx, x: torch.Tensor, cache: LayerCache, state=None) -> torch.Tensor:
         H, T = self.heads, x.shape[0]
@@ -142,10 +159,11 @@ class LatentAttention(Mixer):
             q.unflatten(1, (H, self.nope + self.rot))
         q_lat = ops.head_gemm(q[:, :, :self.nope], self.w_uk_t)
         o_lat = ops.latent_attention(ctx, q_lat, q[:, :, self.nope:], cache.k_pages, table,
-                                     self.rank, self.rot, cache.page_size, self.scale)
+                                     self.rank, self.rot, cache.page_size, self.scale, self.window,
+                                     self.sink_values)
         o = ops.head_gemm(o_lat, self.w_uv)
         if self.gate:          # the gate's launch also lays the heads side by side, whatever the product's strides
-            o = ops.gate_heads(o, proj[:, self._gate_col:self._gate_col + H * self.vdim])
+            o = ops.gate_heads(o, proj[:, self._gate_col:self._gate_col + self._gate_rows], self.gate == "head")
         else:
             o = o.reshape(T, H * self.vdim)
         return ops.linear(o, self.w_o)

@@ -7,7 +7,7 @@ from typing import Dict, Optional
 import torch
 
 from ..csrc import ops
-from .base import Norm, PendingSum, WeightSpec, register_part, settle
+from .base import Norm, PendingNormed, PendingSum, WeightSpec, register_part, settle
 
 
 class RMSNorm(Norm):
@@ -36,6 +36,13 @@ class RMSNorm(Norm):
                 return ops.add_rmsnorm_pair(residual, a, b, self.weight, None, self.eps, out_dtype)[0]
             settle(residual, delta)
             delta = None
+        elif isinstance(delta, PendingNormed):
+            # the norm after the sublayer before rides in this one's launch
+            if type(delta.norm) is RMSNorm and delta.y.dtype == out_dtype:
+                return ops.rmsnorm_add_rmsnorm(residual, delta.y, delta.norm.weight, delta.norm.eps, self.weight,
+                                               self.eps, rows)
+            settle(residual, delta)
+            delta = None
         return ops.add_rmsnorm(residual, delta, self.weight, self.eps, out_dtype, rows)
 
     @staticmethod
@@ -46,6 +53,9 @@ class RMSNorm(Norm):
         """``residual += delta`` (a tensor, a ``PendingSum`` or None), then this norm AND
         ``other`` of the new rows: (self(residual), other(residual)).  Two RMS norms with one
         eps share the row's 1 / rms, and a pending sum of plain terms rides along: one kernel."""
+        if isinstance(delta, PendingNormed):
+            settle(residual, delta)
+            delta = None
         if type(other) is RMSNorm and other.eps == self.eps and other.width == self.width:
             if isinstance(delta, PendingSum):
                 if self._plain(delta):
@@ -104,6 +114,9 @@ class LayerNorm(Norm):
             (a, sa), (b, sb) = (delta.terms + [(None, None)])[:2]
             return ops.add_layernorm(residual, self.weight, self.bias, self.eps, out_dtype, rows,
                                      a=a, scale_a=sa, b=b, scale_b=sb, mult=delta.mult)
+        if isinstance(delta, PendingNormed):
+            settle(residual, delta)
+            delta = None
         return ops.add_layernorm(residual, self.weight, self.bias, self.eps, out_dtype, rows, a=delta)
 
 
