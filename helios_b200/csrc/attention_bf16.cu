@@ -247,7 +247,7 @@ HB_EXPORT int hb_attention_decode_bf16(void* out, float* part_o, float* part_ml,
   const AttnOptions opt = {slopes, (const __nv_bfloat16*)gate, gate_stride, sink, bias_table, bias_rows,
                            sink_values, window > 0 ? keep_first : 0, gate_wide};
   const QkPrepare prep = {norm_wq, norm_wk, norm_eps, temp_coef, temp_every};
-  if ((norm_wq == nullptr) != (norm_wk == nullptr) || temp_every < 0) return HB_BAD_ARGUMENT;
+  if ((write_cache && (norm_wq == nullptr) != (norm_wk == nullptr)) || temp_every < 0) return HB_BAD_ARGUMENT;
   if (norm_wk != nullptr && !write_cache) return HB_BAD_ARGUMENT;     // a cached key is normed already
   if (nkv <= 0 || nh % nkv != 0 || nh / nkv > 16 || page_size <= 0 || n_splits < 1 ||
       (warps != 4 && warps != 8))
