@@ -447,6 +447,28 @@ def mozepel_configs(size):
     return mz, zk
 
 
+def gisodra_configs(size):
+    """(Gisodra config.json, Mozepel config.json of equal width, heads, KV heads, head size, six layers,
+    vocabulary and dense feed-forward): the package's closest model (linear attention, window
+    attention, a gated dense feed-forward).  Gisodra: latent attention, attention, gated linear
+    attention, attention on the keys and values of the second layer, gated linear attention, latent
+    attention, all windows 1,024; Mozepel as in ``mozepel_configs``."""
+    if size == "large":
+        width, heads, kv, hd, rank, ff, vocab = 2048, 16, 4, 128, 512, 8192, 32000
+    else:
+        width, heads, kv, hd, rank, ff, vocab = 1024, 8, 2, 64, 256, 4096, 32000
+    mlp, mask = {"kind": "dense", "ff": ff}, {"size": 1024}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": heads, "dim": hd, "rot_dim": hd // 2, "vdim": hd, "kv_rank": rank, "q_rank": 3 * rank // 2,
+                     "scale": (hd + hd // 2) ** -0.5, "rot": {"dims": hd // 2, "base": 10000.0}, "mask": mask}}
+    att = {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": mask}
+    gla = {"type": "gla", "mlp": mlp, "mixer": {"heads": heads, "dim": hd, "vdim": hd, "tau": 16.0, "decay_rank": 16}}
+    gs = {"architecture": "Gisodra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+          "layers": [lat, {"type": "attention", "mixer": att, "mlp": mlp}, gla,
+                     {"type": "attention", "mixer": dict(att, kv_from=1), "mlp": mlp}, gla, lat]}
+    return gs, mozepel_configs(size)[0]
+
+
 def design_configs(size, design="zokelix"):
     """(Zokelix config.json, dense decoder config.json of equal width, head count, layers, vocabulary
     and active feed-forward size) at layer sizes of a real model.  Six layers: attention over a
@@ -460,6 +482,8 @@ def design_configs(size, design="zokelix"):
         return fobanex_configs(size)
     if design == "mozepel":
         return mozepel_configs(size)
+    if design == "gisodra":
+        return gisodra_configs(size)
     if size == "large":
         width, heads, hd, rank, ff, experts, top, eff, vocab = 2048, 16, 128, 512, 8192, 32, 4, 2048, 32000
     else:
@@ -521,7 +545,8 @@ def run_design(args):
            "add_layernorm", "qk_norm_kv_write", "add_table_rows", "cast_rows",
            "add_rmsnorm_pair", "qk_rotate_norm_write", "ssm_scan", "gated_group_rmsnorm", "unary_act", "sigmoid_gate",
            "latent_prepare_parts", "linear_rows", "gate_heads", "scaled_sum_rmsnorm", "linear_attention",
-           "conv_norm_rotate_write", "pool_blocks", "pooled_attention"]
+           "conv_norm_rotate_write", "pool_blocks", "pooled_attention", "rmsnorm_add_rmsnorm", "softcap",
+           "gated_linear_attention"]
 
     def op_table(core, entries_fn, reps=3):
         """milliseconds per op name over one step, run kernel by kernel (nested ops count inside
@@ -564,7 +589,8 @@ def run_design(args):
     for size in [s for s in args.design_sizes.split(",") if s]:
         zk, dense = design_configs(size, args.design)
         res = {}
-        for label, cfg in ((args.design, zk), ({"gebasun": "mizerax", "fobanex": "mizerax", "mozepel": "zokelix"}.get(
+        for label, cfg in ((args.design, zk), ({"gebasun": "mizerax", "fobanex": "mizerax", "mozepel": "zokelix",
+                                                        "gisodra": "mozepel"}.get(
                 args.design, "dense"), dense)):
             vocab = cfg.get("vocab") or cfg["vocab_size"]
             model = DecoderModel.from_config(cfg, seed=args.seed, dtype="bfloat16", device=dev)
@@ -822,7 +848,7 @@ def main():
     ap.add_argument("--max-prompt", type=int, default=4096)
     ap.add_argument("--budget", type=int, default=2048, help="tokens a step (chunked prefill)")
     ap.add_argument("--new-tokens", type=int, default=256)
-    ap.add_argument("--design", default=None, choices=["zokelix", "mizerax", "gebasun", "fobanex", "mozepel"],
+    ap.add_argument("--design", default=None, choices=["zokelix", "mizerax", "gebasun", "fobanex", "mozepel", "gisodra"],
                     help="measure another design of the package beside its closest model of equal size "
                          "(prefill, decode, time by op) instead of the default workload")
     ap.add_argument("--design-sizes", default="small,large")
