@@ -556,12 +556,42 @@ __global__ void glu_act_kernel(T* __restrict__ out, const T* __restrict__ gu, si
   }
 }
 
+// bfloat16, I a multiple of 8: eight values a thread and step
+__global__ void __launch_bounds__(256)
+glu_act_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gu, size_t pieces, int I8,
+                      int kind, float limit) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < pieces; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / I8;
+    const uint4* row = reinterpret_cast<const uint4*>(gu) + t * 2 * I8 + (idx - t * I8);
+    const uint4 gv = row[0], uv = row[I8];
+    const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(&gv);
+    const __nv_bfloat162* up = reinterpret_cast<const __nv_bfloat162*>(&uv);
+    uint4 ov;
+    __nv_bfloat162* op = reinterpret_cast<__nv_bfloat162*>(&ov);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 g = __bfloat1622float2(gp[i]), u = __bfloat1622float2(up[i]);
+      op[i] = __floats2bfloat162_rn(glu_value(g.x, u.x, kind, limit), glu_value(g.y, u.y, kind, limit));
+    }
+    reinterpret_cast<uint4*>(out)[idx] = ov;
+  }
+}
+
 HB_EXPORT int hb_glu_act(void* out, const void* gate_up, int T, int I, int kind, float limit,
                          int act_dt, cudaStream_t stream) {
   if (T <= 0) return HB_OK;
   if (kind < 0 || kind > 2) return HB_BAD_ARGUMENT;
   const size_t total = (size_t)T * I;
   const int threads = 256;
+  if (act_dt == HB_BF16 && I % 8 == 0 && (((uintptr_t)out | (uintptr_t)gate_up) & 15) == 0) {
+    size_t blocks8 = (total / 8 + threads - 1) / threads;
+    if (blocks8 > 148 * 16) blocks8 = 148 * 16;
+    hb_launch(glu_act_bf16x8_kernel, dim3((unsigned)blocks8), dim3(threads), 0, stream, (__nv_bfloat16*)out,
+              (const __nv_bfloat16*)gate_up, total / 8, I / 8, kind, limit);
+    return hb_check_launch();
+  }
   size_t blocks = (total + threads - 1) / threads;
   if (blocks > 148 * 16) blocks = 148 * 16;
   HB_DISPATCH_DTYPE(act_dt, TA,

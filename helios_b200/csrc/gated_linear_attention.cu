@@ -186,7 +186,7 @@ gla_scan_kernel(float* __restrict__ o, T* __restrict__ out, int out_ld, GlaIn<T>
 //   D      float [tiles, heads, 5, N]: the product of the decays over every sub-chunk, then over the chunk
 //   diag   float [tiles, heads, 64, 16]: query token of the chunk x key token of the same sub-chunk
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 gla_prepare_kernel(float* __restrict__ Q, float* __restrict__ K, float* __restrict__ D, float* __restrict__ diag,
                    GlaIn<T> in, const int* __restrict__ q_tiles, const int* __restrict__ cu_tokens, int heads, int N) {
   pdl_launch_dependents();
@@ -218,17 +218,25 @@ gla_prepare_kernel(float* __restrict__ Q, float* __restrict__ K, float* __restri
     const int n = n0 + d;
     const bool live = n < N;
     const int c = h * N + (live ? n : 0);
-    float qv[GLA_SUB], kv[GLA_SUB], z[GLA_SUB];
+    if (n0 > 0) __syncthreads();
+    {
+      float qv[GLA_SUB], kv[GLA_SUB];
 #pragma unroll
-    for (int i = 0; i < GLA_SUB; ++i) {
-      const int j = sub * GLA_SUB + i;
-      const bool ok = live && j < n_tok;
-      const T* r = in.rows + (size_t)(tok0 + (ok ? j : 0)) * in.ld + c;
-      qv[i] = to_float(r[in.q_off]);
-      kv[i] = to_float(r[in.k_off]);
-      qv[i] = ok ? qv[i] * in.q_scale : 0.f;
-      kv[i] = ok ? kv[i] : 0.f;
+      for (int i = 0; i < GLA_SUB; ++i) {
+        const int j = sub * GLA_SUB + i;
+        const T* r = in.rows + (size_t)(tok0 + (j < n_tok ? j : 0)) * in.ld + c;
+        qv[i] = to_float(r[in.q_off]);
+        kv[i] = to_float(r[in.k_off]);
+      }
+#pragma unroll
+      for (int i = 0; i < GLA_SUB; ++i) {
+        const int j = sub * GLA_SUB + i;
+        const bool ok = live && j < n_tok;
+        qs[j * LA_LD + d] = ok ? qv[i] * in.q_scale : 0.f;
+        ks[j * LA_LD + d] = ok ? kv[i] : 0.f;
+      }
     }
+    float z[GLA_SUB];
     const float b = in.bias[c];
 #pragma unroll
     for (int i = 0; i < GLA_SUB; ++i) z[i] = b;
@@ -246,55 +254,48 @@ gla_prepare_kernel(float* __restrict__ Q, float* __restrict__ K, float* __restri
       }
     }
 #pragma unroll
-    for (int i = 0; i < GLA_SUB; ++i)
-      z[i] = live && sub * GLA_SUB + i < n_tok ? gla_decay(z[i], in.inv_tau) : 1.f;
-    if (n0 > 0) __syncthreads();
-#pragma unroll
     for (int i = 0; i < GLA_SUB; ++i) {
       const int j = sub * GLA_SUB + i;
-      qs[j * LA_LD + d] = qv[i];
-      ks[j * LA_LD + d] = kv[i];
+      z[i] = live && j < n_tok ? gla_decay(z[i], in.inv_tau) : 1.f;
       as[j * LA_LD + d] = z[i];
     }
+    // (a thread reads back the q and k that it wrote itself)
+    float* Dc = D + ((size_t)tile * heads + h) * 5 * N;
+    const size_t at0 = (size_t)(tok0 + sub * GLA_SUB) * heads * N + c, step = (size_t)heads * N;
+    const int own = live ? n_tok - sub * GLA_SUB : 0;            // live tokens of the sub-chunk
     float run = 1.f;
 #pragma unroll
-    for (int i = 0; i < GLA_SUB; ++i) { run *= z[i]; qv[i] *= run; }
+    for (int i = 0; i < GLA_SUB; ++i) {
+      run *= z[i];
+      if (i < own) Q[at0 + i * step] = qs[(sub * GLA_SUB + i) * LA_LD + d] * run;
+    }
     tot[sub * LA_BLK + d] = run;
-    float* Dc = D + ((size_t)tile * heads + h) * 5 * N;
     if (live) Dc[(size_t)sub * N + n] = run;
     run = 1.f;
 #pragma unroll
-    for (int i = GLA_SUB - 1; i >= 0; --i) { kv[i] *= run; run *= z[i]; }
-#pragma unroll
-    for (int i = 0; i < GLA_SUB; ++i) {
-      const int j = sub * GLA_SUB + i;
-      if (live && j < n_tok) {
-        const size_t at = (size_t)(tok0 + j) * heads * N + c;
-        Q[at] = qv[i];
-        K[at] = kv[i];
-      }
+    for (int i = GLA_SUB - 1; i >= 0; --i) {
+      if (i < own) K[at0 + i * step] = ks[(sub * GLA_SUB + i) * LA_LD + d] * run;
+      run *= z[i];
     }
     __syncthreads();
     if (sub == 0 && live)
       Dc[(size_t)4 * N + n] = (tot[d] * tot[LA_BLK + d]) * (tot[2 * LA_BLK + d] * tot[3 * LA_BLK + d]);
     // pairs inside the sub-chunk: k_j times the decays after j, from token to token
-    float4 kj[4], pair[4];
+    float4 pair[4];
 #pragma unroll
-    for (int a = 0; a < 4; ++a) {
-      kj[a] = *reinterpret_cast<const float4*>(ks + (sub * GLA_SUB + 4 * jq + a) * LA_LD + 4 * sl);
-      pair[a] = make_float4(0.f, 0.f, 0.f, 0.f);
-    }
+    for (int a = 0; a < 4; ++a) pair[a] = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < GLA_SUB; ++i) {
       const float4 q4 = *reinterpret_cast<const float4*>(qs + (sub * GLA_SUB + i) * LA_LD + 4 * sl);
       const float4 a4 = *reinterpret_cast<const float4*>(as + (sub * GLA_SUB + i) * LA_LD + 4 * sl);
+      const float4 k4 = *reinterpret_cast<const float4*>(ks + (sub * GLA_SUB + i) * LA_LD + 4 * sl);
 #pragma unroll
       for (int a = 0; a < 4; ++a) {
         const bool own = i == 4 * jq + a;
-        pair[a].x = own ? kj[a].x : pair[a].x * a4.x;
-        pair[a].y = own ? kj[a].y : pair[a].y * a4.y;
-        pair[a].z = own ? kj[a].z : pair[a].z * a4.z;
-        pair[a].w = own ? kj[a].w : pair[a].w * a4.w;
+        pair[a].x = own ? k4.x : pair[a].x * a4.x;
+        pair[a].y = own ? k4.y : pair[a].y * a4.y;
+        pair[a].z = own ? k4.z : pair[a].z * a4.z;
+        pair[a].w = own ? k4.w : pair[a].w * a4.w;
         p[a][i] = fmaf(q4.x, pair[a].x, p[a][i]);
         p[a][i] = fmaf(q4.y, pair[a].y, p[a][i]);
         p[a][i] = fmaf(q4.z, pair[a].z, p[a][i]);

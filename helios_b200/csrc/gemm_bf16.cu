@@ -43,6 +43,7 @@ struct GemmArgs {
   int T, N, K;          // tokens, output features (for GLU: of the result, = half the weight rows), reduction
   int ldo;
   int glu_offset;       // GLU: row of the weight where the second half ("up") begins
+  float glu_a, glu_b;   // GLU: g / (1 + exp(-g (glu_a + glu_b g^2))) * u (glu_value)
   int out_f32;
   int k_splits;
   int cluster_reduce;   // the K slices of a tile form a thread-block cluster and add their
@@ -55,6 +56,12 @@ struct GemmArgs {
   int slots_in = 0;                    //   rsqrt(sum(slots) / width + eps), applied to the
   float width = 1.f, eps = 0.f;        //   accumulators here
 };
+
+// The gated unit's value: g sigmoid(g (a + b g^2)) u.  a = 1, b = 0: silu(g) u.  With a = 2 sqrt(2 / pi) and
+// b = 0.044715 a it is the tanh form of gelu, since (1 + tanh z) / 2 = sigmoid(2 z).
+__device__ __forceinline__ float glu_value(float g, float u, float a, float b) {
+  return g / (1.f + __expf(-g * fmaf(b, g * g, a))) * u;
+}
 
 constexpr int SUMSQ_SLOTS = 8;   // partial sums a feature tile leaves per token (K slices or warps)
 
@@ -352,7 +359,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const bool idle = SWAP ? tile_b * BN + c + j >= args.T : idle_row;
-            val[j] = idle ? 0.f : g[j] / (1.f + __expf(-g[j])) * u[j];
+            val[j] = idle ? 0.f : glu_value(g[j], u[j], args.glu_a, args.glu_b);
           }
           if (SWAP) {
 #pragma unroll
@@ -542,7 +549,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
           for (int sp = 0; sp < 8; ++sp) { g += gv[k][sp]; u += uv[k][sp]; }
           if (SWAP && args.sumsq_in != nullptr) { g *= col_scale[c]; u *= col_scale[c]; }
           float val = g;
-          if (EPI == EPI_GLU) val = g / (1.f + __expf(-g)) * u;
+          if (EPI == EPI_GLU) val = glu_value(g, u, args.glu_a, args.glu_b);
           int t, n;
           if (SWAP) { t = tile_b * BN + c; n = tile_a * BM + rr; }
           else { t = tile_a * BM + rr; n = tile_b * OUT_COLS + c; }
@@ -713,7 +720,7 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
           tmem_ld16(taddr + 128 + c, u);
           if (t < args.T) {       // rows beyond the last token hold zeros: 0 / x is the division's slow path
 #pragma unroll
-            for (int i = 0; i < 16; ++i) val[i] = g[i] / (1.f + __expf(-g[i])) * u[i];
+            for (int i = 0; i < 16; ++i) val[i] = glu_value(g[i], u[i], args.glu_a, args.glu_b);
           }
         } else {
           tmem_ld16(taddr + c, val);
@@ -926,8 +933,9 @@ HB_EXPORT long long hb_gemm_bf16_scratch_floats(int T, int N, int swap_bn, int g
   return (long long)hb_gemm_bf16_tiles(T, N, swap_bn, glu) * k_splits * BM * cols;
 }
 
-// y[T, N] = x[T, K] w[N, K]^T (+ bias), or SwiGLU over w = [gate rows; up rows] with the up
-// rows starting at row glu_offset (then N counts the result's features).
+// y[T, N] = x[T, K] w[N, K]^T (+ bias), or a gated unit (glu 1: SwiGLU, 2: the tanh form of gelu) over
+// w = [gate rows; up rows] with the up rows starting at row glu_offset (then N counts the result's
+// features).
 //   swap_bn = 0: tokens on the M axis (tile 128 x 256).  swap_bn in {16, 32, 64, 128}: swapped,
 //   that many tokens per tile.  With 1 < k_splits <= 8 and `cluster` set, the slices of a tile
 //   run as one thread-block cluster and add up through distributed shared memory; else the
@@ -943,7 +951,7 @@ static int gemm_bf16_call(void* out, const void* x, const void* w, const float* 
   const bool clustered = k_splits > 1 && k_splits <= 8 && cluster != 0;
   if (k_splits > 1 && !clustered && (scratch == nullptr || tickets == nullptr)) return HB_BAD_ARGUMENT;
   if (k_splits > (K + BK - 1) / BK) return HB_BAD_ARGUMENT;
-  if (error == nullptr) return HB_BAD_ARGUMENT;
+  if (error == nullptr || glu < 0 || glu > 2) return HB_BAD_ARGUMENT;
   if (residual != nullptr || sumsq_in != nullptr) {
     // the epilogues of few-token steps: swapped orientation, one token tile
     if (swap_bn == 0 || T > swap_bn) return HB_BAD_ARGUMENT;
@@ -956,6 +964,8 @@ static int gemm_bf16_call(void* out, const void* x, const void* w, const float* 
   GemmArgs a;
   a.out = out; a.bias = bias; a.scratch = scratch; a.tickets = tickets; a.error = error;
   a.T = T; a.N = N; a.K = K; a.ldo = ldo; a.glu_offset = glu_offset; a.out_f32 = out_f32;
+  a.glu_a = glu == 2 ? 1.5957691216057308f : 1.f;          // 2 sqrt(2 / pi)
+  a.glu_b = glu == 2 ? 0.07135481282554186f : 0.f;
   a.k_splits = k_splits;
   a.cluster_reduce = clustered ? 1 : 0;
   a.residual = residual; a.norm_weight = norm_weight; a.sumsq_out = sumsq_out;

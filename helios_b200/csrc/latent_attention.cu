@@ -587,18 +587,31 @@ __global__ void latent_attention_merge_kernel(__nv_bfloat16* __restrict__ out,
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= n_rows) return;
   const float* ml = part_ml + (size_t)row * n_splits * 2;
-  float M = -INFINITY;
-  for (int i = 0; i < n_splits; ++i) M = fmaxf(M, ml[2 * i]);
+  // lane i holds range i's maximum and weight (at most 32 ranges)
+  const float m_i = lane < n_splits ? ml[2 * lane] : -INFINITY;
+  const float M = warp_max(m_i);
+  const float w_i = m_i == -INFINITY ? 0.f : exp2f(m_i - M);
   float L = 0.f;
-  for (int i = 0; i < n_splits; ++i) L += (ml[2 * i] == -INFINITY ? 0.f : exp2f(ml[2 * i] - M)) * ml[2 * i + 1];
+  for (int i = 0; i < n_splits; ++i) L += __shfl_sync(0xffffffffu, w_i, i) * ml[2 * i + 1];
   const float inv = latent_finish(M, L, sink, row % heads);
-  for (int d = lane; d < rank; d += 32) {
-    float a = 0.f;
+  const float* acc = part_acc + (size_t)row * n_splits * rank;
+  for (int d0 = 0; d0 < rank; d0 += 128) {           // a lane four neighbouring values (rank: a multiple of 32)
+    const int d = d0 + 4 * lane;
+    const bool on = d < rank;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
     for (int i = 0; i < n_splits; ++i) {
-      const float w = ml[2 * i] == -INFINITY ? 0.f : exp2f(ml[2 * i] - M);
-      a = fmaf(w, part_acc[((size_t)row * n_splits + i) * rank + d], a);
+      const float w = __shfl_sync(0xffffffffu, w_i, i);
+      if (!on) continue;
+      const float4 x = *reinterpret_cast<const float4*>(acc + (size_t)i * rank + d);
+      a = make_float4(fmaf(w, x.x, a.x), fmaf(w, x.y, a.y), fmaf(w, x.z, a.z), fmaf(w, x.w, a.w));
     }
-    out[(size_t)row * rank + d] = __float2bfloat16_rn(a * inv);
+    if (on) {
+      uint2 y;
+      y.x = pack_bf16(a.x * inv, a.y * inv);
+      y.y = pack_bf16(a.z * inv, a.w * inv);
+      *reinterpret_cast<uint2*>(out + (size_t)row * rank + d) = y;
+    }
   }
 }
 
@@ -614,7 +627,7 @@ HB_EXPORT int hb_latent_attention_mma(void* out, float* part_acc, float* part_ml
   if (rank <= 0 || rank % 32 || rank > 32 * LM_MAXNT || rot < 0 || rot % 16 || heads <= 0 ||
       heads_per_block <= 0 || heads_per_block > LM_ROWS || tokens_per_tile <= 0 ||
       tokens_per_tile * heads_per_block > LM_ROWS || page_size <= 0 || n_splits <= 0 ||
-      n_splits > 65535 || (n_splits > 1 && (part_acc == nullptr || part_ml == nullptr)))
+      n_splits > 32 || (n_splits > 1 && (part_acc == nullptr || part_ml == nullptr)))
     return HB_BAD_ARGUMENT;
   const int RS = rank + rot + 8;
   const size_t smem = (size_t)3 * LM_ROWS * RS * 2 + (size_t)LM_ROWS * LM_SPAD * 4 + 5 * LM_ROWS * 4 +

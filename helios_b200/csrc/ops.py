@@ -669,16 +669,20 @@ def tc_gemm_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0)
 
 
+#: gated units the tcgen05 products have an epilogue for (``linear_bf16``'s ``glu``)
+GLU_EPILOGUES = {False: 0, True: 1, "silu": 1, "gelu_tanh": 2}
+
+
 def linear_bf16(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                glu: bool = False, out_dtype: torch.dtype = torch.bfloat16,
+                glu=False, out_dtype: torch.dtype = torch.bfloat16,
                 plan=None, cluster: Optional[bool] = None, two_sm: Optional[bool] = None,
                 sumsq: Optional[torch.Tensor] = None, eps: float = 0.0,
                 residual: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None,
                 norm_out: Optional[tuple] = None):
     """y = x W^T (+ bias) on tcgen05 tensor cores; bfloat16 operands, float32 accumulate.
 
-    With ``glu`` the weight is [gate rows; up rows] ([2 I, K]) and the result is
-    silu(x gate^T) * (x up^T), [T, I].  ``out_dtype`` bfloat16 or float32.  K must be a
+    With ``glu`` (True or "silu", or "gelu_tanh") the weight is [gate rows; up rows] ([2 I, K]) and
+    the result is act(x gate^T) * (x up^T), [T, I].  ``out_dtype`` bfloat16 or float32.  K must be a
     multiple of 8 (TMA rows are 16-byte aligned); any T and N.
 
     Up to DEFERRED_NORM_MOST tokens there are two more epilogues.  ``sumsq``
@@ -698,6 +702,9 @@ def linear_bf16(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
         raise KernelError(f"the tensor-core product needs K to be a multiple of 8, got {K}")
     if glu and rows % 2:
         raise KernelError("a SwiGLU weight needs an even number of rows")
+    glu_code = GLU_EPILOGUES.get(glu)
+    if glu_code is None:
+        raise KernelError(f"the product has no epilogue for {glu!r}")
     N = rows // 2 if glu else rows
     if bias is not None:
         if glu:
@@ -742,13 +749,13 @@ def linear_bf16(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
         out = torch.empty((T, N), dtype=out_dtype, device=x.device)
     if T == 0:
         return out if residual is None else ((out, sumsq_out) if norm_weight is not None else None)
-    bn, splits = plan if plan is not None else gemm_plan(T, N, K, glu)
+    bn, splits = plan if plan is not None else gemm_plan(T, N, K, bool(glu))
     if few and (bn == 0 or T > bn):
         raise KernelError("the residual and 1 / rms epilogues need the swapped orientation and one token tile")
     if cluster is None:
         cluster = GEMM_CLUSTER_REDUCE
     # slices of a tile as a cluster: at most 8, and the partial sums must fit the stages
-    cluster = bool(cluster) and 1 < splits <= 8 and _cluster_fits(bn, glu)
+    cluster = bool(cluster) and 1 < splits <= 8 and _cluster_fits(bn, bool(glu))
     cluster_arg = 1 if cluster else 0
     if bn == 0 and splits == 1 and (GEMM_TWO_SM if two_sm is None else two_sm):
         cluster_arg = 2                      # prefill tiles on pairs of SMs (cta_group::2)
@@ -756,15 +763,15 @@ def linear_bf16(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
     lib = load_library("gemm_bf16")
     if splits > 1 and not cluster:
         lib.hb_gemm_bf16_scratch_floats.restype = ctypes.c_longlong
-        need = lib.hb_gemm_bf16_scratch_floats(T, N, bn, int(glu), splits)
-        tiles = lib.hb_gemm_bf16_tiles(T, N, bn, int(glu))
+        need = lib.hb_gemm_bf16_scratch_floats(T, N, bn, glu_code, splits)
+        tiles = lib.hb_gemm_bf16_tiles(T, N, bn, glu_code)
         if need > scratch.numel() or tiles > tickets.numel():
             raise KernelError(f"split reduction needs {need} scratch floats and {tiles} tickets; "
                               f"the work space holds {scratch.numel()} and {tickets.numel()}")
     common = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int]
     args = (_p(out), _p(x), _p(weight), _p(bias), _p(scratch), _p(tickets), _p(err), T, N, K, K, K, N,
-            rows, int(glu), N if glu else 0, 1 if out_dtype == torch.float32 else 0, bn, splits, cluster_arg)
+            rows, glu_code, N if glu else 0, 1 if out_dtype == torch.float32 else 0, bn, splits, cluster_arg)
     if few:
         f = _fn("gemm_bf16", "hb_gemm_bf16_fused",
                 common + [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p])
@@ -906,15 +913,23 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
 
 
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
-    """silu(x gate^T) * (x up^T) for ``w_gate_up`` = [gate rows; up rows]; fused into the
-    product's epilogue in bfloat16, two kernels otherwise."""
+    """``linear_glu`` with silu."""
+    return linear_glu(x, w_gate_up, "silu")
+
+
+def linear_glu(x: torch.Tensor, w_gate_up: torch.Tensor, kind: str) -> torch.Tensor:
+    """act(x gate^T) * (x up^T) for ``w_gate_up`` = [gate rows; up rows], ``kind`` "silu" or
+    "gelu_tanh"; fused into the product's epilogue in bfloat16, two kernels otherwise."""
+    def gate(rows):
+        return silu_mul(rows) if kind == "silu" else glu_act(rows, kind)
+
     if x.dtype == torch.bfloat16 and tc_gemm_supported(x, w_gate_up):
         T = x.shape[0]
         if _small_weight_library(T, w_gate_up, glu=True) or \
                 any(lo <= T <= hi for lo, hi in GEMM_LIBRARY_GLU_TOKENS):
-            return silu_mul(_library_linear(x, w_gate_up, None))
-        return linear_bf16(x, w_gate_up, glu=True)
-    return silu_mul(linear(x, w_gate_up))
+            return gate(_library_linear(x, w_gate_up, None))
+        return linear_bf16(x, w_gate_up, glu=kind)
+    return gate(linear(x, w_gate_up))
 
 
 # ------------------------------------------------------------------ sampling
@@ -1875,9 +1890,10 @@ def latent_prepare_parts(q: Optional[torch.Tensor], latent: Optional[torch.Tenso
 
 
 #: from this many tokens on the per-head products of a bfloat16 step go to the library's
-#: batched product (tensor cores); below, and in float32, this package's FMA kernel streams
-#: the small matrices once
-HEAD_GEMM_LIBRARY_TOKENS = 33
+#: batched product (tensor cores); below, and in float32, this package's FMA kernel.  Measured,
+#: microseconds a launch in a chain, FMA kernel / library: 16 heads of 128 -> 512 10.6 / 2.9 at one
+#: token, 11.4 / 3.2 at 32; 512 -> 128 28.9 / 3.7 and 31.0 / 3.5; 8 heads of 64 -> 256 5.0 / 2.7
+HEAD_GEMM_LIBRARY_TOKENS = 1
 
 
 def head_gemm(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -1910,8 +1926,8 @@ LATENT_ATTENTION_TENSOR_CORES = True
 
 def linear_rows(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     """``linear`` for rows that are a column slice of wider rows (last dimension contiguous):
-    no copy is made.  Few tokens and float32 run on ``head_gemm`` with one head, more tokens
-    in bfloat16 on the library, which takes the row stride."""
+    no copy is made.  float32 runs on ``head_gemm`` with one head, bfloat16 on the library, which
+    takes the row stride (``HEAD_GEMM_LIBRARY_TOKENS``)."""
     if x.is_contiguous():
         return linear(x, weight)
     if x.dim() != 2 or x.stride(1) != 1:

@@ -100,8 +100,8 @@ class GatedMLP(FeedForward):
             self.b_down = tensors[d + s].contiguous()
 
     def forward(self, ctx, x: torch.Tensor) -> torch.Tensor:
-        if self.activation == "silu" and not self.bias:
-            return ops.linear(ops.linear_swiglu(x, self.w_gate_up), self.w_down)
+        if self.activation in ops.GLU_EPILOGUES and not self.bias:      # fused into the product
+            return ops.linear(ops.linear_glu(x, self.w_gate_up, self.activation), self.w_down)
         gate_up = ops.linear(x, self.w_gate_up, self.b_gate_up)
         return ops.linear(ops.glu_act(gate_up, self.activation, self.limit), self.w_down, self.b_down)
 

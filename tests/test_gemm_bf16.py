@@ -20,6 +20,11 @@ def _case(T, N, K, seed, glu=False):
     return x, w, b
 
 
+def _gated(gate, up, kind):
+    act = gate * torch.sigmoid(gate) if kind in (True, "silu") else torch.nn.functional.gelu(gate, approximate="tanh")
+    return act * up
+
+
 def _close(got, want, scale=1.0):
     torch.testing.assert_close(got.double().cpu(), want, atol=2e-2 * scale, rtol=2e-2)
 
@@ -40,7 +45,7 @@ def test_plain_and_bias(T, N, K):
 @pytest.mark.parametrize("cluster", [False, True])
 @pytest.mark.parametrize("bn", [0, 16, 32, 64, 128])
 @pytest.mark.parametrize("splits", [1, 2, 5, 8])
-@pytest.mark.parametrize("glu", [False, True])
+@pytest.mark.parametrize("glu", [False, "silu", "gelu_tanh"])
 def test_every_orientation_and_split(bn, splits, glu, cluster):
     """Split reductions both ways: through scratch memory with a ticket per tile, and
     inside a thread-block cluster through distributed shared memory."""
@@ -50,8 +55,8 @@ def test_every_orientation_and_split(bn, splits, glu, cluster):
     xd, wd = x.double(), w.double()
     if glu:
         gate, up = xd @ wd[:N].T, xd @ wd[N:].T
-        want = gate * torch.sigmoid(gate) * up
-        got = ops().linear_bf16(x.to(DEV), w.to(DEV), glu=True, plan=(bn, splits), cluster=cluster)
+        want = _gated(gate, up, glu)
+        got = ops().linear_bf16(x.to(DEV), w.to(DEV), glu=glu, plan=(bn, splits), cluster=cluster)
     else:
         want = xd @ wd.T + b.double()
         got = ops().linear_bf16(x.to(DEV), w.to(DEV), b.to(DEV), plan=(bn, splits), cluster=cluster)
@@ -102,7 +107,7 @@ def test_k_that_is_no_multiple_of_8_goes_to_the_library_and_is_refused_by_the_ke
 @pytest.mark.parametrize("two_sm", [False, True])
 @pytest.mark.parametrize("T,N,K", [(129, 256, 64), (256, 512, 192), (300, 392, 1224), (2048, 4096, 1024),
                                    (1000, 1000, 520), (513, 6144, 4096)])
-@pytest.mark.parametrize("glu", [False, True])
+@pytest.mark.parametrize("glu", [False, "silu", "gelu_tanh"])
 def test_prefill_kernels_one_and_two_sm(T, N, K, glu, two_sm):
     """Tokens on the M axis: one block per 128x256 tile, and the persistent cta_group::2
     kernel (pairs of SMs on 256x256 tiles), ragged in every dimension."""
@@ -110,8 +115,8 @@ def test_prefill_kernels_one_and_two_sm(T, N, K, glu, two_sm):
     xd, wd = x.double(), w.double()
     if glu:
         gate, up = xd @ wd[:N].T, xd @ wd[N:].T
-        want = gate * torch.sigmoid(gate) * up
-        got = ops().linear_bf16(x.to(DEV), w.to(DEV), glu=True, plan=(0, 1), two_sm=two_sm)
+        want = _gated(gate, up, glu)
+        got = ops().linear_bf16(x.to(DEV), w.to(DEV), glu=glu, plan=(0, 1), two_sm=two_sm)
     else:
         want = xd @ wd.T + b.double()
         got = ops().linear_bf16(x.to(DEV), w.to(DEV), b.to(DEV), plan=(0, 1), two_sm=two_sm)
