@@ -546,7 +546,7 @@ def run_design(args):
            "add_rmsnorm_pair", "qk_rotate_norm_write", "ssm_scan", "gated_group_rmsnorm", "unary_act", "sigmoid_gate",
            "latent_prepare_parts", "linear_rows", "gate_heads", "scaled_sum_rmsnorm", "linear_attention",
            "conv_norm_rotate_write", "pool_blocks", "pooled_attention", "rmsnorm_add_rmsnorm", "softcap",
-           "gated_linear_attention", "linear_glu"]
+           "gated_linear_attention", "linear_glu", "latent_attention_expanded"]
 
     def op_table(core, entries_fn, reps=3):
         """milliseconds per op name over one step, run kernel by kernel (nested ops count inside

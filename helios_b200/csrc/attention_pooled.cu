@@ -18,6 +18,7 @@ int pooled_dispatch(int hd, int vd, F f) {
   };
   if (hd <= 64) return values(std::integral_constant<int, 64>());
   if (hd <= 128) return values(std::integral_constant<int, 128>());
+  if (hd <= 192) return values(std::integral_constant<int, 192>());
   return values(std::integral_constant<int, 256>());
 }
 

@@ -47,6 +47,8 @@ struct PooledTiles {
   int hd, vd;               // sizes (multiples of 8) at most the ones the kernel is compiled for
   int out_stride;           // elements between rows of the output
   float factor;             // a constant on the output
+  int side_by_side;         // a token's heads lie beside each other in ONE row of the maps (no page a head):
+                            // head h's columns begin at h * hd / h * vd, a page is page_size rows
 };
 
 struct AttnArgs {
@@ -203,7 +205,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                           (blocks ? key0 < blocks_last : (key0 + ps - 1 >= k_min || key0 < keep) && key0 <= p_last);
         const int count = __popc(__ballot_sync(0xffffffffu, mine));
         int row = 0;
-        if (mine) row = (tab[(key_base + lane * ps) / ps] * a.nkv + kvh) * ps;      // before the wait
+        const bool wide = POOLED && pl.side_by_side;
+        const int col = wide ? kvh * (is_v ? pl.vd : pl.hd) : 0;
+        if (mine) {                                                                 // before the wait
+          const int page = tab[(key_base + lane * ps) / ps];
+          row = wide ? page * ps : (page * a.nkv + kvh) * ps;
+        }
         int go = 1;
         if (lane == 0) {
           go = mbar_wait(bar(empty0 + s), ((it / stages) & 1) ^ 1, abort_flag, a.error, 11) ? 1 : 0;
@@ -216,7 +223,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
 #pragma unroll
           for (int hh = 0; hh < (KH > VH ? KH : VH); ++hh)
             if (hh < halves)
-              tma_load_2d(ring + s * tile_bytes + hh * HALF_BYTES + off, map, bar(full0 + s), hh * 64, row);
+              tma_load_2d(ring + s * tile_bytes + hh * HALF_BYTES + off, map, bar(full0 + s), col + hh * 64, row);
         }
       }
     }

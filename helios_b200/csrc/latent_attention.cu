@@ -10,6 +10,10 @@
 // over the positions j <= own, or, with a window W, own - W < j <= own; with `sink` (float [heads]) the
 // softmax has one more key of score sink[h] that carries no value.
 //
+// A long portion may instead expand the rows it sees to keys and values per head (a product with a
+// matrix that holds the up-projections) and attend those: `latent_gather` copies the rows of a step's
+// requests out of their pages for that product.
+//
 // Three kernels: `latent_prepare` (RMS norm of the latent, rotary on the shared key part
 // and on the queries' rotated parts, cache write), `head_gemm` (the folded products, one
 // small matrix per head) and `latent_attention` (one warp per (token, head), float32
@@ -665,5 +669,67 @@ HB_EXPORT int hb_latent_attention_mma(void* out, float* part_acc, float* part_ml
               (__nv_bfloat16*)out, (const float*)part_acc, (const float*)part_ml, n_rows, rank, n_splits, sink,
               heads);
   }
+  return hb_check_launch();
+}
+
+// ---------------------------------------------------------------- rows out of their pages
+// The pages that the step's tokens see, request by request, as consecutive pages of `dst` [most_pages *
+// page_size, width]; local_table [S, lt_stride] gets their places (logical page -> page of dst).  Rows
+// beyond a request's last token are zeros.  A block a page.
+__global__ void __launch_bounds__(128)
+latent_gather_kernel(uint4* __restrict__ dst, int* __restrict__ local_table, int lt_stride,
+                     const uint4* __restrict__ pages, const int* __restrict__ block_table, int bt_stride,
+                     const int* __restrict__ cu_tokens, const int* __restrict__ start_pos, int S, int window,
+                     int page_size, int width8) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ int found[3];                 // request, logical page, its last position + 1
+  const int b = blockIdx.x;
+  if (threadIdx.x < 32) {
+    if (threadIdx.x == 0) found[0] = -1;
+    __syncwarp();
+    int before = 0;
+    for (int s0 = 0; s0 < S; s0 += 32) {
+      const int s = s0 + threadIdx.x;
+      int n = 0, first = 0, end = 0;
+      if (s < S) {
+        const int tokens = cu_tokens[s + 1] - cu_tokens[s];
+        end = start_pos[s] + tokens;
+        first = (window > 0 ? max(0, start_pos[s] - window + 1) : 0) / page_size;
+        n = tokens > 0 ? (end - 1) / page_size - first + 1 : 0;
+      }
+      int incl = n;
+      for (int w = 1; w < 32; w <<= 1) {
+        const int x = __shfl_up_sync(0xffffffffu, incl, w);
+        if (threadIdx.x >= w) incl += x;
+      }
+      const int lo = before + incl - n;
+      if (b >= lo && b < lo + n) {
+        found[0] = s;
+        found[1] = first + b - lo;
+        found[2] = end;
+      }
+      before += __shfl_sync(0xffffffffu, incl, 31);
+      if (before > b) break;
+    }
+  }
+  __syncthreads();
+  const int seq = found[0], logical = found[1];
+  if (seq < 0) return;                     // more pages than the step sees
+  if (threadIdx.x == 0 && logical < lt_stride) local_table[(size_t)seq * lt_stride + logical] = b;
+  const int live = min(page_size, found[2] - logical * page_size) * width8;
+  const uint4* src = pages + (size_t)block_table[(size_t)seq * bt_stride + logical] * page_size * width8;
+  uint4* out = dst + (size_t)b * page_size * width8;
+  for (int i = threadIdx.x; i < page_size * width8; i += 128) out[i] = i < live ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
+HB_EXPORT int hb_latent_gather(void* dst, int most_pages, int* local_table, int lt_stride, const void* pages,
+                               const int* block_table, int bt_stride, const int* cu_tokens, const int* start_pos,
+                               int S, int window, int page_size, int width, cudaStream_t stream) {
+  if (S <= 0 || most_pages <= 0) return HB_OK;
+  if (page_size <= 0 || width <= 0 || width % 8 || lt_stride < bt_stride || (((uintptr_t)dst | (uintptr_t)pages) & 15))
+    return HB_BAD_ARGUMENT;
+  hb_launch(latent_gather_kernel, dim3(most_pages), dim3(128), 0, stream, (uint4*)dst, local_table, lt_stride,
+            (const uint4*)pages, block_table, bt_stride, cu_tokens, start_pos, S, window, page_size, width / 8);
   return hb_check_launch();
 }

@@ -1998,6 +1998,103 @@ def latent_attention(ctx, q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch
     return out
 
 
+#: portions expand the latent rows they see to keys and values per head where that is estimated to
+#: take less time than attention over the rows themselves: None: by the estimate; True / False: always
+#: (where the sizes allow) / never
+LATENT_EXPAND = None
+#: most bytes of expanded keys and values a step may make
+LATENT_EXPAND_BYTES = 2 << 30
+
+
+def latent_expand_supported(dtype: torch.dtype, heads: int, key_dim: int, value_dim: int, rank: int, rot: int,
+                            page_size: int) -> bool:
+    """Sizes for which latent rows can be expanded and attended as keys and values per head."""
+    return (dtype == torch.bfloat16 and rank % 8 == 0 and rot % 8 == 0
+            and pooled_tc_supported(heads, heads, key_dim, value_dim, page_size))
+
+
+def _visible_pages(ctx, page_size: int, window: int) -> int:
+    """Pages of rows that the step's requests see, each request's from a page of its own: what a
+    step that runs kernel by kernel has, or the most that a captured shape can."""
+    if ctx.extras.get("tile_provider") is None:
+        total = 0
+        for s in ctx.seqs:
+            if s.num_tokens:
+                first = max(0, s.start_pos - window + 1) // page_size if window else 0
+                total += (s.start_pos + s.num_tokens - 1) // page_size - first + 1
+        return total
+    most = -(-ctx.max_context_len // page_size)
+    if not window:
+        return ctx.num_seqs * most
+    return min(ctx.num_seqs * most, -(-ctx.num_tokens // page_size) + ctx.num_seqs * (-(-(window - 1) // page_size) + 2))
+
+
+def latent_expand_pages(ctx, heads: int, key_dim: int, value_dim: int, rank: int, rot: int, page_size: int,
+                        window: Optional[int]) -> int:
+    """Pages to expand in this step, or 0 where attention over the rows themselves is estimated to
+    be ahead.  The estimate counts the products over the latents at 95 TFLOP/s (``mma.sync``), the
+    expansion at 1,000, attention over heads at 300 (tcgen05), and three trips of the expanded rows
+    at 5 TB/s."""
+    if LATENT_EXPAND is False or ctx.decode_only or ctx.max_tokens_per_seq < 16:
+        return 0
+    window = int(window or 0)
+    pages = _visible_pages(ctx, page_size, window)
+    per_row = heads * (key_dim + value_dim)
+    rows = pages * page_size
+    if rows * per_row * 2 > LATENT_EXPAND_BYTES:
+        return 0
+    if LATENT_EXPAND:
+        return pages
+    pairs = ctx.num_tokens * heads * 2.0 * _keys_seen(ctx, window)
+    direct = pairs * (2 * rank + rot) / 95e6
+    expanded = 15.0 + rows * 2.0 * (rank + rot) * per_row / 1e9 + rows * per_row * 6.0 / 5e6 \
+        + pairs * (key_dim + value_dim) / 300e6
+    return pages if expanded < direct else 0
+
+
+def latent_attention_expanded(ctx, q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor,
+                              w_expand: torch.Tensor, most_pages: int, heads: int, key_dim: int, value_dim: int,
+                              page_size: int, scale: float, window: Optional[int] = None,
+                              options: Optional[AttentionOptions] = None) -> torch.Tensor:
+    """``latent_attention`` of a step with portions by way of keys and values per head: the rows the
+    step's requests see are copied out of their pages, ONE product with ``w_expand`` [heads * (key_dim +
+    value_dim), row width] makes every head's keys and values of them, and the tcgen05 prefill kernel
+    attends those.  ``q`` [T, heads * key_dim]; ``most_pages``: ``latent_expand_pages``; ``options``: a
+    sink, a gate.  Returns [T, heads * value_dim], gated."""
+    _check(q, "q", torch.bfloat16, 2)
+    _check(pages, "pages", torch.bfloat16, 4)
+    _check(block_table, "block_table", torch.int32, 2)
+    _check(w_expand, "w_expand", torch.bfloat16, 2)
+    T, width = q.shape[0], pages.shape[3]
+    columns = heads * (key_dim + value_dim)
+    if tuple(w_expand.shape) != (columns, width) or pages.shape[1] != 1 or pages.shape[2] != page_size \
+            or q.shape[1] < heads * key_dim:
+        raise KernelError(f"latent_attention_expanded: q {tuple(q.shape)}, pages {tuple(pages.shape)} and w_expand "
+                          f"{tuple(w_expand.shape)} do not fit {heads} heads of {key_dim} / {value_dim}")
+    opt = options or _NO_OPTIONS
+    rows = torch.empty((most_pages * page_size, width), dtype=torch.bfloat16, device=q.device)
+    local = torch.empty_like(block_table)
+    f = _fn("latent_attention", "hb_latent_gather",
+            [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+             c_void_p])
+    _run(f(_p(rows), most_pages, _p(local), local.shape[1], _p(pages), _p(block_table), block_table.shape[1],
+           _p(ctx.cu_tokens), _p(ctx.start_pos), ctx.num_seqs, int(window or 0), page_size, width, _stream()),
+         "latent_gather")
+    kv = linear(rows, w_expand)
+    out = torch.empty((T, heads * value_dim), dtype=torch.bfloat16, device=q.device)
+    tiles = _step_tiles(ctx, 128, True, q.device)
+    _scratch, _tickets, err = _gemm_workspace(q.device)
+    f = _fn("attention_tc_pooled", "hb_attention_rows_prefill_tc",
+            [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, ctypes.c_longlong, c_void_p, c_int, c_void_p, c_int,
+             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int,
+             c_int, c_void_p])
+    _run(f(_p(out), out.stride(0), _p(q), q.stride(0), _p(kv), kv.stride(0), kv.shape[0], _p(local), local.shape[1],
+           _p(tiles), tiles.shape[0], _p(ctx.cu_tokens), _p(ctx.start_pos), heads, key_dim, value_dim, page_size,
+           int(window or 0), float(scale), _p(err), *_sized_option_args(opt, T, heads, q, value_dim), _stream()),
+         "attention_rows_prefill_tc")
+    return out
+
+
 # ------------------------------------------------------------------ gated delta rule
 def causal_conv_silu(ctx, x: torch.Tensor, channels: int, weight: torch.Tensor,
                      conv_state: torch.Tensor, bias: Optional[torch.Tensor] = None,

@@ -10,7 +10,9 @@ value W_uv[h] c; a query is [q_nope (``nope`` values) | q_rot (``rot`` values, r
 
 The up-projections are folded into the query and the output, so that the cache is never
 expanded: q_lat = W_uk[h]^T q_nope attends the latents themselves, and the head's output is
-W_uv[h] (sum_j p_j c_j).  Rotary pairs dimension 2i with 2i + 1 over the first
+W_uv[h] (sum_j p_j c_j).  Only a long portion, for which the products over the latents are more work
+than making the keys and values per head of the rows it sees, does expand those rows for the step
+(``ops.latent_expand_pages``).  Rotary pairs dimension 2i with 2i + 1 over the first
 ``position.rotary_dim`` of the ``rot`` values.
 """
 from __future__ import annotations
@@ -68,7 +70,7 @@ class LatentAttention(Mixer):
         self.window, self.sink, self.sink_name = window, bool(sink), sink_name
         self.sink_values = None
         self.query_names, self.gate_name = tuple(query_names), gate_name
-        self.w_in = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = None
+        self.w_in = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.w_expand = None
         self.norm_weight = self.query_norm_weight = None
         # columns of the fused first projection: [queries or their latent | latent rows | gate]
         self._n_first = self.q_rank or heads * (nope + rot)
@@ -79,8 +81,9 @@ class LatentAttention(Mixer):
         return PagedCacheSpec(1, self.rank + self.rot, self.window, planes=1)
 
     def kernel_libraries(self, dtype):
+        expand = ops.latent_expand_supported(dtype, self.heads, self.nope + self.rot, self.vdim, self.rank, self.rot, 16)
         return ops.linear_libraries(dtype, self.width) + ("latent_attention",) \
-            + (("elementwise",) if self.gate else ())
+            + (("elementwise",) if self.gate else ()) + (("attention_tc_pooled",) if expand else ())
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         q, dkv, norm, uk, uv, o = self.names
@@ -127,6 +130,15 @@ class LatentAttention(Mixer):
         self.w_uk_t = tensors[uk].view(H, self.nope, self.rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[uv].view(H, self.vdim, self.rank).contiguous()
         self.w_o = tensors[o].contiguous()
+        self.w_expand = None
+        if ops.latent_expand_supported(self.w_o.dtype, H, self.nope + self.rot, self.vdim, self.rank, self.rot, 16):
+            # a row [c | r] -> every head's key [W_uk c | r], then every head's value W_uv c
+            key = torch.zeros((H, self.nope + self.rot, self.rank + self.rot), dtype=self.w_o.dtype, device=self.w_o.device)
+            key[:, :self.nope, :self.rank] = tensors[uk].view(H, self.nope, self.rank)
+            key[:, self.nope:, self.rank:] = torch.eye(self.rot, dtype=key.dtype, device=key.device)
+            value = torch.zeros((H * self.vdim, self.rank + self.rot), dtype=key.dtype, device=key.device)
+            value[:, :self.rank] = tensors[uv]
+            self.w_expand = torch.cat([key.view(-1, self.rank + self.rot), value], dim=0).contiguous()
         if self.sink:
             self.sink_values = tensors[self.sink_name].contiguous()
 
@@ -155,6 +167,16 @@ class LatentAttention(Mixer):
         else:
             q = first
             prepare(q, latent, None)
+        kd = self.nope + self.rot
+        if self.w_expand is not None and q.dtype == torch.bfloat16 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 \
+                and ops.latent_expand_supported(q.dtype, H, kd, self.vdim, self.rank, self.rot, cache.page_size):
+            pages = ops.latent_expand_pages(ctx, H, kd, self.vdim, self.rank, self.rot, cache.page_size, self.window)
+            if pages:
+                gate = proj[:, self._gate_col:self._gate_col + self._gate_rows] if self.gate else None
+                options = ops.AttentionOptions(sink_values=self.sink_values, gate=gate, gate_wide=self.gate == "wide")
+                return ops.linear(ops.latent_attention_expanded(ctx, q, cache.k_pages, table, self.w_expand, pages, H, kd,
+                                                                self.vdim, cache.page_size, self.scale, self.window,
+                                                                options), self.w_o)
         q = q.view(T, H, self.nope + self.rot) if q.is_contiguous() else \
             q.unflatten(1, (H, self.nope + self.rot))
         q_lat = ops.head_gemm(q[:, :, :self.nope], self.w_uk_t)

@@ -676,6 +676,70 @@ def test_latent_window_and_sink_single_out_rows_at_every_edge(dtype, H, rank, ro
         assert (got[r] - want[r]).abs().max() < tol * float(want[r].abs().max()), case
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("captured", [False, True])
+@pytest.mark.parametrize("H,nope,rot,vd,rank,page,W", [
+    (4, 32, 16, 32, 64, 16, 40), (3, 128, 64, 128, 512, 16, 130), (5, 40, 24, 16, 96, 8, 17), (2, 64, 32, 64, 128, 32, 1),
+    (6, 24, 8, 48, 32, 16, None), (2, 192, 64, 96, 64, 64, 300), (16, 16, 16, 16, 32, 16, 16)])
+def test_latent_rows_expanded_to_keys_and_values_per_head(H, nope, rot, vd, rank, page, W, captured):
+    """Four requests in one step (a portion deep in a request, a whole prompt, a single token, a portion
+    of 16): every query singles out one visible row, or one just outside the window.  Pages the window
+    has passed hold NaN and are gone from the tables.  ``captured``: the page count is the bound a
+    captured shape takes."""
+    from helios_b200.csrc import ops
+    from helios_b200.parts.latent_attention import LatentAttention
+
+    g = torch.Generator().manual_seed(H * rank + vd)
+    bf = torch.bfloat16
+    starts, parts = [333, 0, 210, 61], [70, 145, 1, 16]
+    part = LatentAttention(64, H, nope, rot, vd, rank, 0.3, 1e-5, SimpleNamespace(rotary_dim=rot), q_rank=16,
+                           pairing="halves", gate="head", window=W, sink=True)
+    tensors = {n: torch.randn(s.shape, generator=g).cuda() for n, s in part.weight_specs().items()}
+    tensors = {n: (t * rank ** -0.5).to(bf) if part.weight_specs()[n].kind == "matrix" else t for n, t in tensors.items()}
+    part.bind(tensors)
+    uk, uv = tensors["uk"].double().cpu(), tensors["uv"].double().cpu()
+    sink = torch.linspace(-3.0, 25.0, H)
+    gate = (torch.randn(sum(parts), H + 3, generator=g) * 2).to(bf)
+    tables, q_rows, want, off, pool = [], [], [], 0, []
+    most = max(-(-(s + n) // page) for s, n in zip(starts, parts))
+    for s, n in zip(starts, parts):
+        L = s + n
+        rows = torch.randn(L, 1, rank + rot, generator=g).to(bf)
+        first = max(0, s - W + 1) if W else 0
+        kp, _v, table = _pages_for(rows.float(), None, first, page, bf, g)
+        table = torch.where(table >= 0, table + off, table)
+        tables.append(torch.cat([table, torch.full((1, most - table.shape[1]), -1, dtype=torch.int32)], 1))
+        pool.append(kp)
+        off += kp.shape[0]
+        x = rows[:, 0].double()
+        k = torch.cat([(x[:, :rank] @ uk.T).view(L, H, nope), x[:, None, rank:].expand(L, H, rot)], -1)
+        v = (x[:, :rank] @ uv.T).view(L, H, vd)
+        targets = [max(0, min(s + i, [s + i, s + i - (W or 200) + 1, s + i - (W or 200), 0, s + i - 3][i % 5])) for i in range(n)]
+        q = torch.stack([k[j] / k[j].norm(dim=-1, keepdim=True) * 12.0 for j in targets]).to(bf)
+        q_rows.append(q.view(n, -1))
+        want.append(pg.window_softmax_attention(q.double(), k, v, 0.3, s + torch.arange(n), W, sink.double()))
+    ctx = _ctx(parts, [0, 1, 2, 3], starts=starts, tables=[torch.cat(tables).contiguous().cuda()])
+    if captured:
+        ctx.extras["tile_provider"] = lambda tile, longest: ops.query_tiles(
+            parts, tile, "cuda", starts if longest else None)
+    key_dim = nope + rot
+    kept, ops.LATENT_EXPAND = ops.LATENT_EXPAND, True
+    try:
+        n_pages = ops.latent_expand_pages(ctx, H, key_dim, vd, rank, rot, page, W)
+    finally:
+        ops.LATENT_EXPAND = kept
+    exact = sum((s + n - 1) // page - (max(0, s - W + 1) if W else 0) // page + 1 for s, n in zip(starts, parts))
+    assert n_pages == exact if not captured else n_pages >= exact
+    options = ops.AttentionOptions(sink_values=sink.cuda(), gate=gate.cuda()[:, 2:2 + H])
+    got = ops.latent_attention_expanded(ctx, torch.cat(q_rows).contiguous().cuda(), torch.cat(pool), ctx.block_tables[0],
+                                        part.w_expand, n_pages, H, key_dim, vd, page, 0.3, W, options)
+    want = torch.cat(want) * torch.sigmoid(gate.double()[:, 2:2 + H])[:, :, None]
+    got = got.double().cpu().view(-1, H, vd)
+    assert torch.isfinite(got).all()
+    err = (got - want).abs().amax(-1) / want.abs().amax()
+    assert float(err.max()) < 2.5e-2, (float(err.max()), divmod(int(err.argmax()), H))
+
+
 # ====================================================================== one key that stands out, in whole models
 def _marked_model(kind, W):
     if kind == "attention":
@@ -852,6 +916,28 @@ def test_mixed_batches_with_pages_and_slots_used_again(gs_folders, name, dtype, 
     core = _core(gs_folders[name], dtype, tb.live_tokens_peak, max_slots=3, graphs=graphs)
     _check(tb, tu.run_in_process(core, tb), plain, dtype, f"{name} mixed")
     assert core.cache.num_free_slots == 3 and all(p.num_used == 0 for p in core.cache.pools)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("graphs", [True, False])
+@pytest.mark.parametrize("name", ["latent_only", "gs_a", "gs_c"])
+def test_models_whose_portions_expand_their_latent_rows(gs_folders, name, graphs, monkeypatch):
+    """Portions of 16 tokens and more by way of keys and values per head, beside decoded tokens and
+    shorter portions that attend the rows themselves."""
+    from helios_b200.csrc import ops
+
+    made = []
+    monkeypatch.setattr(ops, "LATENT_EXPAND", True)
+    inner = ops.latent_attention_expanded
+    monkeypatch.setattr(ops, "latent_attention_expanded", lambda *a, **kw: made.append(1) or inner(*a, **kw))
+    cfg, weights = read_folder(gs_folders[name])
+    reqs = _requests(cfg, [140, 23, 277, 18, 52, 131], 700)
+    plain = _plain(cfg, weights, "bfloat16", reqs)
+    tb = tu.TraceBuilder()
+    tu.mixed(tb, reqs, seed=5, max_live=3, decode_tail=10, portion_choices=(2, 16, 40, 70))
+    core = _core(gs_folders[name], "bfloat16", tb.live_tokens_peak, max_slots=3, graphs=graphs)
+    _check(tb, tu.run_in_process(core, tb), plain, "bfloat16", f"{name} expanded")
+    assert made
 
 
 @pytest.mark.gpu
