@@ -32,7 +32,7 @@ constexpr int BK = 64;           // 64 bfloat16 = 128 bytes = one swizzle span
 constexpr int UMMA_K = 16;
 constexpr int GEMM_THREADS = 192;  // warp 0: TMA, warp 1: MMA + tensor memory, warps 2-5: epilogue
 
-enum { EPI_STORE = 0, EPI_GLU = 1 };
+enum { EPI_STORE = 0, EPI_GLU = 1, EPI_GELU = 2 };     // EPI_GELU: the two-SM kernel's second gated unit
 
 struct GemmArgs {
   void* out;            // [T, ldo] bfloat16 or float32
@@ -61,6 +61,14 @@ struct GemmArgs {
 // b = 0.044715 a it is the tanh form of gelu, since (1 + tanh z) / 2 = sigmoid(2 z).
 __device__ __forceinline__ float glu_value(float g, float u, float a, float b) {
   return g / (1.f + __expf(-g * fmaf(b, g * g, a))) * u;
+}
+
+constexpr float GELU_A = 1.5957691216057308f, GELU_B = 0.044715f * GELU_A;       // 2 sqrt(2 / pi)
+
+// The second of the two, its constants known and its division the approximate one (a denominator
+// too large for it belongs to a value that is 0): for the kernel whose epilogue is long.
+__device__ __forceinline__ float gelu_value(float g, float u) {
+  return __fdividef(g, 1.f + __expf(-g * fmaf(GELU_B, g * g, GELU_A))) * u;
 }
 
 constexpr int SUMSQ_SLOTS = 8;   // partial sums a feature tile leaves per token (K slices or warps)
@@ -611,7 +619,8 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
   const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
   const int kb_total = (args.K + BK - 1) / BK;
   const int n_tiles = tiles_m * tiles_n;             // tiles of 256 x 256
-  constexpr int RESULT_COLS = (EPI == EPI_GLU) ? 128 : 256;
+  constexpr bool GATED = EPI != EPI_STORE;
+  constexpr int RESULT_COLS = GATED ? 128 : 256;
 
   auto full_bar = [&](int s) { return smem_u32(bars + s); };
   auto empty_bar = [&](int s) { return smem_u32(bars + T2_STAGES + s); };
@@ -651,7 +660,7 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
         const int q = pair + j * n_pairs;
         const int tile_m = q % tiles_m, tile_n = q / tiles_m;
         const int a_row = tile_m * 256 + (int)rank * 128;
-        const int b_row = (EPI == EPI_GLU) ? (rank ? args.glu_offset : 0) + tile_n * 128
+        const int b_row = GATED ? (rank ? args.glu_offset : 0) + tile_n * 128
                                            : tile_n * 256 + (int)rank * 128;
         for (int kb = 0; kb < kb_total; ++kb, ++it) {
           const int s = it % T2_STAGES;
@@ -714,13 +723,14 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
       const int t = tile_m * 256 + (int)rank * 128 + r;
       for (int c = 0; c < RESULT_COLS; c += 16) {
         float val[16];
-        if (EPI == EPI_GLU) {
+        if (GATED) {
           float g[16], u[16];
           tmem_ld16(taddr + c, g);
           tmem_ld16(taddr + 128 + c, u);
           if (t < args.T) {       // rows beyond the last token hold zeros: 0 / x is the division's slow path
 #pragma unroll
-            for (int i = 0; i < 16; ++i) val[i] = glu_value(g[i], u[i], args.glu_a, args.glu_b);
+            for (int i = 0; i < 16; ++i)
+              val[i] = EPI == EPI_GELU ? gelu_value(g[i], u[i]) : g[i] / (1.f + __expf(-g[i])) * u[i];
           }
         } else {
           tmem_ld16(taddr + c, val);
@@ -851,7 +861,7 @@ int launch_2sm(const void* x, const void* w, const GemmArgs& args, int w_rows, i
     sm_counts[dev] = n;
   }
   const int sm_count = sm_counts[dev];
-  const int per_tile = (EPI == EPI_GLU) ? 128 : 256;
+  const int per_tile = EPI != EPI_STORE ? 128 : 256;
   const int tiles_m = (args.T + 255) / 256, tiles_n = (args.N + per_tile - 1) / per_tile;
   const int n_tiles = tiles_m * tiles_n;
   int pairs = sm_count / 2;
@@ -964,8 +974,8 @@ static int gemm_bf16_call(void* out, const void* x, const void* w, const float* 
   GemmArgs a;
   a.out = out; a.bias = bias; a.scratch = scratch; a.tickets = tickets; a.error = error;
   a.T = T; a.N = N; a.K = K; a.ldo = ldo; a.glu_offset = glu_offset; a.out_f32 = out_f32;
-  a.glu_a = glu == 2 ? 1.5957691216057308f : 1.f;          // 2 sqrt(2 / pi)
-  a.glu_b = glu == 2 ? 0.07135481282554186f : 0.f;
+  a.glu_a = glu == 2 ? GELU_A : 1.f;
+  a.glu_b = glu == 2 ? GELU_B : 0.f;
   a.k_splits = k_splits;
   a.cluster_reduce = clustered ? 1 : 0;
   a.residual = residual; a.norm_weight = norm_weight; a.sumsq_out = sumsq_out;
@@ -974,8 +984,9 @@ static int gemm_bf16_call(void* out, const void* x, const void* w, const float* 
   return glu ? launch<BN_, SWAP_, EPI_GLU>(x, w, a, w_rows, ldx, ldw, stream)                 \
              : launch<BN_, SWAP_, EPI_STORE>(x, w, a, w_rows, ldx, ldw, stream)
   if (swap_bn == 0 && k_splits == 1 && cluster == 2)    // prefill: a persistent kernel on pairs of SMs
-    return glu ? launch_2sm<EPI_GLU>(x, w, a, w_rows, ldx, ldw, stream)
-               : launch_2sm<EPI_STORE>(x, w, a, w_rows, ldx, ldw, stream);
+    return glu == 2 ? launch_2sm<EPI_GELU>(x, w, a, w_rows, ldx, ldw, stream)
+           : glu    ? launch_2sm<EPI_GLU>(x, w, a, w_rows, ldx, ldw, stream)
+                    : launch_2sm<EPI_STORE>(x, w, a, w_rows, ldx, ldw, stream);
   switch (swap_bn) {
     case 0: HB_GEMM_CASE(256, false);
     case 16: HB_GEMM_CASE(16, true);
