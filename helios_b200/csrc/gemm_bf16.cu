@@ -11,9 +11,9 @@
 //     on a narrow N axis, so that a step streams every weight once at full width; the
 //     K range can be split over several blocks, whose partial sums the last block to
 //     finish adds in a fixed order (scratch memory + a ticket per tile).
-// Epilogues: + bias, bfloat16 or float32 out; or SwiGLU, where the block accumulates the
+// Epilogues: + bias, bfloat16 or float32 out; or a gated unit, where the block accumulates the
 // gate tile and the up tile of the same feature range side by side and writes
-// silu(gate) * up.
+// silu(gate) * up (SwiGLU), or gelu(gate) * up with the tanh form of gelu.
 // Two more for steps of few tokens (swapped orientation), which together take the RMSNorm
 // launches out of a decode step: a product can ADD its result into the float32 residual
 // stream and leave, for the norm that follows, bfloat16(residual * norm weight) and per-token
@@ -32,7 +32,7 @@ constexpr int BK = 64;           // 64 bfloat16 = 128 bytes = one swizzle span
 constexpr int UMMA_K = 16;
 constexpr int GEMM_THREADS = 192;  // warp 0: TMA, warp 1: MMA + tensor memory, warps 2-5: epilogue
 
-enum { EPI_STORE = 0, EPI_GLU = 1, EPI_GELU = 2 };     // EPI_GELU: the two-SM kernel's second gated unit
+enum { EPI_STORE = 0, EPI_GLU = 1, EPI_GELU = 2 };     // plain | silu(g) u | gelu(g) u, the tanh form
 
 struct GemmArgs {
   void* out;            // [T, ldo] bfloat16 or float32
@@ -43,7 +43,6 @@ struct GemmArgs {
   int T, N, K;          // tokens, output features (for GLU: of the result, = half the weight rows), reduction
   int ldo;
   int glu_offset;       // GLU: row of the weight where the second half ("up") begins
-  float glu_a, glu_b;   // GLU: g / (1 + exp(-g (glu_a + glu_b g^2))) * u (glu_value)
   int out_f32;
   int k_splits;
   int cluster_reduce;   // the K slices of a tile form a thread-block cluster and add their
@@ -57,18 +56,16 @@ struct GemmArgs {
   float width = 1.f, eps = 0.f;        //   accumulators here
 };
 
-// The gated unit's value: g sigmoid(g (a + b g^2)) u.  a = 1, b = 0: silu(g) u.  With a = 2 sqrt(2 / pi) and
-// b = 0.044715 a it is the tanh form of gelu, since (1 + tanh z) / 2 = sigmoid(2 z).
-__device__ __forceinline__ float glu_value(float g, float u, float a, float b) {
-  return g / (1.f + __expf(-g * fmaf(b, g * g, a))) * u;
-}
-
-constexpr float GELU_A = 1.5957691216057308f, GELU_B = 0.044715f * GELU_A;       // 2 sqrt(2 / pi)
-
-// The second of the two, its constants known and its division the approximate one (a denominator
-// too large for it belongs to a value that is 0): for the kernel whose epilogue is long.
-__device__ __forceinline__ float gelu_value(float g, float u) {
-  return __fdividef(g, 1.f + __expf(-g * fmaf(GELU_B, g * g, GELU_A))) * u;
+// The gated unit's value.  The tanh form of gelu is g sigmoid(2 z), z = sqrt(2 / pi) (g + 0.044715 g^3),
+// since (1 + tanh z) / 2 = sigmoid(2 z); its division is the approximate one (a denominator too large
+// for it belongs to a value that is 0).
+template <int EPI>
+__device__ __forceinline__ float glu_value(float g, float u) {
+  if (EPI == EPI_GELU) {
+    constexpr float A = 1.5957691216057308f, B = 0.044715f * A;       // 2 sqrt(2 / pi)
+    return __fdividef(g, 1.f + __expf(-g * fmaf(B, g * g, A))) * u;
+  }
+  return g / (1.f + __expf(-g)) * u;
 }
 
 constexpr int SUMSQ_SLOTS = 8;   // partial sums a feature tile leaves per token (K slices or warps)
@@ -78,7 +75,7 @@ constexpr uint32_t pow2_cols(int n) { return n <= 32 ? 32 : n <= 64 ? 64 : n <= 
 template <int BN, bool SWAP, int EPI>
 struct Config {
   // A-side tiles per stage: two for the swapped SwiGLU (gate rows, up rows)
-  static constexpr int A_TILES = (SWAP && EPI == EPI_GLU) ? 2 : 1;
+  static constexpr int A_TILES = (SWAP && EPI != EPI_STORE) ? 2 : 1;
   static constexpr int A_BYTES = BM * BK * 2;
   static constexpr int B_BYTES = BN * BK * 2;
   static constexpr int STAGE_BYTES = A_TILES * A_BYTES + B_BYTES;
@@ -149,7 +146,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
     b_row0 = tile_b * BN;                       // token rows
   } else {
     a_row0 = tile_a * BM;                       // token rows
-    if (EPI == EPI_GLU) {
+    if (EPI != EPI_STORE) {
       b_row0 = tile_b * (BN / 2);               // gate rows
       b_row1 = args.glu_offset + tile_b * (BN / 2);
     } else {
@@ -174,7 +171,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
       if (SWAP) {
         tma_load_2d(sa, &map_a, full_bar(s), k0, a_row0);
         if (Cfg::A_TILES == 2) tma_load_2d(sa + Cfg::A_BYTES, &map_a, full_bar(s), k0, a_row1);
-      } else if (EPI == EPI_GLU) {
+      } else if (EPI != EPI_STORE) {
         tma_load_2d(sb, &map_b, full_bar(s), k0, b_row0);
         tma_load_2d(sb + Cfg::B_BYTES / 2, &map_b, full_bar(s), k0, b_row1);
       } else {
@@ -349,7 +346,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
           else reinterpret_cast<__nv_bfloat16*>(args.out)[(size_t)t * args.ldo + n] = __float2bfloat16_rn(val);
         }
       };
-      if (EPI == EPI_GLU) {
+      if (EPI != EPI_STORE) {
         constexpr int HALF = SWAP ? BN : BN / 2;   // columns of the gate accumulator
         for (int c = 0; c < HALF; c += 16) {
           if (SWAP && tile_b * BN + c >= args.T) break;           // columns without tokens
@@ -367,7 +364,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const bool idle = SWAP ? tile_b * BN + c + j >= args.T : idle_row;
-            val[j] = idle ? 0.f : glu_value(g[j], u[j], args.glu_a, args.glu_b);
+            val[j] = idle ? 0.f : glu_value<EPI>(g[j], u[j]);
           }
           if (SWAP) {
 #pragma unroll
@@ -515,8 +512,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
         }
       }
     } else if (warp >= 2 && !*abort_flag) {
-      constexpr int OUT_COLS = (EPI == EPI_GLU && !SWAP) ? BN / 2 : BN;   // columns of the result tile
-      constexpr int GLU_SHIFT = (EPI == EPI_GLU) ? (SWAP ? BN : BN / 2) : 0;
+      constexpr int OUT_COLS = (EPI != EPI_STORE && !SWAP) ? BN / 2 : BN;   // columns of the result tile
+      constexpr int GLU_SHIFT = (EPI != EPI_STORE) ? (SWAP ? BN : BN / 2) : 0;
       const uint32_t part_addr = base;
       const int S = args.k_splits;
       // swapped: only the columns that hold tokens are shared out (the others are padding of
@@ -543,7 +540,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
           for (int sp = 0; sp < 8; ++sp) {
             const bool on = live[k] && sp < S;
             gv[k][sp] = on ? ld_peer_smem(part_addr + (uint32_t)(c * BM + rr) * 4u, sp) : 0.f;
-            uv[k][sp] = (EPI == EPI_GLU && on)
+            uv[k][sp] = (EPI != EPI_STORE && on)
                             ? ld_peer_smem(part_addr + (uint32_t)((GLU_SHIFT + c) * BM + rr) * 4u, sp) : 0.f;
           }
         }
@@ -557,7 +554,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
           for (int sp = 0; sp < 8; ++sp) { g += gv[k][sp]; u += uv[k][sp]; }
           if (SWAP && args.sumsq_in != nullptr) { g *= col_scale[c]; u *= col_scale[c]; }
           float val = g;
-          if (EPI == EPI_GLU) val = glu_value(g, u, args.glu_a, args.glu_b);
+          if (EPI != EPI_STORE) val = glu_value<EPI>(g, u);
           int t, n;
           if (SWAP) { t = tile_b * BN + c; n = tile_a * BM + rr; }
           else { t = tile_a * BM + rr; n = tile_b * OUT_COLS + c; }
@@ -729,8 +726,7 @@ gemm_bf16_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
           tmem_ld16(taddr + 128 + c, u);
           if (t < args.T) {       // rows beyond the last token hold zeros: 0 / x is the division's slow path
 #pragma unroll
-            for (int i = 0; i < 16; ++i)
-              val[i] = EPI == EPI_GELU ? gelu_value(g[i], u[i]) : g[i] / (1.f + __expf(-g[i])) * u[i];
+            for (int i = 0; i < 16; ++i) val[i] = glu_value<EPI>(g[i], u[i]);
           }
         } else {
           tmem_ld16(taddr + c, val);
@@ -799,7 +795,7 @@ int launch(const void* x, const void* w, const GemmArgs& args, int w_rows, int l
     if (!make_map(&map_b, x, args.T, args.K, ldx, BN)) return HB_LAUNCH_FAILED;
   } else {
     if (!make_map(&map_a, x, args.T, args.K, ldx, BM)) return HB_LAUNCH_FAILED;
-    if (!make_map(&map_b, w, w_rows, args.K, ldw, EPI == EPI_GLU ? BN / 2 : BN)) return HB_LAUNCH_FAILED;
+    if (!make_map(&map_b, w, w_rows, args.K, ldw, EPI != EPI_STORE ? BN / 2 : BN)) return HB_LAUNCH_FAILED;
   }
   auto kernel = gemm_bf16_kernel<BN, SWAP, EPI>;
   // the shared-memory limit is a per-device attribute of the kernel
@@ -815,7 +811,7 @@ int launch(const void* x, const void* w, const GemmArgs& args, int w_rows, int l
   if (SWAP) {
     grid = dim3((args.N + BM - 1) / BM, (args.T + BN - 1) / BN, args.k_splits);
   } else {
-    const int per_tile = (EPI == EPI_GLU) ? BN / 2 : BN;
+    const int per_tile = (EPI != EPI_STORE) ? BN / 2 : BN;
     grid = dim3((args.T + BM - 1) / BM, (args.N + per_tile - 1) / per_tile, args.k_splits);
   }
   if (args.cluster_reduce) {
@@ -974,14 +970,13 @@ static int gemm_bf16_call(void* out, const void* x, const void* w, const float* 
   GemmArgs a;
   a.out = out; a.bias = bias; a.scratch = scratch; a.tickets = tickets; a.error = error;
   a.T = T; a.N = N; a.K = K; a.ldo = ldo; a.glu_offset = glu_offset; a.out_f32 = out_f32;
-  a.glu_a = glu == 2 ? GELU_A : 1.f;
-  a.glu_b = glu == 2 ? GELU_B : 0.f;
   a.k_splits = k_splits;
   a.cluster_reduce = clustered ? 1 : 0;
   a.residual = residual; a.norm_weight = norm_weight; a.sumsq_out = sumsq_out;
   a.sumsq_in = sumsq_in; a.slots_in = slots_in; a.width = (float)K; a.eps = eps;
 #define HB_GEMM_CASE(BN_, SWAP_)                                                              \
-  return glu ? launch<BN_, SWAP_, EPI_GLU>(x, w, a, w_rows, ldx, ldw, stream)                 \
+  return glu == 2 ? launch<BN_, SWAP_, EPI_GELU>(x, w, a, w_rows, ldx, ldw, stream)           \
+             : glu ? launch<BN_, SWAP_, EPI_GLU>(x, w, a, w_rows, ldx, ldw, stream)           \
              : launch<BN_, SWAP_, EPI_STORE>(x, w, a, w_rows, ldx, ldw, stream)
   if (swap_bn == 0 && k_splits == 1 && cluster == 2)    // prefill: a persistent kernel on pairs of SMs
     return glu == 2 ? launch_2sm<EPI_GELU>(x, w, a, w_rows, ldx, ldw, stream)
