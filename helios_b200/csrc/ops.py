@@ -2063,11 +2063,13 @@ def latent_attention_expanded(ctx, q: torch.Tensor, pages: torch.Tensor, block_t
     step's requests see are copied out of their pages, ONE product with ``w_expand`` [heads * (key_dim +
     value_dim), row width] makes every head's keys and values of them, and the tcgen05 prefill kernel
     attends those.  ``q`` [T, heads * key_dim]; ``most_pages``: ``latent_expand_pages``; ``options``: a
-    sink, a gate.  Returns [T, heads * value_dim], gated."""
-    _check(q, "q", torch.bfloat16, 2)
+    sink, a gate.  Rows of q may be strided.  Returns [T, heads * value_dim], gated."""
     _check(pages, "pages", torch.bfloat16, 4)
     _check(block_table, "block_table", torch.int32, 2)
     _check(w_expand, "w_expand", torch.bfloat16, 2)
+    if not q.is_cuda or q.dim() != 2 or q.dtype != torch.bfloat16 or q.stride(1) != 1 or q.stride(0) % 8 \
+            or q.data_ptr() % 16:
+        raise KernelError("latent_attention_expanded: q must be bfloat16 rows at 16-byte boundaries")
     T, width = q.shape[0], pages.shape[3]
     columns = heads * (key_dim + value_dim)
     if tuple(w_expand.shape) != (columns, width) or pages.shape[1] != 1 or pages.shape[2] != page_size \

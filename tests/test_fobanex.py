@@ -730,6 +730,32 @@ def test_mixed_batches_with_pages_and_slots_used_again(fb_folders, name, dtype, 
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("graphs", [True, False])
+@pytest.mark.parametrize("name", ["latent_borrowed", "fb_a", "fb_c"])
+def test_models_whose_portions_expand_their_latent_rows(fb_folders, name, graphs, monkeypatch):
+    """Portions of 16 tokens and more by way of keys and values per head (a gate per value, rows that
+    another layer keeps), beside decoded tokens that attend the rows."""
+    from helios_b200.csrc import ops
+
+    made = []
+    monkeypatch.setattr(ops, "LATENT_EXPAND", True)
+    inner = ops.latent_attention_expanded
+    monkeypatch.setattr(ops, "latent_attention_expanded", lambda *a, **kw: made.append(1) or inner(*a, **kw))
+    cfg, weights = read_folder(fb_folders[name])
+    reqs = _requests(cfg, [140, 23, 177, 18, 52, 131], 700)
+    plain = _plain(cfg, weights, "bfloat16", reqs)
+    tb = tu.TraceBuilder()
+    tu.mixed(tb, reqs, seed=5, max_live=3, decode_tail=10, portion_choices=(2, 16, 40, 70))
+    core = _core(fb_folders[name], "bfloat16", tb.live_tokens_peak, max_slots=3, graphs=graphs)
+    got = tu.run_in_process(core, tb)
+    assert made
+    for step, rows in tb.rows.items():               # root mean square over the vocabulary, relative to the row's
+        want = torch.stack([plain[rid][pos] for rid, pos in rows])
+        err = (torch.from_numpy(got[step]).double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
+        assert float(err.max()) < 0.04, (name, tb.steps[step], rows[int(err.argmax())], float(err.max()))
+
+
+@pytest.mark.gpu
 @pytest.mark.parametrize("name", ["fb_a", "fb_b"])
 def test_a_batch_gives_each_request_what_it_gets_alone(fb_folders, name):
     """float32: the same rows bit for bit, alone or beside others, in one step or in portions,

@@ -731,7 +731,8 @@ def test_latent_rows_expanded_to_keys_and_values_per_head(H, nope, rot, vd, rank
     exact = sum((s + n - 1) // page - (max(0, s - W + 1) if W else 0) // page + 1 for s, n in zip(starts, parts))
     assert n_pages == exact if not captured else n_pages >= exact
     options = ops.AttentionOptions(sink_values=sink.cuda(), gate=gate.cuda()[:, 2:2 + H])
-    got = ops.latent_attention_expanded(ctx, torch.cat(q_rows).contiguous().cuda(), torch.cat(pool), ctx.block_tables[0],
+    wide = torch.cat([torch.cat(q_rows), torch.full((sum(parts), 24), float("nan"), dtype=bf)], 1).cuda()
+    got = ops.latent_attention_expanded(ctx, wide[:, :H * key_dim], torch.cat(pool), ctx.block_tables[0],
                                         part.w_expand, n_pages, H, key_dim, vd, page, 0.3, W, options)
     want = torch.cat(want) * torch.sigmoid(gate.double()[:, 2:2 + H])[:, :, None]
     got = got.double().cpu().view(-1, H, vd)

@@ -630,6 +630,28 @@ def test_mixed_batches_with_pages_and_slots_used_again(zk_folders, name, dtype, 
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("graphs", [True, False])
+@pytest.mark.parametrize("name", ["latent_only", "zk_a", "zk_b"])
+def test_models_whose_portions_expand_their_latent_rows(zk_folders, name, graphs, monkeypatch):
+    """Portions of 16 tokens and more by way of keys and values per head (no window, no sink, no
+    gate; the queries are columns of wider rows), beside decoded tokens that attend the rows."""
+    from helios_b200.csrc import ops
+
+    made = []
+    monkeypatch.setattr(ops, "LATENT_EXPAND", True)
+    inner = ops.latent_attention_expanded
+    monkeypatch.setattr(ops, "latent_attention_expanded", lambda *a, **kw: made.append(1) or inner(*a, **kw))
+    cfg, weights = read_folder(zk_folders[name])
+    reqs = _requests(cfg, [140, 23, 177, 18, 52, 131], 700)
+    plain = _plain(cfg, weights, "bfloat16", reqs)
+    tb = tu.TraceBuilder()
+    tu.mixed(tb, reqs, seed=5, max_live=3, decode_tail=10, portion_choices=(2, 16, 40, 70))
+    core = _core(zk_folders[name], "bfloat16", tb.live_tokens_peak, max_slots=3, graphs=graphs)
+    _check(tb, tu.run_in_process(core, tb), plain, "bfloat16", f"{name} expanded")
+    assert made
+
+
+@pytest.mark.gpu
 def test_a_batch_gives_each_request_what_it_gets_alone(zk_folders):
     """float32: the same rows bit for bit, alone or beside others, whatever the slots and pages."""
     from helios_b200.engine.batch import StepEntry
